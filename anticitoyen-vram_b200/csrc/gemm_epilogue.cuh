@@ -21,8 +21,9 @@ struct GemmParams {
     const float* bias;      // float [N]: added to the product's feature n before anything else is made of it (null: none)
     const float* row_scale; // act 2, and act 0 with tokens on rows: w of each row of A (null: 1)
     float glu_limit, glu_alpha;
-    int gate_fn;            // act 1: what the gate passes through: 0 silu (with the roundings of the unfused path), 1 the tanh
-                            // form of gelu (in float on the accumulators, the product rounded once)
+    int gate_fn;            // act 1: what the pair becomes: 0 silu(gate) * up (with the roundings of the unfused path), 1 the
+                            // tanh form of gelu instead (in float on the accumulators, the product rounded once), 2 the
+                            // clamped gated unit of act 2 without a row scale (tokens on rows or on columns)
     int unary;              // act 0: an activation on every output (with tokens on rows: after the row's scale)
                             // (1 gelu by tanh, 2 silu, 3 gelu by erf; 0: none)
     // grouped product (tokens on rows): tile ta of A multiplies the rows [tile_expert[ta] * N, +N) of the B operand,
@@ -77,7 +78,6 @@ __device__ __forceinline__ bf16 geglu_pair(float gate, float up) {
     const float t = tanhf(0.7978845608028654f * (gate + 0.044715f * gate * gate * gate));
     return __float2bfloat16_rn(0.5f * gate * (1.f + t) * up);
 }
-__device__ __forceinline__ bf16 gated_pair(float gate, float up, int fn) { return fn ? geglu_pair(gate, up) : swiglu_pair(gate, up); }
 
 // An activation on one output (GemmParams.unary), in float.
 __device__ __forceinline__ float unary_act(float z, int kind) {
@@ -94,17 +94,22 @@ __device__ __forceinline__ bf16 glu_clamped_pair(float gate, float up, float w, 
     return __float2bfloat16_rn(g * __fdividef(1.f, 1.f + __expf(-alpha * g)) * (u + 1.f));
 }
 
+__device__ __forceinline__ bf16 gated_pair(const GemmParams& p, float gate, float up) {
+    if (p.gate_fn == 2) return glu_clamped_pair(gate, up, 1.f, p.glu_limit, p.glu_alpha);
+    return p.gate_fn ? geglu_pair(gate, up) : swiglu_pair(gate, up);
+}
+
 // Swapped roles: features lie on lanes, an even lane holds the gate of 16 tokens and the next lane their up.  The two
 // share the work: each sends the other the eight values that it does not need, the even lane makes the tokens 0..7,
 // the odd lane the tokens 8..15 (all exchanges first, then the arithmetic, so that the eight chains run side by
 // side: done token by token, with the odd lane idle, this took 75 ns a token).  Returns the first of this lane's tokens.
-__device__ __forceinline__ int swiglu_lane_pair(const float (&v)[16], int lane, bf16 (&o)[8], int fn = 0) {
+__device__ __forceinline__ int swiglu_lane_pair(const GemmParams& p, const float (&v)[16], int lane, bf16 (&o)[8]) {
     const bool odd = lane & 1;
     float other[8];
 #pragma unroll
     for (int c = 0; c < 8; ++c) other[c] = __shfl_xor_sync(0xffffffffu, odd ? v[c] : v[c + 8], 1);
 #pragma unroll
-    for (int c = 0; c < 8; ++c) o[c] = gated_pair(odd ? other[c] : v[c], odd ? v[c + 8] : other[c], fn);
+    for (int c = 0; c < 8; ++c) o[c] = gated_pair(p, odd ? other[c] : v[c], odd ? v[c + 8] : other[c]);
     return odd ? 8 : 0;
 }
 
@@ -132,7 +137,7 @@ __device__ __forceinline__ void gt_store16(const GemmParams& p, int row_a, int c
     if (p.act) {
         if (p.swap) {       // features lie on lanes: an even lane holds a gate, the next lane its up
             bf16 o[8];
-            const int first = swiglu_lane_pair(v, lane, o, p.gate_fn);
+            const int first = swiglu_lane_pair(p, v, lane, o);
             const int f = row_a & ~1;           // the pair's gate row
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
@@ -148,7 +153,7 @@ __device__ __forceinline__ void gt_store16(const GemmParams& p, int row_a, int c
                 for (int k = 0; k < 8; ++k) o[k] = glu_clamped_pair(v[2 * k], v[2 * k + 1], w, p.glu_limit, p.glu_alpha);
             } else {
 #pragma unroll
-                for (int k = 0; k < 8; ++k) o[k] = gated_pair(v[2 * k], v[2 * k + 1], p.gate_fn);
+                for (int k = 0; k < 8; ++k) o[k] = gated_pair(p, v[2 * k], v[2 * k + 1]);
             }
             if (col0 + 16 <= p.N && (((uintptr_t)dst) & 15) == 0) {
                 *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(o);
@@ -219,7 +224,7 @@ __device__ __forceinline__ void gt_store16_rows(const GemmParams& p, int row_a, 
 __device__ __forceinline__ void gt_stage16(const GemmParams& p, unsigned char* stage, int f, int col0, const float (&v)[16], int lane) {
     if (p.act) {            // an even lane holds a gate, the next lane its up: 64 output features per tile
         bf16 o[8];
-        const int first = swiglu_lane_pair(v, lane, o, p.gate_fn);
+        const int first = swiglu_lane_pair(p, v, lane, o);
 #pragma unroll
         for (int c = 0; c < 8; ++c) reinterpret_cast<bf16*>(stage)[(col0 + first + c) * 64 + (f >> 1)] = o[c];
     } else if (p.out_f32) {

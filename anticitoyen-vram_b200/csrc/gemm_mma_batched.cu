@@ -6,7 +6,8 @@
 // sums of the latent attention).  The tcgen05 product of the framework takes one weight for all rows; here every batch
 // has its own small one (64 to 512 on a side), so a CTA computes a 64 x 64 tile of one batch with mma.sync m16n8k16,
 // four warps of 16 rows each, K in steps of 64 through two cp.async buffers (rows padded by 16 bytes against bank
-// conflicts).  acv_gemm_simt_batched takes what this kernel refuses (float32, K or strides that are no 16-byte pieces).
+// conflicts).  With a gate ([M][batches][N], any strides) every element of C is multiplied by sigmoid of the gate's, in
+// float.  acv_gemm_simt_batched takes what this kernel refuses (float32, K or strides that are no 16-byte pieces).
 #include "mma_tiles.cuh"
 
 #define GB_BM 64
@@ -16,7 +17,8 @@
 
 __global__ void __launch_bounds__(128)
 gemm_mma_batched_kernel(const bf16* __restrict__ A, int lda, long long a_batch, const bf16* __restrict__ W, int ldw,
-                        long long w_batch, bf16* __restrict__ C, int ldc, long long c_batch, int M, int N, int K) {
+                        long long w_batch, bf16* __restrict__ C, int ldc, long long c_batch, int M, int N, int K,
+                        const bf16* __restrict__ gate, int ldg, long long g_batch) {
     __shared__ __align__(128) unsigned char a_s[2][GB_BM * GB_PITCH];
     __shared__ __align__(128) unsigned char w_s[2][GB_BN * GB_PITCH];
     pdl_launch_dependents();
@@ -26,6 +28,7 @@ gemm_mma_batched_kernel(const bf16* __restrict__ A, int lda, long long a_batch, 
     A += (size_t)b * a_batch;
     W += (size_t)b * w_batch;
     C += (size_t)b * c_batch;
+    if (gate) gate += (size_t)b * g_batch;
     const int nk = (K + GB_BK - 1) / GB_BK;
 
     auto load = [&](int kt) {
@@ -74,8 +77,15 @@ gemm_mma_batched_kernel(const bf16* __restrict__ A, int lda, long long a_batch, 
 #pragma unroll
         for (int i = 0; i < GB_BN / 8; ++i) {
             const int gn = n0 + i * 8 + c_lo;
-            if (gn < N)     // N is even: the pair is inside
-                *reinterpret_cast<__nv_bfloat162*>(C + (size_t)gm * ldc + gn) = __floats2bfloat162_rn(acc[i][2 * hh], acc[i][2 * hh + 1]);
+            if (gn < N) {   // N is even: the pair is inside
+                float x = acc[i][2 * hh], y = acc[i][2 * hh + 1];
+                if (gate) {
+                    const __nv_bfloat162 z = *reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)gm * ldg + gn);
+                    x *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(z.x)));
+                    y *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(z.y)));
+                }
+                *reinterpret_cast<__nv_bfloat162*>(C + (size_t)gm * ldc + gn) = __floats2bfloat162_rn(x, y);
+            }
         }
     }
 }
@@ -89,12 +99,14 @@ ACV_API int acv_gemm_mma_batched_takes(const void* A, int lda, long long a_batch
 }
 
 ACV_API int acv_gemm_mma_batched(const void* A, int lda, long long a_batch, const void* W, int ldw, long long w_batch,
-                                 void* C, int ldc, long long c_batch, int M, int N, int K, int batches, cudaStream_t stream) {
+                                 void* C, int ldc, long long c_batch, int M, int N, int K, int batches, const void* gate,
+                                 int ldg, long long g_batch, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || batches <= 0) return 0;
     if (!acv_gemm_mma_batched_takes(A, lda, a_batch, W, ldw, w_batch, C, ldc, c_batch, N, K)) return ACV_ERR_ALIGN;
+    if (gate && (ldg % 2 || g_batch % 2 || ((uintptr_t)gate & 3))) return ACV_ERR_ALIGN;
     dim3 grid((N + GB_BN - 1) / GB_BN, (M + GB_BM - 1) / GB_BM, batches);
     if (grid.y > 65535 || batches > 65535) return ACV_ERR_SIZE;
     acv_launch(PDL_GEMM, gemm_mma_batched_kernel, grid, dim3(128), 0, stream, (const bf16*)A, lda, a_batch, (const bf16*)W, ldw,
-               w_batch, (bf16*)C, ldc, c_batch, M, N, K);
+               w_batch, (bf16*)C, ldc, c_batch, M, N, K, (const bf16*)gate, ldg, g_batch);
     return acv_launch_status();
 }

@@ -822,7 +822,7 @@ static int gemm_tc_run(GemmParams& p, const void* x, int ldx, const void* w, int
     p.gate_fn = p.act == 1 ? act >> 4 : 0;
     p.unary = p.act == 0 ? act >> 4 : 0;
     act = p.act;
-    if (p.gate_fn > 1 || p.unary > 3 || (p.row_scale && act == 0 && (swap || splits > 1))) return ACV_ERR_SIZE;
+    if (p.gate_fn > 2 || p.unary > 3 || (p.row_scale && act == 0 && (swap || splits > 1))) return ACV_ERR_SIZE;
     if (act && (out_f32 || (N & 1))) return ACV_ERR_SIZE;
     if (act == 2 && swap) return ACV_ERR_SIZE;
     if (p.tile_expert && (swap || splits > 1 || (flags & 6) || p.experts < 1 || (N % 8))) return ACV_ERR_SIZE;
@@ -882,14 +882,15 @@ ACV_API int acv_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* C,
 }
 
 // The same with a bias: float [N], added to feature n of the product before the activation (for the paired SiLU form
-// the bias lists the pairs as the weight's rows do).
+// the bias lists the pairs as the weight's rows do; null: none).  limit, alpha: of the clamped gated unit (gate_fn 2).
 ACV_API int acv_gemm_tc_bias(const void* x, int ldx, const void* w, int ldw, void* C, int ldc, int M, int N, int K,
                              int out_f32, int act, int swap, int bn, int splits, float* workspace, long long workspace_floats,
                              int* counters, long long n_counters, int* status, int sm_count, int stages, int flags,
-                             const float* bias, cudaStream_t stream) {
+                             const float* bias, float limit, float alpha, cudaStream_t stream) {
     GemmParams p = {};
     p.qkv = 0;
     p.bias = bias;
+    p.glu_limit = limit; p.glu_alpha = alpha;
     return gemm_tc_run(p, x, ldx, w, ldw, C, ldc, M, N, K, out_f32, act, swap, bn, splits, workspace, workspace_floats,
                        counters, n_counters, status, sm_count, stages, flags, stream);
 }

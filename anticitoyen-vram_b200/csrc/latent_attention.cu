@@ -15,12 +15,18 @@
 //     [c | r] goes into the token's row of its page (a page index < 0 writes nothing);
 //   q rows [H][D + R]: rot(q_h[D:]) goes to q_out[h][KR:], beside the place where the caller's per-head product leaves
 //     W_uk,h^T q_h[:D].
-// rot turns the interleaved pairs (2i, 2i+1), 2i < rot, by the angle of pair i at the token's position (cos and sin
-// from a float table [positions][rot]: rot/2 cosines, then rot/2 sines); elements from rot on pass unchanged.
+// rot turns the interleaved pairs (2i, 2i+1), 2i < rot, or with `halves` the pairs (i, i + rot/2), by the angle of pair i at
+// the token's position (cos and sin from a float table [positions][rot]: rot/2 cosines, then rot/2 sines); elements from
+// rot on pass unchanged.  A layer that reads rows kept by another one gives no kv: queries only.
 #include "common.cuh"
 
-__device__ __forceinline__ float rot_interleaved(const float* x, int e, int rot, const float* cs) {
+__device__ __forceinline__ float rot_pairs(const float* x, int e, int rot, const float* cs, int halves) {
     if (e >= rot) return x[e];
+    if (halves) {
+        const int m = rot >> 1, i = e < m ? e : e - m;
+        const float c = cs[i], s = cs[m + i];
+        return e < m ? fmaf(x[e], c, -x[e + m] * s) : fmaf(x[e], c, x[e - m] * s);
+    }
     const int i = e >> 1;
     const float c = cs[i], s = cs[(rot >> 1) + i];
     return (e & 1) ? fmaf(x[e], c, x[e - 1] * s) : fmaf(x[e], c, -x[e + 1] * s);
@@ -32,7 +38,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* 
                                       const float* __restrict__ cos_sin, int rot, int table_rows,
                                       const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                                       const int* __restrict__ block_table, int bt_stride, const int* __restrict__ bt_rows,
-                                      T* __restrict__ pages, int page_size, int num_pages, int H, int D, int R, int KR) {
+                                      T* __restrict__ pages, int page_size, int num_pages, int H, int D, int R, int KR, int halves) {
     extern __shared__ float sm[];           // [KR + R] the kv row, then [H * R] the heads' rotated parts
     __shared__ float red[32];
     pdl_launch_dependents();
@@ -43,12 +49,14 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* 
     const float* cs = cos_sin + (size_t)pos * rot;
     float* row = sm;
     float* qr = sm + KR + R;
-    const T* kvr = kv + (size_t)t * kv_stride;
     float ss = 0.f;
-    for (int e = tid; e < KR + R; e += nthr) {
-        const float v = to_f32(kvr[e]);
-        row[e] = v;
-        if (e < KR) ss = fmaf(v, v, ss);
+    if (kv) {
+        const T* kvr = kv + (size_t)t * kv_stride;
+        for (int e = tid; e < KR + R; e += nthr) {
+            const float v = to_f32(kvr[e]);
+            row[e] = v;
+            if (e < KR) ss = fmaf(v, v, ss);
+        }
     }
     for (int i = tid; i < H * R; i += nthr) {
         const int h = i / R, e = i - h * R;
@@ -58,15 +66,15 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* 
     const float inv = 1.f / sqrtf(ss / (float)KR + eps);
     for (int i = tid; i < H * R; i += nthr) {
         const int h = i / R, e = i - h * R;
-        q_out[(size_t)t * qo_stride + (size_t)h * (KR + R) + KR + e] = from_f32<T>(rot_interleaved(qr + h * R, e, rot, cs));
+        q_out[(size_t)t * qo_stride + (size_t)h * (KR + R) + KR + e] = from_f32<T>(rot_pairs(qr + h * R, e, rot, cs, halves));
     }
-    if (!pages) return;
+    if (!pages || !kv) return;
     const int seq = seq_of_token[t];
     const int pg = block_table[(size_t)(bt_rows ? bt_rows[seq] : seq) * bt_stride + positions[t] / page_size];
     if (pg < 0 || pg >= num_pages) return;
     T* dst = pages + ((size_t)pg * page_size + (positions[t] % page_size)) * (KR + R);
     for (int e = tid; e < KR; e += nthr) dst[e] = from_f32<T>(row[e] * inv * w[e]);
-    for (int e = tid; e < R; e += nthr) dst[KR + e] = from_f32<T>(rot_interleaved(row + KR, e, rot, cs));
+    for (int e = tid; e < R; e += nthr) dst[KR + e] = from_f32<T>(rot_pairs(row + KR, e, rot, cs, halves));
 }
 
 // q: rows of H*(D+R) at q_stride; q_out: rows of H*(KR+R) at qo_stride; kv: rows of KR+R at kv_stride; w float [KR];
@@ -75,7 +83,7 @@ ACV_API int acv_latent_prepare(const void* q, int q_stride, void* q_out, int qo_
                                const float* w, float eps, const float* cos_sin, int rot, int table_rows,
                                const int* positions, const int* seq_of_token, const int* block_table, int bt_stride,
                                const int* bt_rows, void* pages, int page_size, int num_pages, int T_tokens, int H, int D,
-                               int R, int KR, int dtype, cudaStream_t stream) {
+                               int R, int KR, int dtype, int halves, cudaStream_t stream) {
     if (T_tokens <= 0) return 0;
     if (H <= 0 || D < 0 || R <= 0 || KR <= 0 || rot < 0 || rot > R || (rot & 1) || (rot && (!cos_sin || table_rows <= 0)))
         return ACV_ERR_SIZE;
@@ -91,7 +99,7 @@ ACV_API int acv_latent_prepare(const void* q, int q_stride, void* q_out, int qo_
         }                                                                                                               \
         acv_launch(PDL_ROPE, latent_prepare_kernel<T>, T_tokens, threads, smem, stream, (const T*)q, q_stride, (T*)q_out, \
                    qo_stride, (const T*)kv, kv_stride, w, eps, cos_sin, rot, table_rows, positions, seq_of_token,       \
-                   block_table, bt_stride, bt_rows, (T*)pages, page_size, num_pages, H, D, R, KR);                      \
+                   block_table, bt_stride, bt_rows, (T*)pages, page_size, num_pages, H, D, R, KR, halves);                      \
     } while (0)
     if (dtype == ACV_F32) LP_LAUNCH(float);
     else if (dtype == ACV_BF16) LP_LAUNCH(bf16);

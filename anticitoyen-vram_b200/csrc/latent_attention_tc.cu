@@ -37,6 +37,7 @@ struct LatentArgs {
     int n_split;            // CTAs that share the rows of a one-token request (1: none)
     float* part_acc;        // n_split > 1: [n_dec][n_split][NH][KR] unnormalised sums
     float* part_ml;         //              [n_dec][n_split][NH][2] running maximum (in powers of two) and sum
+    const float* sinks;     // [NH] or null: exp(sink_h) joins the denominator, once for a row
 };
 
 template <int BN, int S, int NDV>
@@ -301,7 +302,12 @@ attn_latent_tc_kernel(const LatentArgs a) {
     for (int hh = 0; hh < 2; ++hh) {
         const int R = rg * 16 + r_lo + hh * 8;
         if (R >= n_rows) continue;
-        const float inv = l_run[hh] > 0.f ? 1.f / l_run[hh] : 0.f;
+        float inv = l_run[hh] > 0.f ? 1.f / l_run[hh] : 0.f;
+        if (a.sinks) {          // (a row of the unit has seen a key: m_run is finite)
+            const float sk = a.sinks[h_first + R % HPC] * LT_LOG2E, M = fmaxf(m_run[hh], sk);
+            const float al = fast_exp2(m_run[hh] - M);
+            inv = al / fmaf(l_run[hh], al, fast_exp2(sk - M));
+        }
         bf16* o = a.out + (size_t)(tok0 + R / HPC) * a.out_stride + (size_t)(h_first + R % HPC) * KR + sl * NDV * 16 + c_lo;
 #pragma unroll
         for (int i = 0; i < 2 * NDV; ++i)
@@ -314,15 +320,18 @@ attn_latent_tc_kernel(const LatentArgs a) {
 // a block a (request, head), a thread a few columns
 __global__ void attn_latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                          const int* __restrict__ dec_tokens, bf16* __restrict__ out, int out_stride,
-                                         int n_split, int NH, int KR) {
+                                         int n_split, int NH, int KR, const float* __restrict__ sinks) {
     pdl_launch_dependents();
     pdl_wait();
     const int i = blockIdx.x / NH, h = blockIdx.x % NH;
     float M = -INFINITY;
     for (int s = 0; s < n_split; ++s) M = fmaxf(M, part_ml[(((size_t)i * n_split + s) * NH + h) * 2]);
+    const bool any = M != -INFINITY;
+    if (any && sinks) M = fmaxf(M, sinks[h] * LT_LOG2E);
+    const float L0 = any && sinks ? fast_exp2(sinks[h] * LT_LOG2E - M) : 0.f;
     for (int e = threadIdx.x; e < KR; e += blockDim.x) {
-        float sum = 0.f, L = 0.f;
-        if (M != -INFINITY)
+        float sum = 0.f, L = L0;
+        if (any)
             for (int s = 0; s < n_split; ++s) {
                 const size_t at = ((size_t)i * n_split + s) * NH + h;
                 const float m = part_ml[at * 2];
@@ -380,7 +389,7 @@ static int launch_latent_tc(const LatentArgs& a, const LatentShape& sh, cudaStre
     acv_launch(PDL_ATTN, attn_latent_tc_kernel<BN, S, NDV>, dim3(units * a.HB), dim3(a.RG * S * 32), sh.smem, stream, a);
     if (a.n_split > 1 && a.n_dec > 0)
         acv_launch(PDL_ATTN, attn_latent_merge_kernel, dim3(a.n_dec * a.NH), dim3(128), 0, stream, (const float*)a.part_acc,
-                   (const float*)a.part_ml, a.dec_tokens, a.out, a.out_stride, a.n_split, a.NH, a.KR);
+                   (const float*)a.part_ml, a.dec_tokens, a.out, a.out_stride, a.n_split, a.NH, a.KR, a.sinks);
     return acv_launch_status();
 }
 
@@ -399,7 +408,7 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
                                     const int* dec_seqs, int n_dec, const int* cu_q, const int* kv_len,
                                     const int* block_table, int bt_stride, const int* bt_rows, int NH, int ROW, int KR,
                                     int page_size, int num_pages, float scale, int window, int n_split, float* part_acc,
-                                    float* part_ml, cudaStream_t stream) {
+                                    float* part_ml, const float* sinks, cudaStream_t stream) {
     if (n_split < 1 || (n_split > 1 && (!part_acc || !part_ml))) return ACV_ERR_SIZE;
     if (n_tiles < 0) n_tiles = 0;
     if (n_dec < 0) n_dec = 0;
@@ -410,7 +419,7 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
         return ACV_ERR_ALIGN;
     LatentArgs a = {(const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)pages, tile_seq, tile_q0, n_tiles,
                     dec_tokens, dec_seqs, n_dec, cu_q, kv_len, block_table, bt_stride, bt_rows, NH, ROW, KR, page_size,
-                    num_pages, scale, window, sh.TOK, sh.HPC, sh.HB, sh.RG, n_split, part_acc, part_ml};
+                    num_pages, scale, window, sh.TOK, sh.HPC, sh.HB, sh.RG, n_split, part_acc, part_ml, sinks};
 #define LT_CASE(B, SS, N) if (sh.BN == B && sh.S == SS && sh.NDV == N) return launch_latent_tc<B, SS, N>(a, sh, stream);
     LT_CASE(64, 1, 4) LT_CASE(64, 1, 8) LT_CASE(64, 2, 8) LT_CASE(64, 4, 8)
     LT_CASE(32, 1, 4) LT_CASE(32, 1, 8) LT_CASE(32, 2, 8) LT_CASE(32, 4, 8)

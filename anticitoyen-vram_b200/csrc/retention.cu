@@ -288,8 +288,8 @@ ACV_API int acv_retention(const void* q, const void* k, const void* v, int ld, c
 // out[t][u*group + e] = o / sqrt(mean_e(o^2) + eps) * w[u*group + e] * gate_fn(gate) * out_scale over groups of `group`
 // elements (a head's DV: each head by itself; all H*DV: the heads side by side normed together); w null: no weight;
 // gate_fn silu (0) or sigmoid (1).  One warp per (token, group).
-template <typename T>
-__global__ void retention_gate_kernel(const float* __restrict__ o, int ldo, const T* __restrict__ gate, int ldg,
+template <typename TG, typename T>
+__global__ void retention_gate_kernel(const float* __restrict__ o, int ldo, const TG* __restrict__ gate, int ldg,
                                       T* __restrict__ out, int ld_out, int groups, int group, const float* __restrict__ w,
                                       int gate_kind, float eps, float out_scale, int T_tokens) {
     pdl_launch_dependents();
@@ -303,7 +303,7 @@ __global__ void retention_gate_kernel(const float* __restrict__ o, int ldo, cons
     for (int e = lane; e < group; e += 32) ss = fmaf(orow[e], orow[e], ss);
     ss = warp_sum(ss);
     const float inv = out_scale / sqrtf(ss / (float)group + eps);
-    const T* grow = gate + (size_t)t * ldg + (size_t)u * group;
+    const TG* grow = gate + (size_t)t * ldg + (size_t)u * group;
     const float* wr = w ? w + (size_t)u * group : nullptr;
     T* dst = out + (size_t)t * ld_out + (size_t)u * group;
     for (int e = lane; e < group; e += 32) {
@@ -317,16 +317,19 @@ __global__ void retention_gate_kernel(const float* __restrict__ o, int ldo, cons
 
 ACV_API int acv_retention_gate(const float* o, int ldo, const void* gate, int ldg, void* out, int ld_out, int T_tokens,
                                int H, int DV, float eps, float out_scale, int dtype, const float* weight, int joint,
-                               int gate_kind, cudaStream_t stream) {
+                               int gate_kind, int gate_dtype, cudaStream_t stream) {
     if (T_tokens <= 0) return 0;
     const int warps = 8;
     const int groups = joint ? 1 : H, group = joint ? H * DV : DV;
     const int grid = (T_tokens * groups + warps - 1) / warps;
-    if (dtype == ACV_F32)
-        acv_launch(PDL_MISC, retention_gate_kernel<float>, grid, warps * 32, 0, stream, o, ldo, (const float*)gate, ldg,
+    if (dtype == ACV_F32 && gate_dtype == ACV_F32)
+        acv_launch(PDL_MISC, retention_gate_kernel<float, float>, grid, warps * 32, 0, stream, o, ldo, (const float*)gate, ldg,
                    (float*)out, ld_out, groups, group, weight, gate_kind, eps, out_scale, T_tokens);
-    else if (dtype == ACV_BF16)
-        acv_launch(PDL_MISC, retention_gate_kernel<bf16>, grid, warps * 32, 0, stream, o, ldo, (const bf16*)gate, ldg,
+    else if (dtype == ACV_BF16 && gate_dtype == ACV_F32)
+        acv_launch(PDL_MISC, retention_gate_kernel<float, bf16>, grid, warps * 32, 0, stream, o, ldo, (const float*)gate, ldg,
+                   (bf16*)out, ld_out, groups, group, weight, gate_kind, eps, out_scale, T_tokens);
+    else if (dtype == ACV_BF16 && gate_dtype == ACV_BF16)
+        acv_launch(PDL_MISC, retention_gate_kernel<bf16, bf16>, grid, warps * 32, 0, stream, o, ldo, (const bf16*)gate, ldg,
                    (bf16*)out, ld_out, groups, group, weight, gate_kind, eps, out_scale, T_tokens);
     else
         return ACV_ERR_DTYPE;

@@ -89,11 +89,15 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_block_gates_mma": [P, P, P, P, P, P, F, P, P, I, I, I, P],
         "acv_gated_scan": [P, P, P, I, P, P, P, P, P, P, I, P, I, P, I, I, I, I, I, P],
         "acv_retention": [P, P, P, I, P, I, I, P, P, F, P, P, P, P, P, I, P, I, P, I, I, I, I, I, I, I, P],
-        "acv_retention_gate": [P, I, P, I, P, I, I, I, I, F, F, I, P, I, I, P],
+        "acv_retention_gate": [P, I, P, I, P, I, I, I, I, F, F, I, P, I, I, I, P],
+        "acv_delta_prepare": [P, I, P, P, P, P, I, I, I, I, P],
+        "acv_delta": [P, I, P, P, P, P, P, P, I, I, I, P],
+        "acv_delta_step_takes": [I, I],
+        "acv_delta_step": [P, I, P, P, P, F, P, P, P, P, I, I, I, I, I, I, P],
         "acv_gemm_simt": [P, I, P, I, P, I, I, I, I, I, I, P],
-        "acv_gemm_simt_batched": [P, I, LL, P, I, LL, P, I, LL, I, I, I, I, I, I, P],
+        "acv_gemm_simt_batched": [P, I, LL, P, I, LL, P, I, LL, I, I, I, I, I, I, P, I, LL, P],
         "acv_gemm_mma_batched_takes": [P, I, LL, P, I, LL, P, I, LL, I, I],
-        "acv_gemm_mma_batched": [P, I, LL, P, I, LL, P, I, LL, I, I, I, I, P],
+        "acv_gemm_mma_batched": [P, I, LL, P, I, LL, P, I, LL, I, I, I, I, P, I, LL, P],
         "acv_attention_mixed": [P, I, P, I, P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, P, F, P, P, I, I, P, I, P],
         "acv_attention_mixed_tc_takes": [I, I, I, I, I],
         "acv_attention_mixed_dec_takes": [I, I, I, I, I],
@@ -102,12 +106,12 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_cast_rows_f32": [P, I, P, I, I, I, I, P],
         "acv_activation": [P, P, LL, I, F, F, I, P],
         "acv_rmsnorm_rows": [P, I, P, F, P, I, I, I, I, P],
-        "acv_latent_prepare": [P, I, P, I, P, I, P, F, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, P],
+        "acv_latent_prepare": [P, I, P, I, P, I, P, F, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, P],
         "acv_attention_latent_tc_takes": [I, I, I],
-        "acv_attention_latent_tc": [P, I, P, I, P, P, P, I, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, P, P, P],
+        "acv_attention_latent_tc": [P, I, P, I, P, P, P, I, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, P, P, P, P],
         "acv_gemm_tc_qkv": [P, I, P, I, P, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, I, I, I, P, P, F, P, I, P, P, P, I, P, P, P, I, I, P],
         "acv_gemm_tc": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P],
-        "acv_gemm_tc_bias": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P, P],
+        "acv_gemm_tc_bias": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P, F, F, P],
         "acv_attention_decode": [P, I, P, I, P, P, P, P, I, P, P, I, P, I, I, I, I, I, F, I, I, I, P, P, P, LL, LL, LL, I, I, I, I, P, P, P],
         "acv_attention_tc": [P, I, I, P, I, P, P, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, I, P, I, P, P, P],
         "acv_attention_chunk": [P, I, P, I, P, P, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, I, I, P],
@@ -462,7 +466,7 @@ def gemm_tc_plan(M: int, N: int, K: int, sms: int | None = None, bn_multiple: in
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: tuple | None = None,
             swiglu_pairs: bool = False, static_weights: bool = False, bias: torch.Tensor | None = None,
-            gate_fn: int = 0, unary: str | None = None) -> torch.Tensor:
+            gate_fn: int = 0, unary: str | None = None, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """out[M,N] = x[M,K] @ w[N,K]^T (+ bias) on tcgen05; x, w bfloat16, out bfloat16 or float32; ``bias`` float32 [N],
     added in the epilogue to the float accumulator (before the activation of the paired form).
 
@@ -471,7 +475,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: tuple | N
 
     With ``swiglu_pairs`` the rows of w come in (gate, up) pairs and out is [M, N/2]:
     out[:, i] = silu(x . w[2i]) * (x . w[2i+1]), rounded as the separate kernels round; with ``gate_fn`` 1 the gate
-    passes through the tanh form of gelu instead (in float on the accumulators, the product rounded once).
+    passes through the tanh form of gelu instead (in float on the accumulators, the product rounded once), with ``gate_fn``
+    2 the pair is the clamped gated unit: g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, +-limit).
     ``unary`` (not with ``swiglu_pairs``): an activation of ``ACTIVATIONS`` (not the first) on every output."""
     _need_cuda(x, w, out)
     if unary is not None and (swiglu_pairs or ACTIVATIONS.get(unary, 0) == 0):
@@ -496,10 +501,10 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: tuple | N
             (1 | (int(gate_fn) << 4)) if swiglu_pairs else ((ACTIVATIONS[unary] << 4) if unary else 0), swap, bn, splits, _p(ws),
             ws.numel(), _p(cnt),
             cnt.numel(), _p(status), sm_count(x.device), stages, cluster | (2 if static_weights else 0))
-    if bias is not None:
-        if bias.dtype != torch.float32 or bias.numel() != N or not bias.is_contiguous():
+    if bias is not None or (swiglu_pairs and gate_fn == 2):
+        if bias is not None and (bias.dtype != torch.float32 or bias.numel() != N or not bias.is_contiguous()):
             raise KernelError("gemm_tc: the bias is a contiguous float32 vector with one entry for each row of the weight")
-        _check(library().acv_gemm_tc_bias(*args, _p(bias), _stream()), "gemm_tc")
+        _check(library().acv_gemm_tc_bias(*args, _p(bias), float(limit), float(alpha), _stream()), "gemm_tc")
     else:
         _check(library().acv_gemm_tc(*args, _stream()), "gemm_tc")
     return out
@@ -1000,11 +1005,13 @@ def linear_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, static_weig
 
 
 def linear_bf16_swiglu(x: torch.Tensor, w_pairs: torch.Tensor, out: torch.Tensor,
-                       static_weights: bool = False, bias: torch.Tensor | None = None, act: int = 1) -> torch.Tensor:
+                       static_weights: bool = False, bias: torch.Tensor | None = None, act: int = 1, limit: float = 0.0,
+                       alpha: float = 0.0) -> torch.Tensor:
     """out[M, I] = silu(x @ Wg^T + bg) * (x @ Wu^T + bu) in one kernel; w_pairs [2I, K] holds (gate_i, up_i) in rows
     2i, 2i+1, and ``bias`` (float32 [2I]) their biases in the same order.  ``act``: a code of ``GATED_EPILOGUE_ACTS``
-    (1: silu; 2: the tanh form of gelu on the gate)."""
-    return gemm_tc(x, w_pairs, out, swiglu_pairs=True, static_weights=static_weights, bias=bias, gate_fn=act - 1)
+    (1: silu; 2: the tanh form of gelu on the gate; 3: the clamped gated unit with ``limit`` and ``alpha``)."""
+    return gemm_tc(x, w_pairs, out, swiglu_pairs=True, static_weights=static_weights, bias=bias, gate_fn=act - 1, limit=limit,
+                   alpha=alpha)
 
 
 def linear_bf16_f32out(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, static_weights: bool = False,
@@ -1521,11 +1528,12 @@ def retention_gate(o: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, num_h
         raise KernelError("retention_gate: the weight is a contiguous float32 vector over all heads' values")
     if gate_fn not in ("silu", "sigmoid"):
         raise KernelError(f"retention_gate: no gate function '{gate_fn}'")
-    if o.dtype != torch.float32 or gate.dtype != out.dtype or gate.stride(1) != 1 or out.stride(1) != 1 or o.stride(1) != 1:
-        raise KernelError("retention_gate: float32 o, and gate and out of one type with dense rows, are wanted")
+    if o.dtype != torch.float32 or gate.dtype not in (out.dtype, torch.float32) or gate.stride(1) != 1 or out.stride(1) != 1 or o.stride(1) != 1:
+        raise KernelError("retention_gate: float32 o, and out and a gate of its type (or float32) with dense rows, are wanted")
     _check(library().acv_retention_gate(_p(o), o.stride(0), _p(gate), gate.stride(0), _p(out), out.stride(0), o.shape[0],
                                         num_heads, value_dim, eps, float(out_scale), dtype_code(out.dtype), _p(weight),
-                                        1 if joint else 0, 1 if gate_fn == "sigmoid" else 0, _stream()), "retention_gate")
+                                        1 if joint else 0, 1 if gate_fn == "sigmoid" else 0, dtype_code(gate.dtype), _stream()),
+           "retention_gate")
     return out
 
 
@@ -1644,7 +1652,7 @@ def cast_rows_f32(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
 
 ACTIVATIONS = {"xielu": 0, "gelu_tanh": 1, "silu": 2, "gelu": 3}
 # gate activations that the tensor-core product applies in its own epilogue: name -> the epilogue's code
-GATED_EPILOGUE_ACTS = {"silu": 1, "gelu_tanh": 2}
+GATED_EPILOGUE_ACTS = {"silu": 1, "gelu_tanh": 2, "swish_clamped": 3}
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str, p0: float = 0.0, p1: float = 0.0) -> torch.Tensor:
@@ -1661,10 +1669,11 @@ def activation(x: torch.Tensor, out: torch.Tensor, kind: str, p0: float = 0.0, p
 
 
 # ----------------------------------------------------------------------------- attention through a kept latent
-def gemm_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+def gemm_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None) -> torch.Tensor:
     """out[:, b, :] = a[:, b, :] @ w[b]^T for every b: a [M, B, K] and out [M, B, N] are views with dense last
     dimension (any row and batch strides), w [B, N, K] contiguous; 32-bit accumulation.  bfloat16 views made of 16-byte
-    pieces run on the tensor cores (csrc/gemm_mma_batched.cu), everything else on the CUDA cores."""
+    pieces run on the tensor cores (csrc/gemm_mma_batched.cu), everything else on the CUDA cores.  ``gate`` (a view of
+    out's shape, of a's type): out is multiplied by sigmoid(gate) in float before it is rounded."""
     _need_cuda(a, w, out)
     M, B, K = a.shape
     N = w.shape[1]
@@ -1672,34 +1681,41 @@ def gemm_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.T
             or a.dtype != w.dtype:
         raise KernelError(f"gemm_batched: shapes {tuple(a.shape)} x {tuple(w.shape)} -> {tuple(out.shape)} do not fit")
     lib = library()
+    if gate is not None and (gate.shape != out.shape or gate.stride(2) != 1 or gate.dtype != a.dtype):
+        raise KernelError("gemm_batched: the gate is a view of the output's shape, of the operands' type, with dense rows")
+    g = (_p(gate), gate.stride(0), gate.stride(1)) if gate is not None else (None, 0, 0)
     if a.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and lib.acv_gemm_mma_batched_takes(
-            _p(a), a.stride(0), a.stride(1), _p(w), K, N * K, _p(out), out.stride(0), out.stride(1), N, K):
+            _p(a), a.stride(0), a.stride(1), _p(w), K, N * K, _p(out), out.stride(0), out.stride(1), N, K) and \
+            (gate is None or (g[1] % 2 == 0 and g[2] % 2 == 0 and gate.data_ptr() % 4 == 0)):
         _check(lib.acv_gemm_mma_batched(_p(a), a.stride(0), a.stride(1), _p(w), K, N * K, _p(out), out.stride(0),
-                                        out.stride(1), M, N, K, B, _stream()), "gemm_mma_batched")
+                                        out.stride(1), M, N, K, B, *g, _stream()), "gemm_mma_batched")
         return out
     _check(library().acv_gemm_simt_batched(_p(a), a.stride(0), a.stride(1), _p(w), K, N * K, _p(out), out.stride(0),
-                                           out.stride(1), M, N, K, B, dtype_code(a.dtype), dtype_code(out.dtype), _stream()),
+                                           out.stride(1), M, N, K, B, dtype_code(a.dtype), dtype_code(out.dtype), *g, _stream()),
            "gemm_batched")
     return out
 
 
-def latent_prepare(q: torch.Tensor, q_out: torch.Tensor, kv: torch.Tensor, weight: torch.Tensor, eps: float,
+def latent_prepare(q: torch.Tensor, q_out: torch.Tensor, kv: torch.Tensor | None, weight: torch.Tensor | None, eps: float,
                    cos_sin: torch.Tensor | None, positions: torch.Tensor, seq_of_token: torch.Tensor,
                    block_table: torch.Tensor | None, pages: torch.Tensor | None, num_heads: int, dim: int, rot_dim: int,
-                   rank: int, table_rows: torch.Tensor | None = None) -> None:
+                   rank: int, table_rows: torch.Tensor | None = None, rotate_half: bool = False) -> None:
     """The kept row of every token, [normed latent | rotated shared key part], into its page, and every head's rotated
     query part into ``q_out[:, h, rank:]`` (csrc/latent_attention.cu).  q: [T, heads*(dim+rot_dim)]; q_out:
-    [T, heads*(rank+rot_dim)]; kv: [T, rank+rot_dim]; pages [num_pages, 1, page_size, rank+rot_dim] or None."""
-    _need_cuda(q, q_out, kv)
-    if q.stride(1) != 1 or q_out.stride(1) != 1 or kv.stride(1) != 1 or q.dtype != kv.dtype or q_out.dtype != q.dtype:
+    [T, heads*(rank+rot_dim)]; kv: [T, rank+rot_dim], or None for a layer that reads rows kept by another one (queries
+    only); pages [num_pages, 1, page_size, rank+rot_dim] or None.  Rotated pairs are (2i, 2i+1), with ``rotate_half``
+    (i, i + rot/2)."""
+    _need_cuda(q, q_out)
+    if q.stride(1) != 1 or q_out.stride(1) != 1 or q_out.dtype != q.dtype or (kv is not None and (kv.stride(1) != 1 or q.dtype != kv.dtype)):
         raise KernelError("latent_prepare: q, q_out and kv have dense rows and one type")
     rot = cos_sin.shape[1] if cos_sin is not None else 0
     _check(library().acv_latent_prepare(
-        _p(q), q.stride(0), _p(q_out), q_out.stride(0), _p(kv), kv.stride(0), _p(weight), float(eps), _p(cos_sin), rot,
+        _p(q), q.stride(0), _p(q_out), q_out.stride(0), _p(kv), kv.stride(0) if kv is not None else 0, _p(weight), float(eps),
+        _p(cos_sin), rot,
         cos_sin.shape[0] if cos_sin is not None else 0, _p(positions), _p(seq_of_token), _p(block_table),
         block_table.stride(0) if block_table is not None else 0, _p(table_rows), _p(pages),
         pages.shape[2] if pages is not None else 1, pages.shape[0] if pages is not None else 0, q.shape[0], num_heads, dim,
-        rot_dim, rank, dtype_code(q.dtype), _stream()), "latent_prepare")
+        rot_dim, rank, dtype_code(q.dtype), 1 if rotate_half else 0, _stream()), "latent_prepare")
 
 
 def attention_latent_tc_takes(dtype: torch.dtype, num_heads: int, row: int, rank: int) -> bool:
@@ -1710,15 +1726,17 @@ def attention_latent_tc_takes(dtype: torch.dtype, num_heads: int, row: int, rank
 
 def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ctx, block_table: torch.Tensor,
                      num_heads: int, row: int, rank: int, scale: float, window: int = 0,
-                     work: dict | None = None) -> torch.Tensor:
+                     work: dict | None = None, sinks: torch.Tensor | None = None) -> torch.Tensor:
     """Attention of every token of the step over its request's kept rows: ``q`` [T, heads*row] are the queries that meet
     the rows of ``pages`` [num_pages, 1, page_size, row]; ``out`` [T, heads*rank] gets the weighted sums of the rows'
-    first ``rank`` elements.  Causal, with ``window`` > 0 limited to the last ``window`` rows.
+    first ``rank`` elements.  Causal, with ``window`` > 0 limited to the last ``window`` rows.  ``sinks`` (float32 [heads]):
+    exp(sink_h) joins the softmax's denominator.
 
     With the step's attention work lists (``work``) bfloat16 runs take the tensor-core kernel (one launch for portions
     and one-token requests; csrc/latent_attention_tc.cu); float32 runs, and sizes that kernel refuses, take the generic
     paged kernel with the pages as keys and as values."""
     _need_cuda(q, out, pages)
+    _head_vectors(num_heads, sinks)
     rows = getattr(ctx, "table_rows", None)
     if work is not None and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and pages.is_contiguous() and \
             attention_latent_tc_takes(q.dtype, num_heads, row, rank):
@@ -1736,10 +1754,10 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ct
             _p(q), q.stride(0), _p(out), out.stride(0), _p(pages), _p(work["tile_seq"]), _p(work["tile_q0"]),
             work["n_tiles"], _p(work["dec_tokens"]), _p(work["dec_seqs"]), work["n_dec"], _p(ctx.cu_q), _p(ctx.kv_len),
             _p(block_table), block_table.stride(0), _p(rows), num_heads, row, rank, pages.shape[2], pages.shape[0],
-            float(scale), int(window), n_split, _p(acc), _p(ml), _stream()), "attention_latent_tc")
+            float(scale), int(window), n_split, _p(acc), _p(ml), _p(sinks), _stream()), "attention_latent_tc")
         return out
     return attention_generic(q, out, pages, pages, ctx.positions, ctx.seq_of_token, block_table, num_heads, 1, row, scale,
-                             window, table_rows=rows, value_dim=rank)
+                             window, table_rows=rows, value_dim=rank, sinks=sinks)
 
 
 def rmsnorm_rows(x: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor) -> torch.Tensor:
@@ -1887,3 +1905,61 @@ def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, u: t
                              _p(seg_idx), seg_len, _p(seg), _p(seg_decay), 1 if summaries else 0, _p(out), out.stride(0),
                              n_items, num_heads, dim, value_dim, dtype_code(r.dtype), _stream()), "wkv")
     return out
+
+
+# ----------------------------------------------------------------------------- a generalized delta rule
+def delta_prepare(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor,
+                  num_heads: int, dim: int) -> None:
+    """What enters the delta recurrence, from a token's row of the input product [r | k | v | z | g | x] (float32 [T, >=
+    5 I + L], I = heads * dim, L rows of ``w2_t`` [L, I]): ``decay`` [T, I] = exp(-exp(-1/2) sigmoid(w0 + tanh(x) w2_t));
+    z in place becomes sigmoid(z) u, u = k / sqrt(sum(k^2) + 1e-6) per head; ``scalars`` [T, heads, 2]: that inverse root,
+    and the product of the next token's k with the new z (csrc/general_delta.cu)."""
+    _need_cuda(proj, w2_t, w0, decay, scalars)
+    T, (L, I) = proj.shape[0], w2_t.shape
+    if any(t.dtype != torch.float32 for t in (proj, w2_t, w0, decay, scalars)) or I != num_heads * dim or proj.stride(1) != 1 \
+            or proj.shape[1] < 5 * I + L or not all(t.is_contiguous() for t in (w2_t, w0, decay, scalars)) \
+            or decay.shape != (T, I) or scalars.shape != (T, num_heads, 2):
+        raise KernelError("delta_prepare: float32 rows [r | k | v | z | g | x], w2_t [L, I], w0 [I], decay [T, I] and scalars [T, heads, 2] are wanted")
+    _check(library().acv_delta_prepare(_p(proj), proj.stride(0), _p(w2_t), _p(w0), _p(decay), _p(scalars), T, num_heads, dim, L,
+                                       _stream()), "delta_prepare")
+
+
+def delta(proj: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+          cu_q: torch.Tensor, num_seqs: int, out: torch.Tensor, num_heads: int, dim: int) -> torch.Tensor:
+    """S = diag(w) S - (a u) (u^T S) + k v^T, o = S^T r along each request's tokens, per head, after ``delta_prepare``;
+    state float32 [slots, heads, dim, dim], out float32 [T, heads * dim].  Heads of up to 512 channels."""
+    _need_cuda(proj, decay, scalars, state, out)
+    if state.dtype != torch.float32 or not state.is_contiguous() or out.dtype != torch.float32 or not out.is_contiguous() \
+            or state.shape[1:] != (num_heads, dim, dim) or out.shape != (proj.shape[0], num_heads * dim):
+        raise KernelError("delta: a float32 state [slots, heads, dim, dim] and output [T, heads * dim] are wanted")
+    _check(library().acv_delta(_p(proj), proj.stride(0), _p(decay), _p(scalars), _p(state), _p(slots), _p(cu_q), _p(out),
+                               num_seqs, num_heads, dim, _stream()), "delta")
+    return out
+
+
+def general_delta(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, weight: torch.Tensor, eps: float,
+                  state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor, num_seqs: int, max_q_len: int,
+                  out: torch.Tensor, num_heads: int, dim: int, rank: int) -> torch.Tensor:
+    """From the input product (``delta_prepare``; z is changed in place) to the gated heads: every head's o of the
+    recurrence to unit RMS (``eps``), times ``weight`` (float32 [heads * dim]), times sigmoid(g), into ``out`` (a view
+    [T, heads * dim] with dense rows).  Steps in which every request brings one token are one launch; others prepare,
+    recurrence and gate."""
+    _need_cuda(proj, w2_t, w0, weight, state, out)
+    T, I = out.shape
+    if weight.dtype != torch.float32 or weight.numel() != I or not weight.is_contiguous() or out.stride(1) != 1:
+        raise KernelError("general_delta: a float32 weight over all heads and an output with dense rows are wanted")
+    lib = library()
+    if max_q_len == 1 and T == num_seqs and lib.acv_delta_step_takes(dim, rank):
+        if proj.dtype != torch.float32 or proj.stride(1) != 1 or state.dtype != torch.float32 or not state.is_contiguous() \
+                or w2_t.shape != (rank, I) or not w2_t.is_contiguous() or state.shape[1:] != (num_heads, dim, dim):
+            raise KernelError("general_delta: float32 projections, w2_t [L, I] and a float32 state are wanted")
+        _check(lib.acv_delta_step(_p(proj), proj.stride(0), _p(w2_t), _p(w0), _p(weight), float(eps), _p(state), _p(slots),
+                                  _p(cu_q), _p(out), out.stride(0), num_seqs, num_heads, dim, rank, dtype_code(out.dtype),
+                                  _stream()), "delta_step")
+        return out
+    decay = torch.empty((T, I), device=proj.device, dtype=torch.float32)
+    scalars = torch.empty((T, num_heads, 2), device=proj.device, dtype=torch.float32)
+    delta_prepare(proj, w2_t, w0, decay, scalars, num_heads, dim)
+    o = torch.empty((T, I), device=proj.device, dtype=torch.float32)
+    delta(proj, decay, scalars, state, slots, cu_q, num_seqs, o, num_heads, dim)
+    return retention_gate(o, proj[:, 4 * I:5 * I], out, num_heads, dim, eps, weight=weight, gate_fn="sigmoid")

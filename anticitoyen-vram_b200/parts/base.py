@@ -117,10 +117,18 @@ class Mixer(Part):
         """Bytes of cache that the step has to read for these requests."""
         return 0
 
+    # A mixer that can stand beside a feed-forward under one output product (the "parallel" block) names the columns in
+    # front of its output projection ``self.o`` (``inner_size``) and fills them itself: ``inner(h, ctx, cache, out)``, out a
+    # view [T, inner_size] with dense rows at any stride.  A mixer that offers ``qkv`` and ``mix`` gets it from those.
+    def inner(self, h: torch.Tensor, ctx, cache: CacheView | None, out: torch.Tensor) -> None:
+        self.mix(self.qkv(h), ctx, cache, out)
+
     def forward(self, h: torch.Tensor, ctx, cache: CacheView | None) -> torch.Tensor:
         raise NotImplementedError
 
 
 class FeedForward(Part):
+    # the same for a feed-forward: ``inner_size`` columns in front of its last product ``self.down``, filled by
+    # ``inner(h, ctx, out)``
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
         raise NotImplementedError

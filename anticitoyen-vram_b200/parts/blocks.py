@@ -8,6 +8,7 @@ from ..cache.manager import StateNeed
 from ..kernels import ops
 from ..weights.needs import TensorNeed
 from .base import CacheView, Runtime
+from .linear import Linear
 from .norms import LayerNorm
 from .plan import LayerSpec
 from .registry import build, register
@@ -187,6 +188,81 @@ class PreNormBlock:
             return x, a
         h = self.post_norm.forward(x, a, **kw, **scale)
         return x, self.feed_forward.forward(h, ctx)
+
+
+@register("block", "parallel")
+class ParallelBlock:
+    """x += mixer(norm(x)) + feed_forward(norm(x)): one norm, both parts read its output and both join the stream
+    together.
+
+    A part's last product is linear, so the two are one product over the parts' inner columns side by side,
+    [mixer's | feed-forward's] @ [W_o | W_down]^T (+ bias): the two outputs are added in its float accumulators, and what
+    joins the float32 stream leaves it unrounded.  Both parts must offer ``inner_size`` and ``inner`` (parts/base.py).
+    A layer without a feed-forward is its mixer alone.  The norm is ``LayerSpec.norm`` under the first of
+    ``norm_prefixes``."""
+
+    residual_mult = 1.0
+
+    def __init__(self, spec: LayerSpec, hidden_size: int) -> None:
+        self.hidden_size = hidden_size
+        self.prefix = spec.prefix
+        self.pre = spec.norm_prefixes[0]
+        self.input_norm = build("norm", spec.norm, hidden_size)
+        self.mixer = build("mixer", spec.mixer, hidden_size)
+        self.feed_forward = build("feed_forward", spec.feed_forward, hidden_size) if spec.feed_forward is not None else None
+        if self.feed_forward is not None:
+            for part in (self.mixer, self.feed_forward):
+                if not hasattr(part, "inner_size") or not hasattr(part, "inner"):
+                    raise ValueError(f"a '{part.kind}' part cannot stand beside another one (it offers no inner columns)")
+        self.run_dtype = None
+        self.out = None
+
+    def tensor_needs(self):
+        needs = {self.pre + name: need for name, need in self.input_norm.tensor_needs().items()}
+        needs.update(self.mixer.tensor_needs())
+        if self.feed_forward is not None:
+            needs.update(self.feed_forward.tensor_needs())
+        return needs
+
+    def load(self, tensors, rt: Runtime) -> None:
+        self.run_dtype = rt.dtype
+        own = self.input_norm.tensor_needs()
+        self.input_norm.load({n: tensors[self.pre + n] for n in own}, rt)
+        self.mixer.load(tensors, rt)
+        if self.feed_forward is None:
+            return
+        self.feed_forward.load(tensors, rt)
+        o, down = self.mixer.o, self.feed_forward.down
+        bias = o.bias if down.bias is None else down.bias if o.bias is None else o.bias + down.bias
+        self.out = Linear(torch.cat([o.weight, down.weight], dim=1), bias)
+        # each part keeps its own last product as columns of the joint weight (no second copy)
+        o.weight, down.weight = self.out.weight[:, :o.in_features], self.out.weight[:, o.in_features:]
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def _parts(self):
+        return [p for p in (self.input_norm, self.mixer, self.feed_forward) if p is not None]
+
+    def weight_bytes(self) -> int:
+        return sum(p.weight_bytes() for p in self._parts())
+
+    def step_weight_bytes(self, num_tokens: int) -> int:
+        return sum(p.step_weight_bytes(num_tokens) if hasattr(p, "step_weight_bytes") else p.weight_bytes() for p in self._parts())
+
+    def flops(self, num_tokens: int) -> float:
+        return self.mixer.flops(num_tokens) + (self.feed_forward.flops(num_tokens) if self.feed_forward is not None else 0.0)
+
+    def forward(self, x, delta, ctx, cache: CacheView | None):
+        kw = {"out_dtype": self.run_dtype} if self.run_dtype is not None and x.dtype != self.run_dtype else {}
+        h = self.input_norm.forward(x, delta, **kw)
+        if self.feed_forward is None:
+            return x, self.mixer.forward(h, ctx, cache)
+        m = self.mixer.inner_size
+        inner = torch.empty((h.shape[0], m + self.feed_forward.inner_size), device=h.device, dtype=h.dtype)
+        self.mixer.inner(h, ctx, cache, inner[:, :m])
+        self.feed_forward.inner(h, ctx, inner[:, m:])
+        return x, self.out(inner, out_dtype=x.dtype)
 
 
 class NormedDelta:

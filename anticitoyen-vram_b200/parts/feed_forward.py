@@ -19,14 +19,19 @@ class SwiGLU(FeedForward):
     (acvram/engine/attention.py:705-783)."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, prefix: str = "mlp.", bias: bool | None = None,
-                 names: dict | None = None, activation: str = "silu") -> None:
+                 names: dict | None = None, activation: str = "silu", limit: float = 0.0, alpha: float = 0.0) -> None:
         """``bias``: True, the three projections have biases; False, none; None, those that the file holds.
         ``names``: the tensors' names behind ``prefix``, {"gate": w, "gate.bias": b, "up": ..., "down": ...}.
         ``activation``: what the gate passes through, "silu" or "gelu_tanh" (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))),
-        computed in float."""
-        if activation not in ("silu", "gelu_tanh"):
-            raise ValueError(f"gated feed-forward: no activation '{activation}' (silu and gelu_tanh are built)")
+        computed in float; or "swish_clamped": with g = min(gate, limit) and u = clamp(up, -limit, limit) the unit is
+        g * sigmoid(alpha g) * (u + 1), in float."""
+        if activation not in ("silu", "gelu_tanh", "swish_clamped"):
+            raise ValueError(f"gated feed-forward: no activation '{activation}' (silu, gelu_tanh and swish_clamped are built)")
+        if activation == "swish_clamped" and not limit > 0.0:
+            raise ValueError("gated feed-forward: swish_clamped wants a positive limit")
         self.activation = activation
+        self.limit, self.alpha = float(limit), float(alpha)
+        self.inner_size = intermediate_size
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
         self.prefix = prefix
         self.bias = bias
@@ -83,21 +88,29 @@ class SwiGLU(FeedForward):
             return None
         return {"intermediate_size": self.intermediate_size, "w_gate_up_pairs": self.gate_up.weight, "w_down": self.down.weight}
 
-    def forward(self, h, ctx):
+    def inner(self, h, ctx, out) -> None:
+        """The unit's output in front of the down product into ``out`` [T, inner_size] (dense rows at any stride)."""
         if self.fused and self.fused_act is not None and h.shape[0] and ops.gemm_tc_takes(h, self.gate_up.weight):
-            act = torch.empty((h.shape[0], self.intermediate_size), device=h.device, dtype=h.dtype)
-            ops.linear_bf16_swiglu(h, self.gate_up.weight, act, static_weights=True, bias=self.gate_up.bias,
-                                   **({"act": self.fused_act} if self.activation != "silu" else {}))
-            return self.down(act)
-        act = torch.empty((h.shape[0], self.intermediate_size), device=h.device, dtype=h.dtype)
-        if self.activation != "silu":
-            # the gate's activation in float on the stacked product's output, rounded once
-            return self.down(ops.glu(self.gate_up(h), act, ops.ACTIVATIONS[self.activation], 0.0, 0.0, pairs=self.fused))
-        if self.fused:      # an input the tensor-core kernel does not take: undo the interleaving for this call
-            gu = self.gate_up(h).view(h.shape[0], self.intermediate_size, 2).transpose(1, 2).reshape(h.shape[0], -1)
+            ops.linear_bf16_swiglu(h, self.gate_up.weight, out, static_weights=True, bias=self.gate_up.bias,
+                                   **({"act": self.fused_act} if self.activation != "silu" else {}),
+                                   **({"limit": self.limit, "alpha": self.alpha} if self.activation == "swish_clamped" else {}))
+        elif self.activation != "silu":
+            # the unit in float on the stacked product's output, rounded once
+            kind = ops.GLU_SWISH_CLAMPED if self.activation == "swish_clamped" else ops.ACTIVATIONS[self.activation]
+            ops.glu(self.gate_up(h), out, kind, self.limit, self.alpha, pairs=self.fused)
         else:
-            gu = self.gate_up(h)
-        ops.swiglu(gu, act)
+            if self.fused:      # an input the tensor-core kernel does not take: undo the interleaving for this call
+                gu = self.gate_up(h).view(h.shape[0], self.intermediate_size, 2).transpose(1, 2).reshape(h.shape[0], -1)
+            else:
+                gu = self.gate_up(h)
+            if out.is_contiguous():
+                ops.swiglu(gu, out)
+            else:
+                ops.glu(gu, out, ops.ACTIVATIONS["silu"], 0.0, 0.0)
+
+    def forward(self, h, ctx):
+        act = torch.empty((h.shape[0], self.intermediate_size), device=h.device, dtype=h.dtype)
+        self.inner(h, ctx, act)
         return self.down(act)
 
 

@@ -554,7 +554,14 @@ class LatentAttention(Mixer):
         key_h = [W_uk,h c | r],     value_h = W_uv,h c,   score = scale <q_h, key_h> with q_rot rotated as r is
 
     under a causal mask, with ``window`` > 0 limited to the last ``window`` keys; softmax; W_o over the heads.  rot
-    turns interleaved pairs (2i, 2i+1) of the first ``position.dim`` elements by position * theta^(-2i/dim).
+    turns interleaved pairs (2i, 2i+1) of the first ``position.dim`` elements by position * theta^(-2i/dim); with
+    ``rotate_half`` the pairs are (i, i + dim/2).  A scaled position encoding's factor on cos and sin acts on q_rot and r
+    alike; ``scale`` is used as it is given.
+
+    ``sink``: the name of one learned number per head: exp(sink_h) joins the softmax's denominator.  ``gate``: the name
+    of a matrix W_g over the heads' values: the heads side by side are multiplied by sigmoid(W_g h) in front of W_o.
+    ``own_kv`` False: the layer has no W_dkv and reads the rows [c | r] of the cache slot that another layer writes (the
+    plan's schedule says which; the sizes of a row and the rotation are the same), through its own W_uk and W_uv.
 
     Per token the layer keeps [c | r] and nothing else: one key/value head of rank + rot_dim elements whose values are
     the first ``rank`` elements of the same rows.  The products with W_uk and W_uv are made on the query's side
@@ -574,8 +581,11 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, dim: int, rot_dim: int, value_dim: int, q_rank: int, kv_rank: int,
                  scale: float | None, norm_eps: float, position: PartSpec, window: int = 0, prefix: str = "mix.",
-                 names: dict | None = None) -> None:
+                 names: dict | None = None, rotate_half: bool = False, sink: str | None = None, gate: str | None = None,
+                 own_kv: bool = True) -> None:
         self.hidden_size = hidden_size
+        self.rotate_half, self.sink, self.gate, self.own_kv = bool(rotate_half), sink, gate, bool(own_kv)
+        self.sinks = self.kv_norm = None
         self.num_heads, self.dim, self.rot_dim, self.value_dim = num_heads, dim, rot_dim, value_dim
         self.q_rank, self.kv_rank = q_rank, kv_rank
         self.scale = float(scale) if scale is not None else (dim + rot_dim) ** -0.5
@@ -585,6 +595,7 @@ class LatentAttention(Mixer):
         self.names = {**self.NAMES, **(names or {})}
         self.position = build("position", position, hidden_size)
         self.row = kv_rank + rot_dim            # elements of a kept row, and of a query that meets it
+        self.inner_size = num_heads * value_dim # columns in front of the output projection
 
     def _n(self, role: str) -> str:
         return self.prefix + self.names[role]
@@ -594,20 +605,40 @@ class LatentAttention(Mixer):
 
     def tensor_needs(self):
         W, H, D, R, DV = self.hidden_size, self.num_heads, self.dim, self.rot_dim, self.value_dim
-        return {self._n("dq"): TensorNeed((self.q_rank, W)), self._n("dq.norm"): TensorNeed((self.q_rank,), "norm"),
-                self._n("uq"): TensorNeed((H * (D + R), self.q_rank)), self._n("dkv"): TensorNeed((self.row, W)),
-                self._n("dkv.norm"): TensorNeed((self.kv_rank,), "norm"), self._n("uk"): TensorNeed((H * D, self.kv_rank)),
-                self._n("uv"): TensorNeed((H * DV, self.kv_rank)), self._n("o"): TensorNeed((W, H * DV))}
+        needs = {self._n("dq"): TensorNeed((self.q_rank, W)), self._n("dq.norm"): TensorNeed((self.q_rank,), "norm"),
+                 self._n("uq"): TensorNeed((H * (D + R), self.q_rank)), self._n("uk"): TensorNeed((H * D, self.kv_rank)),
+                 self._n("uv"): TensorNeed((H * DV, self.kv_rank)), self._n("o"): TensorNeed((W, H * DV))}
+        if self.own_kv:
+            needs[self._n("dkv")] = TensorNeed((self.row, W))
+            needs[self._n("dkv.norm")] = TensorNeed((self.kv_rank,), "norm")
+        if self.sink is not None:
+            needs[self.prefix + self.sink] = TensorNeed((H,), "norm")
+        if self.gate is not None:
+            needs[self.prefix + self.gate] = TensorNeed((H * DV, W))
+        return needs
 
     def load(self, tensors, rt: Runtime) -> None:
         w = lambda role: tensors[self._n(role)].to(device=rt.device, dtype=rt.dtype)
         f = lambda role: tensors[self._n(role)].to(device=rt.device, dtype=torch.float32).contiguous()
         H, D, DV, KR = self.num_heads, self.dim, self.value_dim, self.kv_rank
-        # both down projections read the same input: one stacked product, [c_q' | c' | r']
-        self.down = Linear.stacked([w("dq"), w("dkv")])
+        # everything that reads the mixer's input is one stacked product, [c_q' | gate | c' | r'] (a part that the layer does
+        # not have is left out; zero rows behind it make the product's rows 16-byte pieces)
+        parts = [w("dq")]
+        if self.gate is not None:
+            parts.append(tensors[self.prefix + self.gate].to(device=rt.device, dtype=rt.dtype))
+        if self.own_kv:
+            parts.append(w("dkv"))
+        pad = -sum(p.shape[0] for p in parts) % 8
+        if pad:
+            parts.append(torch.zeros((pad, self.hidden_size), device=rt.device, dtype=rt.dtype))
+        self.down = Linear.stacked(parts)
         self.uq = Linear(w("uq"))
         self.o = Linear(w("o"))
-        self.q_norm, self.kv_norm = f("dq.norm"), f("dkv.norm")
+        self.q_norm = f("dq.norm")
+        if self.own_kv:
+            self.kv_norm = f("dkv.norm")
+        if self.sink is not None:
+            self.sinks = tensors[self.prefix + self.sink].to(device=rt.device, dtype=torch.float32).contiguous()
         # per head: W_uk,h^T as the weight [rank, dim] of q_plain -> latent space; W_uv,h [value_dim, rank] as it is
         self.uk_t = w("uk").view(H, D, KR).transpose(1, 2).contiguous()
         self.uv = w("uv").view(H, DV, KR).contiguous()
@@ -619,7 +650,8 @@ class LatentAttention(Mixer):
 
     # ---- cost of a step
     def weight_bytes(self) -> int:
-        own = sum(t.numel() * t.element_size() for t in (self.uk_t, self.uv, self.q_norm, self.kv_norm))
+        own = sum(t.numel() * t.element_size() for t in (self.uk_t, self.uv, self.q_norm, self.kv_norm, self.sinks)
+                  if t is not None)
         return self.down.weight_bytes() + self.uq.weight_bytes() + self.o.weight_bytes() + own
 
     def flops(self, num_tokens: int) -> float:
@@ -639,22 +671,31 @@ class LatentAttention(Mixer):
         keys = sum(min(kv, self.window + q - 1) if self.window > 0 else kv for q, kv in zip(q_lens, kv_lens))
         return keys * self.row * itemsize
 
-    def forward(self, h, ctx, cache: CacheView):
+    def inner(self, h, ctx, cache: CacheView, out) -> None:
         H, D, R, DV, KR = self.num_heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank
         T = h.shape[0]
+        if cache.writes != self.own_kv:
+            raise ValueError("a latent_attention layer writes its cache slot exactly when it makes its own kept rows")
         table = ctx.block_tables[cache.group]
-        down = self.down(h)                                     # [T, q_rank + rank + rot_dim]
+        down = self.down(h)                                     # [T, q_rank (+ gate) (+ rank + rot_dim)]
+        gate_at = self.q_rank
+        kv_at = gate_at + (self.inner_size if self.gate is not None else 0)
         cq = torch.empty((T, self.q_rank), device=h.device, dtype=h.dtype)
         ops.rmsnorm_rows(down[:, :self.q_rank], self.q_norm, self.norm_eps, cq)
         q = self.uq(cq)                                         # [T, H, dim + rot_dim]
         met = torch.empty((T, H * self.row), device=h.device, dtype=h.dtype)      # the queries that meet the kept rows
-        ops.latent_prepare(q, met, down[:, self.q_rank:], self.kv_norm, self.norm_eps, self.position.rotary_table(),
-                           ctx.positions, ctx.seq_of_token, table if cache.writes else None,
-                           cache.k_pages if cache.writes else None, H, D, R, KR, table_rows=ctx.table_rows)
+        ops.latent_prepare(q, met, down[:, kv_at:kv_at + self.row] if self.own_kv else None, self.kv_norm, self.norm_eps,
+                           self.position.rotary_table(), ctx.positions, ctx.seq_of_token, table if self.own_kv else None,
+                           cache.k_pages if self.own_kv else None, H, D, R, KR, table_rows=ctx.table_rows,
+                           rotate_half=self.rotate_half)
         ops.gemm_batched(q.view(T, H, D + R)[:, :, :D], self.uk_t, met.view(T, H, self.row)[:, :, :KR])
         lat = torch.empty((T, H * KR), device=h.device, dtype=h.dtype)            # weighted sums of latents
         ops.attention_latent(met, lat, cache.k_pages, ctx, table, H, self.row, KR, self.scale, self.window,
-                             work=ctx.work.get(self.metadata_key))
-        out = torch.empty((T, H * DV), device=h.device, dtype=h.dtype)
-        ops.gemm_batched(lat.view(T, H, KR), self.uv, out.view(T, H, DV))
+                             work=ctx.work.get(self.metadata_key), sinks=self.sinks)
+        gate = down[:, gate_at:gate_at + self.inner_size].unflatten(1, (H, DV)) if self.gate is not None else None
+        ops.gemm_batched(lat.view(T, H, KR), self.uv, out.unflatten(1, (H, DV)), gate=gate)
+
+    def forward(self, h, ctx, cache: CacheView):
+        out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
+        self.inner(h, ctx, cache, out)
         return self.o(out)

@@ -16,23 +16,30 @@ class RMSNorm(Norm):
     (acvram/engine/layers.py:607-630); with ``delta`` the sum x + delta is made first,
     in 32-bit, and written back (acvram/engine/layers.py:633-651)."""
 
-    def __init__(self, hidden_size: int, eps: float, size: int | None = None, tensor: str = "weight", groups: int = 1) -> None:
+    def __init__(self, hidden_size: int, eps: float, size: int | None = None, tensor: str = "weight", groups: int = 1,
+                 offset: float = 0.0) -> None:
         """``tensor``: the weight's name behind the norm's prefix ("" where the prefix is the whole name).
         ``groups`` > 1: the row is split into that many equal consecutive parts and each is divided by its own root mean
-        square (the weight still spans the whole row); such a norm wants a float32 residual stream."""
+        square (the weight still spans the whole row); such a norm wants a float32 residual stream.
+        ``offset``: the row is multiplied by offset + w (a weight stored around zero); the sum is made once, in 32-bit, when
+        the weight is loaded."""
         self.size = size or hidden_size
         self.groups = int(groups)
         if self.groups < 1 or self.size % self.groups:
             raise ValueError(f"a norm over {self.size} elements does not split into {groups} equal groups")
         self.eps = float(eps)
         self.tensor = tensor
+        self.offset = float(offset)
         self.weight: torch.Tensor | None = None
 
     def tensor_needs(self):
-        return {self.tensor: TensorNeed((self.size,), "norm")}
+        # (a random weight lies where the file's would: around one, or around zero)
+        return {self.tensor: TensorNeed((self.size,), "norm" if self.offset == 0.0 else "bias")}
 
     def load(self, tensors, rt: Runtime) -> None:
         self.weight = tensors[self.tensor].to(device=rt.device, dtype=torch.float32).contiguous()
+        if self.offset != 0.0:
+            self.weight = self.weight + self.offset
 
     def decode_layer_spec(self):
         """What the fused decode-layer kernel needs of this norm."""

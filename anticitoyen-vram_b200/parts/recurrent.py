@@ -326,3 +326,90 @@ class TimeMix(SegmentedRecurrence):
         out = torch.empty((T, I), device=h.device, dtype=h.dtype)
         ops.retention_gate(o, gate, out, H, D, self.norm_eps, weight=self.norm_weight)
         return self.o(out)
+
+
+@register("mixer", "general_delta")
+class GeneralDelta(Mixer):
+    """A linear recurrence with a generalized delta rule, per head a state S [dim, dim] (key channel by value channel):
+
+        r, k, v = W_r h, W_k h, W_v h   (heads x dim),     u = k / sqrt(sum(k^2) + 1e-6) per head
+        w = exp(-exp(-1/2) sigmoid(W_2 tanh(W_1 h) + w_0))      decay of every head and key channel
+        a = sigmoid(W_a h + b_a)                                 removal rate of every head and key channel
+        S_t = diag(w_t) S_{t-1} - (a_t u_t) (u_t^T S_{t-1}) + k_t v_t^T,     o_t = S_t^T r_t       (S_{-1} = 0)
+
+    (both terms read the old state).  Each head's o is brought to unit RMS (``norm_eps``), the heads side by side are
+    multiplied by a weight and by sigmoid(W_g h), and projected by W_o.  A request keeps S, float32.  32-bit in every run
+    precision: all of the above behind the projections, which leave their product as float.
+    Tensors behind ``prefix`` (``names`` renames them): r, k, v, a, a.b, g, w1, w2, w0, norm, o; the rows of w1 are
+    whatever the file holds."""
+
+    NAMES = {n: n for n in ("r", "k", "v", "a", "a.b", "g", "w1", "w2", "w0", "norm", "o")}
+
+    def __init__(self, hidden_size: int, num_heads: int, dim: int, norm_eps: float, prefix: str = "mix.",
+                 names: dict | None = None) -> None:
+        self.hidden_size, self.num_heads, self.dim = hidden_size, int(num_heads), int(dim)
+        self.norm_eps = float(norm_eps)
+        self.prefix = prefix
+        self.names = {**self.NAMES, **(names or {})}
+        self.inner_size = self.num_heads * self.dim
+        self.rank = None        # rows of W_1: whatever the file holds
+
+    def _n(self, role: str) -> str:
+        return self.prefix + self.names[role]
+
+    def cache_need(self):
+        return StateNeed((self.num_heads, self.dim, self.dim), "float32")
+
+    def tensor_needs(self):
+        H, I = self.hidden_size, self.inner_size
+        needs = {self._n(role): TensorNeed((I, H)) for role in ("r", "k", "v", "a", "g")}
+        needs[self._n("a.b")] = TensorNeed((I,), "bias")
+        needs[self._n("w1")] = TensorNeed((-1, H))          # the decay's inner size is the file's to choose
+        needs[self._n("w2")] = TensorNeed((I, -1))
+        needs[self._n("w0")] = TensorNeed((I,), "norm")
+        needs[self._n("norm")] = TensorNeed((I,), "norm")
+        needs[self._n("o")] = TensorNeed((H, I))
+        return needs
+
+    def load(self, tensors, rt: Runtime) -> None:
+        w = lambda role: tensors[self._n(role)].to(device=rt.device, dtype=rt.dtype)
+        f = lambda role: tensors[self._n(role)].to(device=rt.device, dtype=torch.float32).contiguous()
+        self.rank = tensors[self._n("w1")].shape[0]
+        if tuple(tensors[self._n("w2")].shape) != (self.inner_size, self.rank):
+            raise ValueError(f"general_delta: w2 is {tuple(tensors[self._n('w2')].shape)}, w1 has {self.rank} rows")
+        # everything that reads the mixer's input is one product, [r | k | v | a + b_a | g | w1] (and zero rows that make
+        # its output's rows 16-byte pieces); it leaves as float
+        rows = [w(role) for role in ("r", "k", "v", "a", "g", "w1")]
+        pad = -sum(t.shape[0] for t in rows) % 8
+        if pad:
+            rows.append(torch.zeros((pad, self.hidden_size), device=rt.device, dtype=rt.dtype))
+        biases = [None] * len(rows)
+        biases[3] = f("a.b")
+        self.qkv = Linear.stacked(rows, biases)
+        self.w2_t = f("w2").t().contiguous()        # [rank, I]: the threads of a warp read neighbouring channels
+        self.w0, self.norm_weight = f("w0"), f("norm")
+        self.o = Linear(w("o"))
+
+    def weight_bytes(self) -> int:
+        return self.qkv.weight_bytes() + self.o.weight_bytes() + \
+            sum(t.numel() * 4 for t in (self.w2_t, self.w0, self.norm_weight))
+
+    def flops(self, num_tokens: int) -> float:
+        return self.qkv.flops(num_tokens) + self.o.flops(num_tokens) + 2.0 * num_tokens * self.rank * self.inner_size
+
+    def mixing_flops(self, q_lens, kv_lens) -> float:
+        # per token, head and state element: the products with u and r, the decay, the removal and the update
+        return 9.0 * self.num_heads * self.dim * self.dim * sum(q_lens)
+
+    def cache_bytes_read(self, q_lens, kv_lens, itemsize: int) -> int:
+        return len(q_lens) * self.num_heads * self.dim * self.dim * 4
+
+    def inner(self, h, ctx, cache: CacheView, out) -> None:
+        proj = self.qkv(h, out_dtype=torch.float32)
+        ops.general_delta(proj, self.w2_t, self.w0, self.norm_weight, self.norm_eps, cache.state, ctx.state_slots[cache.group],
+                          ctx.cu_q, ctx.num_seqs, ctx.max_q_len, out, self.num_heads, self.dim, self.rank)
+
+    def forward(self, h, ctx, cache: CacheView):
+        out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
+        self.inner(h, ctx, cache, out)
+        return self.o(out)
