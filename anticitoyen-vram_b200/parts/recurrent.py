@@ -305,7 +305,7 @@ class TimeMix(SegmentedRecurrence):
     def cache_bytes_read(self, q_lens, kv_lens, itemsize: int) -> int:
         return len(q_lens) * (self.num_heads * self.dim * self.dim + self.hidden_size) * 4
 
-    def forward(self, h, ctx, cache: CacheView):
+    def inner(self, h, ctx, cache: CacheView, out) -> None:
         T = h.shape[0]
         H, D, I = self.num_heads, self.dim, self.inner_size
         state, previous = cache.parts["state"], cache.parts["previous"]
@@ -323,8 +323,11 @@ class TimeMix(SegmentedRecurrence):
         o = torch.empty((T, I), device=h.device, dtype=torch.float32)
         ops.wkv(r, k, v, decay, self.u, state.state, ctx.state_slots[state.group], ctx.cu_q, ctx.num_seqs, o, H, D, D,
                 work=ctx.work.get(self.metadata_key))
-        out = torch.empty((T, I), device=h.device, dtype=h.dtype)
         ops.retention_gate(o, gate, out, H, D, self.norm_eps, weight=self.norm_weight)
+
+    def forward(self, h, ctx, cache: CacheView):
+        out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
+        self.inner(h, ctx, cache, out)
         return self.o(out)
 
 

@@ -294,6 +294,32 @@ def retention_case(q_len: int, batch: int, reps: int, H: int = 16, D: int = 64, 
             "gbs": nbytes / us / 1e3}
 
 
+def delta_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, rank: int = 32) -> dict:
+    """The delta recurrence behind its input product: prepare, recurrence and gate of ``batch`` portions of ``q_len`` tokens,
+    or the one launch of steps of single tokens."""
+    T, I = q_len * batch, H * D
+    dev = "cuda:0"
+    proj = torch.randn(T, 5 * I + rank, device=dev)
+    w2_t, w0 = torch.randn(rank, I, device=dev) * 0.3, torch.randn(I, device=dev) - 1.0
+    weight = torch.ones(I, device=dev)
+    state = torch.zeros(batch, H, D, D, device=dev)
+    slots = torch.arange(batch, dtype=torch.int32, device=dev)
+    cu = torch.arange(0, T + 1, q_len, dtype=torch.int32, device=dev)
+    out = torch.empty(T, I, device=dev, dtype=torch.bfloat16)
+    decay, scalars, o = torch.empty(T, I, device=dev), torch.empty(T, H, 2, device=dev), torch.empty(T, I, device=dev)
+    us_all = _time(lambda i: ops.general_delta(proj, w2_t, w0, weight, 1e-6, state, slots, cu, batch, q_len, out, H, D, rank), reps)
+    us_prep = _time(lambda i: ops.delta_prepare(proj, w2_t, w0, decay, scalars, H, D), reps)
+    proj[:, 3 * I:4 * I] *= 0.1
+    us = _time(lambda i: ops.delta(proj, decay, scalars, state, slots, cu, batch, o, H, D), reps)
+    us_gate = _time(lambda i: ops.retention_gate(o, proj[:, 4 * I:5 * I], out, H, D, 1e-6, weight=weight, gate_fn="sigmoid"), reps)
+    flops = 10.0 * H * D * D * T        # five multiply-adds a state element and token
+    print(f"delta q_len={q_len} batch={batch} heads={H} of {D}x{D}: all {us_all:.1f} us, recurrence {us:.1f} us ({flops / us / 1e6:.2f} "
+          f"TFLOP/s float, state {2 * batch * H * D * D * 4 / us / 1e3:.0f} GB/s), prepare {us_prep:.1f} us, gate {us_gate:.1f} us; "
+          f"all: state {2 * batch * H * D * D * 4 / us_all / 1e3:.0f} GB/s")
+    return {"kernel": "delta", "q_len": q_len, "batch": batch, "us": us, "us_all": us_all, "us_prepare": us_prep, "us_gate": us_gate,
+            "tflops_f32": flops / us / 1e6}
+
+
 def wkv_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, C: int = 2048, rank: int = 32) -> dict:
     """Time mixing's own kernels for ``batch`` requests that bring ``q_len`` tokens each: the five mixes of the token
     shift, the decays, and the recurrence of 32 heads of 64 x 64 with decays of the token's own."""
@@ -460,6 +486,11 @@ CASES = {
     "latent_attention_decode_b64": lambda r: latent_attention_case(1, 64, 2048, r),
     "retention_prefill": lambda r: retention_case(2048, 1, r),
     "retention_decode_b64": lambda r: retention_case(1, 64, r),
+    "delta_prefill": lambda r: delta_case(2048, 1, r),
+    "delta_prefill_small": lambda r: delta_case(512, 1, r),
+    "delta_prefill_b8": lambda r: delta_case(512, 8, r),
+    "delta_prefill_128": lambda r: delta_case(2048, 1, r, H=16, D=128),
+    "delta_decode_b64": lambda r: delta_case(1, 64, r),
     "wkv_prefill": lambda r: wkv_case(2048, 1, r),
     "wkv_prefill_small": lambda r: wkv_case(512, 1, r),
     "wkv_decode_b64": lambda r: wkv_case(1, 64, r),

@@ -334,6 +334,103 @@ VADELIX_SIZES = {
 }
 
 
+LODALIX_SIZES = {
+    # width; latent attention (both kinds): heads, unrotated and rotated key size, value size, ranks of the query and key/value
+    # latents; recurrence: heads, head size; gated feed-forward size
+    "s": dict(width=2048, heads=16, dim=64, rot=64, vdim=128, q_rank=768, kv_rank=512, t_heads=32, t_dim=64, ff=6144),
+    "m": dict(width=4096, heads=32, dim=64, rot=64, vdim=128, q_rank=1536, kv_rank=512, t_heads=64, t_dim=64, ff=12288),
+}
+
+
+def run_lodalix(args) -> int:
+    """``--design lodalix``: prefill and decode throughput of the Lodalix design at layer sizes of real models (random
+    weights; six layers: gated latent attention, latent attention with sinks, delta recurrence, gated latent attention on the
+    first layer's rows, latent attention, recurrence), beside the closest models of the framework at equal size: a Nizedra
+    model with latent attention of the same sizes and no window, and its other recurrence, in the same order of layers; and
+    a Vadelix model's time mixing and gated unit.  Whole steps through the step function, and the mixer and feed-forward
+    of each kind of layer alone with their rooflines (L2 flushed before each timed run).  One JSON line."""
+    import torch
+
+    from acvram_b200 import bench as B
+    from acvram_b200.config import LodalixConfig, NizedraConfig, VadelixConfig
+    from acvram_b200.engine.runner import ModelRunner
+    from acvram_b200.models import build_random
+
+    pk, pk_src = peaks()
+    K, W = args.steps, args.warmup
+    page = 64
+    layers, vocab = args.layers or 6, 32768
+    out = {"design": "lodalix", "beside": ["nizedra", "vadelix"], "layers": layers, "vocab": vocab, "dtype": "bf16",
+           "page_size": page, "data": "synthetic token ids, random weights", "peaks": {**pk, "source": pk_src}, "sizes": {}}
+    for name in args.sizes.split(","):
+        z = LODALIX_SIZES[name]
+        rows = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot"], "vdim": z["vdim"], "q_rank": z["q_rank"],
+                "kv_rank": z["kv_rank"], "scale": (z["dim"] + z["rot"]) ** -0.5, "rot": {"base": 1e6, "dims": z["rot"]}}
+        gated = {**rows, "rot": {**rows["rot"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        head = {"heads": z["t_heads"], "dim": z["t_dim"]}
+        order = (("latent_attention_2", gated), ("latent_attention", rows), ("general_delta", head),
+                 ("latent_attention_2", {**gated, "kv_from": 0}), ("latent_attention", rows), ("general_delta", head))
+        unit = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+        lcfg = LodalixConfig.from_dict({"architecture": "Lodalix", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6},
+                                        "layers": [{"type": order[i % 6][0], "mixer": order[i % 6][1], "mlp": unit} for i in range(layers)]})
+        light = {"heads": z["heads"], "dim": z["vdim"], "vdim": z["vdim"], "decay": [1.0 - 2.0 ** (-4 - i % 8) for i in range(z["heads"])]}
+        ncfg = NizedraConfig.from_dict({
+            "architecture": "Nizedra", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [{"type": "lightning", "mixer": light, "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2}} if i % 3 == 2 else
+                       {"type": "latent_attention", "mixer": rows, "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2}} for i in range(layers)]})
+        vcfg = VadelixConfig.from_dict({
+            "architecture": "Vadelix", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6, "groups": 1}, "residual_mult": 1.0,
+            "canon": {"taps": 1}, "layers": [{"type": "wkv", "mixer": head, "mlp": {"kind": "dense", "ff": z["ff"]}}]})
+        kinds_of = {"lodalix": (("gated_latent", 0), ("sink_latent", 1), ("delta", 2), ("borrowed_latent", 3)),
+                    "nizedra": (("latent", 0), ("lightning", 2)), "vadelix": (("wkv", 0),)}
+        res = {"sizes": dict(z)}
+        for arm, cfg in (("lodalix", lcfg), ("nizedra", ncfg), ("vadelix", vcfg)):
+            model = build_random(cfg, seed=0, dtype=torch.bfloat16, device="cuda:0")
+            batch_max = 64
+            tokens = batch_max * (args.context + 2 * (K + W) + 2 * page) + 4096
+            runner = ModelRunner(model, page, tokens // page + 8, batch_max + 2, max_len=8192)
+            if not args.no_cuda_graphs:
+                runner.enable_graphs()
+            r = {"weights_gb": round(model.weight_bytes() / 1e9, 3)}
+            try:
+                if arm != "vadelix":
+                    pre = B.time_prefill(runner, 2048, reps=5, warmup=3)
+                    flops = B.prefill_flops(model, 2048)
+                    r["prefill_2048"] = {"tokens_per_s": round(pre["tokens_per_s"], 1), "ms": round(pre["ms"], 3),
+                                         "tflops_frac": round(flops / (pre["ms"] * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)}
+                    for b in (8, 64):
+                        names = [f"d{b}-{i}" for i in range(b)]
+                        B.fill_contexts(runner, names, args.context)
+                        try:
+                            d = B.time_decode(runner, names, K, W)
+                        finally:
+                            for n in names:
+                                runner.release(n)
+                        nbytes = B.decode_step_bytes(model, b, args.context + W + K // 2)
+                        r[f"decode_b{b}"] = {"tokens_per_s": round(d["tokens_per_s"], 1), "ms_per_step": round(d["ms_per_step"], 4),
+                                             "hbm_frac": round(nbytes / (d["ms_per_step"] * 1e-3) / 1e9 / pk["hbm_gbs"], 4)}
+                for kind, layer in kinds_of[arm]:
+                    if layer >= layers:
+                        continue
+                    for label, ql, kl in (("prefill_2048", [2048], [2048]), ("decode_b64", [1] * 64, [args.context] * 64)):
+                        for part, v in B.time_parts(runner, ql, kl, layer=layer).items():
+                            if part == "feed_forward" and layer:
+                                continue        # (the same in every layer)
+                            sec = v["ms"] * 1e-3
+                            r[f"{kind if part == 'mixer' else 'feed_forward'}_{label}"] = {
+                                "us": round(v["ms"] * 1e3, 1),
+                                "tflops_frac": round(v["flops"] / sec / (pk["bf16_tflops"] * 1e12), 4),
+                                "hbm_frac": round(v["bytes"] / sec / 1e9 / pk["hbm_gbs"], 4)}
+            except B.Refused as exc:
+                r["refused"] = str(exc)
+            res[arm + "_result"] = r
+            del runner, model
+            _free_device_memory()
+        out["sizes"][name] = res
+    print(json.dumps(out))
+    return 0
+
+
 def run_vadelix(args) -> int:
     """``--design vadelix``: prefill and decode throughput of the Vadelix design at layer sizes of real models (random
     weights; six layers: time mixing, rotated attention with sinks, windowed attention with slopes, twice, gated
@@ -694,7 +791,7 @@ def main() -> int:
     ap.add_argument("--page-size", type=int, default=16, help="tokens in a page of the cache (the engine's own default is 64)")
     ap.add_argument("--skip-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--no-cuda-graphs", action="store_true")
-    ap.add_argument("--design", default="", choices=["", "zotonex", "redudra", "nizedra", "vadelix"],
+    ap.add_argument("--design", default="", choices=["", "zotonex", "redudra", "nizedra", "vadelix", "lodalix"],
                     help="measure another design beside its closest relative instead of the headline (see run_design)")
     ap.add_argument("--sizes", default="s,m", help="with --design: which of its sizes (s: width 2048, m: width 4096)")
     ap.add_argument("--time-limit", type=float, default=240.0,
@@ -713,6 +810,8 @@ def main() -> int:
         return run_nizedra(args)
     if args.design == "vadelix":
         return run_vadelix(args)
+    if args.design == "lodalix":
+        return run_lodalix(args)
     if args.design:
         return run_design(args)
     return run_ours(args)
