@@ -129,6 +129,31 @@ __device__ __forceinline__ void gt_add_bias(const GemmParams& p, int row_a, int 
     }
 }
 
+// The same in two steps for tokens on rows, so that the loads are in flight while the accumulators are read: the bias of
+// the columns col0 .. col0 + 15 (16-byte loads, the same for every lane), then the sum.
+__device__ __forceinline__ void gt_load_bias(const GemmParams& p, int col0, float (&b)[16]) {
+    if (!p.bias || p.swap) return;
+    if (col0 + 16 <= p.N && !((uintptr_t)p.bias & 15)) {
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            const float4 x = __ldg(reinterpret_cast<const float4*>(p.bias + col0) + q);
+            b[4 * q] = x.x; b[4 * q + 1] = x.y; b[4 * q + 2] = x.z; b[4 * q + 3] = x.w;
+        }
+    } else {
+#pragma unroll
+        for (int c = 0; c < 16; ++c) b[c] = col0 + c < p.N ? p.bias[col0 + c] : 0.f;
+    }
+}
+__device__ __forceinline__ void gt_sum_bias(const GemmParams& p, int row_a, int col0, const float (&b)[16], float (&v)[16]) {
+    if (!p.bias) return;
+    if (p.swap) {
+        gt_add_bias(p, row_a, col0, v);
+        return;
+    }
+#pragma unroll
+    for (int c = 0; c < 16; ++c) v[c] += b[c];
+}
+
 __device__ __forceinline__ void gt_store16_rows(const GemmParams& p, int row_a, int col0, const float (&v)[16]);
 
 // Write 16 accumulator columns of one tensor-memory lane: row_a is the A-operand row the lane holds,
@@ -196,9 +221,15 @@ __device__ __forceinline__ void gt_store16_rows(const GemmParams& p, int row_a, 
     {
         if (p.out_f32) {
             float* dst = (float*)p.C + (size_t)row_a * p.ldc + col0;
+            if (col0 + 16 <= p.N && (((uintptr_t)dst) & 15) == 0) {
 #pragma unroll
-            for (int c = 0; c < 16; ++c)
-                if (col0 + c < p.N) dst[c] = v[c];
+                for (int k = 0; k < 4; ++k)
+                    reinterpret_cast<float4*>(dst)[k] = make_float4(v[4 * k], v[4 * k + 1], v[4 * k + 2], v[4 * k + 3]);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 16; ++c)
+                    if (col0 + c < p.N) dst[c] = v[c];
+            }
         } else {
             bf16* dst = (bf16*)p.C + (size_t)row_a * p.ldc + col0;
             if (col0 + 16 <= p.N && (((uintptr_t)dst) & 15) == 0) {

@@ -388,15 +388,21 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             }
             if (p.splits == 1) {
                 const int rows_b = min(BN, p.RB - tb * BN);
+                float next_bias[16];            // a piece ahead of its use
+                gt_load_bias(p, tb * BN, next_bias);
 #pragma unroll 1
                 for (int c0 = 0; c0 < BN; c0 += 16) {
                     if (p.staged && c0 >= rows_b) break;
                     uint32_t r[16];
+                    float bias[16];
+#pragma unroll
+                    for (int c = 0; c < 16; ++c) bias[c] = next_bias[c];
+                    if (c0 + 16 < BN) gt_load_bias(p, tb * BN + c0 + 16, next_bias);
                     tc_ld16(taddr + c0, r);
                     float v[16];
 #pragma unroll
                     for (int c = 0; c < 16; ++c) v[c] = __uint_as_float(r[c]);
-                    if (p.bias) gt_add_bias(p, row_a, tb * BN + c0, v);
+                    gt_sum_bias(p, row_a, tb * BN + c0, bias, v);
                     if (p.staged) gt_stage16(p, tiles, wq * 32 + lane, c0, v, lane);
                     else gt_store16(p, row_a, tb * BN + c0, v, lane);
                 }
@@ -675,14 +681,20 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 if (p.head_dim == 128) gt_store_qkv_rows<GP_BN, 128>(p, taddr, row_a, tb);
                 else gt_store_qkv_rows<GP_BN, 64>(p, taddr, row_a, tb);
             } else {
+                float next_bias[16];            // a piece ahead of its use
+                gt_load_bias(p, tb * GP_BN, next_bias);
 #pragma unroll 1
                 for (int c0 = 0; c0 < GP_BN; c0 += 16) {
                     uint32_t r[16];
+                    float bias[16];
+#pragma unroll
+                    for (int c = 0; c < 16; ++c) bias[c] = next_bias[c];
+                    if (c0 + 16 < GP_BN) gt_load_bias(p, tb * GP_BN + c0 + 16, next_bias);
                     tc_ld16(taddr + c0, r);
                     float v[16];
 #pragma unroll
                     for (int c = 0; c < 16; ++c) v[c] = __uint_as_float(r[c]);
-                    if (p.bias) gt_add_bias(p, row_a, tb * GP_BN + c0, v);
+                    gt_sum_bias(p, row_a, tb * GP_BN + c0, bias, v);
                     gt_store16(p, row_a, tb * GP_BN + c0, v, lane);
                 }
             }

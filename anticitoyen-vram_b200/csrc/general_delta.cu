@@ -32,12 +32,12 @@ __device__ __forceinline__ float dl_sigmoid(float z) { return 1.f / (1.f + expf(
 
 // ----------------------------------------------------------------------------- decays, removal vectors
 #define DP_TOK 8
-// grid (tiles of DP_TOK tokens, tiles of whole heads).  proj: rows of `ld` floats; w2t float [L][I].
-__global__ void __launch_bounds__(128)
+// grid (tiles of DP_TOK tokens, tiles of whole heads).  proj: rows of `ld` floats; w2t float [L][I].  Half of the block's
+// threads take the first four tokens' decays, half the others; then a warp a (token, head).
+__global__ void __launch_bounds__(256)
 delta_prepare_kernel(float* __restrict__ proj, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
                      float* __restrict__ w, float2* __restrict__ sc, int T_tokens, int H, int D, int L, int heads_per) {
-    extern __shared__ float th[];           // [L][DP_TOK]
-    pdl_launch_dependents();
+    extern __shared__ __align__(16) float th[];         // [L][DP_TOK]
     pdl_wait();
     const int I = H * D;
     const int t0 = blockIdx.x * DP_TOK;
@@ -48,40 +48,42 @@ delta_prepare_kernel(float* __restrict__ proj, int ld, const float* __restrict__
         th[j * DP_TOK + tt] = tt < n ? tanhf(proj[(size_t)(t0 + tt) * ld + 5 * (size_t)I + j]) : 0.f;
     }
     __syncthreads();
-    for (int c = h0 * D + threadIdx.x; c < h1 * D; c += blockDim.x) {
-        float z[DP_TOK];
+    const int half = threadIdx.x >> 7;
+    for (int c = h0 * D + (threadIdx.x & 127); c < h1 * D; c += 128) {
         const float z0 = w0[c];
-#pragma unroll
-        for (int tt = 0; tt < DP_TOK; ++tt) z[tt] = z0;
+        float z[4] = {z0, z0, z0, z0};
+#pragma unroll 8
         for (int j = 0; j < L; ++j) {
             const float m = w2t[(size_t)j * I + c];
-#pragma unroll
-            for (int tt = 0; tt < DP_TOK; ++tt) z[tt] = fmaf(m, th[j * DP_TOK + tt], z[tt]);
+            const float4 x = *reinterpret_cast<const float4*>(th + j * DP_TOK + half * 4);
+            z[0] = fmaf(m, x.x, z[0]); z[1] = fmaf(m, x.y, z[1]); z[2] = fmaf(m, x.z, z[2]); z[3] = fmaf(m, x.w, z[3]);
         }
 #pragma unroll
-        for (int tt = 0; tt < DP_TOK; ++tt)
-            if (tt < n) w[(size_t)(t0 + tt) * I + c] = expf(-DL_RATE * dl_sigmoid(z[tt]));
+        for (int i = 0; i < 4; ++i)
+            if (half * 4 + i < n) w[(size_t)(t0 + half * 4 + i) * I + c] = expf(-DL_RATE * dl_sigmoid(z[i]));
     }
-    // a warp a (token, head)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     for (int u = warp; u < n * (h1 - h0); u += nw) {
         const int tt = u / (h1 - h0), h = h0 + u - tt * (h1 - h0), t = t0 + tt;
         const float* k = proj + (size_t)t * ld + I + (size_t)h * D;
-        const float* kn = t + 1 < T_tokens ? k + ld : nullptr;
+        const float* kn = t + 1 < T_tokens ? k + ld : k;        // (behind the last token: never used)
         float* z = proj + (size_t)t * ld + 3 * (size_t)I + (size_t)h * D;
-        float ss = 0.f;
-        for (int e = lane; e < D; e += 32) ss = fmaf(k[e], k[e], ss);
-        ss = warp_sum(ss);
-        const float inv = 1.f / sqrtf(ss + DL_UNIT_EPS);
-        float dot = 0.f;
+        // one pass: the removal vector without its inverse root, and both sums
+        float ss = 0.f, dot = 0.f;
         for (int e = lane; e < D; e += 32) {
-            const float al = dl_sigmoid(z[e]) * (k[e] * inv);
-            z[e] = al;
-            if (kn) dot = fmaf(kn[e], al, dot);
+            const float kk = k[e], al = dl_sigmoid(z[e]) * kk;
+            ss = fmaf(kk, kk, ss);
+            dot = fmaf(kn[e], al, dot);
         }
+        ss = warp_sum(ss);
         dot = warp_sum(dot);
-        if (lane == 0) sc[(size_t)t * H + h] = make_float2(inv, dot);
+        const float inv = 1.f / sqrtf(ss + DL_UNIT_EPS);
+        for (int e = lane; e < D; e += 32) z[e] = dl_sigmoid(z[e]) * (k[e] * inv);
+        if (lane == 0) sc[(size_t)t * H + h] = make_float2(inv, dot * inv);
     }
+    // the recurrence has few, long-lived blocks: begun while these blocks fill the SMs they would pile up on whichever
+    // SMs have room first
+    pdl_launch_dependents();
 }
 
 // proj: float [T][ld], rows [r | k | v | z | g | x]; w: float [T][H*D]; sc: float2 [T][H].
@@ -93,12 +95,35 @@ ACV_API int acv_delta_prepare(float* proj, int ld, const float* w2t, const float
     heads_per = heads_per < 1 ? 1 : (heads_per > H ? H : heads_per);
     const dim3 grid((T_tokens + DP_TOK - 1) / DP_TOK, (H + heads_per - 1) / heads_per);
     if (grid.y > 65535) return ACV_ERR_SIZE;
-    acv_launch(PDL_MISC, delta_prepare_kernel, grid, 128, (size_t)L * DP_TOK * sizeof(float), stream, proj, ld, w2t, w0, w,
+    acv_launch(PDL_MISC, delta_prepare_kernel, grid, 256, (size_t)L * DP_TOK * sizeof(float), stream, proj, ld, w2t, w0, w,
                (float2*)sc, T_tokens, H, D, L, heads_per);
     return acv_launch_status();
 }
 
 // ----------------------------------------------------------------------------- the recurrence
+// two floats that one instruction works on
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 f2_pack(float a, float b) {
+    f2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float f2_total(f2 x) {
+    float a, b;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(x));
+    return a + b;
+}
+__device__ __forceinline__ f2 f2_fma(f2 a, f2 b, f2 c) {
+    f2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f2 f2_mul(f2 a, f2 b) {
+    f2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
 template <int G>
 __device__ __forceinline__ float lanes_sum(float v) {
 #pragma unroll
@@ -111,45 +136,52 @@ __device__ __forceinline__ float lanes_sum(float v) {
 // eight_first(lane) + i.
 template <int G>
 __device__ __forceinline__ void lanes_sum8(float (&v)[8], int lane) {
-    int n = 8;
+    if constexpr (G > 1) {
+        const bool up = lane & 1;
 #pragma unroll
-    for (int o = 1; o < G; o <<= 1) {
-        if (n > 1) {
-            n >>= 1;
-            const bool up = lane & o;
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-                if (i < n) {
-                    const float keep = up ? v[i + n] : v[i], give = up ? v[i] : v[i + n];
-                    v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
-                }
-        } else {
-            v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+        for (int i = 0; i < 4; ++i) {
+            const float keep = up ? v[i + 4] : v[i], give = up ? v[i] : v[i + 4];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
         }
     }
+    if constexpr (G > 2) {
+        const bool up = lane & 2;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const float keep = up ? v[i + 2] : v[i], give = up ? v[i] : v[i + 2];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+        }
+    }
+    if constexpr (G > 4) {
+        const bool up = lane & 4;
+        const float keep = up ? v[1] : v[0], give = up ? v[0] : v[1];
+        v[0] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+    }
+#pragma unroll
+    for (int o = 8; o < G; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
 }
 template <int G>
 __device__ __forceinline__ int eight_first(int lane) {
     return (G > 1 ? (lane & 1) * 4 : 0) + (G > 2 ? (lane & 2) : 0) + (G > 4 ? (lane & 4) >> 2 : 0);
 }
 
-template <int R, int G>
-__global__ void __launch_bounds__(DL_WARPS * 32)
+// R rows and C neighbouring columns of S a thread, G lanes a column group, NW warps a block
+template <int R, int G, int C, int NW>
+__global__ void __launch_bounds__(NW * 32)
 delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w, const float2* __restrict__ sc,
              float* __restrict__ state, const int* __restrict__ slots, const int* __restrict__ cu_q, float* __restrict__ o,
              int H, int D, int TC, int vec) {
-    constexpr int DP = R * G, CW = 32 / G, DVT = DL_WARPS * CW, R4 = R / 4;
+    constexpr int DP = R * G, DVT = NW * (32 / G) * C, R2 = R / 2;
     extern __shared__ __align__(16) float sm[];
     const int set = TC * (4 * DP + DVT + 2) + DP;       // floats of a staged chunk (k has one row more)
-    pdl_launch_dependents();
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DVT;
-    const int tid = threadIdx.x, nthr = DL_WARPS * 32, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, nthr = NW * 32, lane = tid & 31, warp = tid >> 5;
     if (DP != D || c0 + DVT > D)                        // columns that no copy writes read as zeros
         for (int i = tid; i < 2 * set; i += nthr) sm[i] = 0.f;
     pdl_wait();
     const int t0 = cu_q[seq], t1 = cu_q[seq + 1];
     if (t1 <= t0) return;
-    const int g = lane % G, cl = warp * CW + lane / G, c = c0 + cl;
+    const int g = lane % G, cl = (warp * (32 / G) + lane / G) * C, c = c0 + cl;
     const int I = H * D;
     float* st = state + ((size_t)slots[seq] * H + h) * D * D;
     const float* base = proj + (size_t)h * D;
@@ -195,30 +227,36 @@ delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w
         for (int tt = tid; tt < n; tt += nthr) reinterpret_cast<float2*>(ss)[tt] = sc[(size_t)(tb + tt) * H + h];
     };
 
-    float S[R];
+    // a thread's rows: pairs of neighbours, four neighbours to a 16-byte piece, pieces G apart
+    f2 S[C][R2];
 #pragma unroll
-    for (int i = 0; i < R; ++i) {
-        const int d = ((i >> 2) * G + g) * 4 + (i & 3);
-        S[i] = (d < D && c < D) ? st[(size_t)d * D + c] : 0.f;
-    }
+    for (int j = 0; j < C; ++j)
+#pragma unroll
+        for (int i = 0; i < R2; ++i) {
+            const int d = ((i >> 1) * G + g) * 4 + (i & 1) * 2;
+            const bool in = c + j < D;
+            S[j][i] = f2_pack(in && d < D ? st[(size_t)d * D + c + j] : 0.f, in && d + 1 < D ? st[(size_t)(d + 1) * D + c + j] : 0.f);
+        }
     __syncthreads();            // (the zeros stand before the first copies)
     stage(t0, sm);
     cp_async_commit();
-    auto vec4 = [&](const float* row, float (&x)[R]) {
+    auto rows = [&](const float* row, f2 (&x)[R2]) {
 #pragma unroll
-        for (int i4 = 0; i4 < R4; ++i4) {
-            const float4 q = reinterpret_cast<const float4*>(row)[i4 * G + g];
-            x[4 * i4] = q.x; x[4 * i4 + 1] = q.y; x[4 * i4 + 2] = q.z; x[4 * i4 + 3] = q.w;
+        for (int i = 0; i < R2; i += 2) {
+            const ulonglong2 q = reinterpret_cast<const ulonglong2*>(row)[(i >> 1) * G + g];
+            x[i] = q.x; x[i + 1] = q.y;
         }
     };
-    auto dot = [&](const float (&x)[R], const float (&y)[R]) {
-        float a0 = 0.f, a1 = 0.f;
+    auto dot = [&](const f2 (&x)[R2], const f2 (&y)[R2]) {
+        f2 a = f2_mul(x[0], y[0]);
 #pragma unroll
-        for (int i = 0; i < R; i += 2) { a0 = fmaf(x[i], y[i], a0); a1 = fmaf(x[i + 1], y[i + 1], a1); }
-        return a0 + a1;
+        for (int i = 1; i < R2; ++i) a = f2_fma(x[i], y[i], a);
+        return f2_total(a);
     };
-    float kc[R];                // the current token's key rows
-    float q = 0.f, cp = 0.f, p = 0.f;
+    f2 kc[R2];                  // the current token's key rows
+    float q[C], p[C], cp = 0.f;
+#pragma unroll
+    for (int j = 0; j < C; ++j) q[j] = p[j] = 0.f;
     bool first = true;
     int turn = 0;
     for (int tb = t0; tb < t1; tb += TC, turn ^= 1) {
@@ -233,85 +271,158 @@ delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w
         const float* vs = ks + (TC + 1) * DP + cl; const float2* ss = reinterpret_cast<const float2*>(ks + (TC + 1) * DP + TC * DVT);
         if (first) {
             first = false;
-            vec4(ks, kc);
-            q = lanes_sum<G>(dot(kc, S));
+            rows(ks, kc);
+#pragma unroll
+            for (int j = 0; j < C; ++j) q[j] = lanes_sum<G>(dot(kc, S[j]));
         }
-        // one token: from S_{t-1} and q = k_t^T X_{t-1} to S_t, this lane's part of o_t, and the next q
-        auto token = [&](int tt) {
-            float wr[R], al[R], kn[R], rr[R];
-            vec4(wsm + tt * DP, wr);
-            vec4(ks + (tt + 1) * DP, kn);
-            const float v = vs[tt * DVT];
-            const float2 nc = ss[tt];
-            float X[R];
+        // a token's own vectors, read one token ahead of their use
+        struct Token { f2 w[R2], k[R2], al[R2], r[R2]; float v[C]; float2 nc; };
+        auto fetch = [&](Token& x, int tt) {
+            rows(wsm + tt * DP, x.w);
+            rows(ks + (tt + 1) * DP, x.k);          // the key of the token behind it
+            rows(asm_ + tt * DP, x.al);
+            rows(rs + tt * DP, x.r);
 #pragma unroll
-            for (int i = 0; i < R; ++i) X[i] = fmaf(wr[i], S[i], kc[i] * v);
-            const float qn = lanes_sum<G>(dot(kn, X));
-            p = nc.x * fmaf(-cp, p, q);
-            vec4(asm_ + tt * DP, al);
-            vec4(rs + tt * DP, rr);
+            for (int j = 0; j < C; ++j) x.v[j] = vs[tt * DVT + j];
+            x.nc = ss[tt];
+        };
+        // one token: from S_{t-1} and q = k_t^T X_{t-1} to S_t, this lane's part of o_t, and the next q, whose exchanges
+        // between the lanes are issued among the work that does not wait for them
+        auto token = [&](const Token& x, float (&part)[C]) {
+            f2 X[C][R2];
+            float d[C];
 #pragma unroll
-            for (int i = 0; i < R; ++i) { S[i] = fmaf(-al[i], p, X[i]); kc[i] = kn[i]; }
-            q = qn;
-            cp = nc.y;
-            return dot(rr, S);
+            for (int j = 0; j < C; ++j) {
+                const f2 vv = f2_pack(x.v[j], x.v[j]);
+#pragma unroll
+                for (int i = 0; i < R2; ++i) X[j][i] = f2_fma(x.w[i], S[j][i], f2_mul(kc[i], vv));
+            }
+#pragma unroll
+            for (int j = 0; j < C; ++j) d[j] = dot(x.k, X[j]);
+            if constexpr (G > 1)
+#pragma unroll
+                for (int j = 0; j < C; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], 1);
+#pragma unroll
+            for (int j = 0; j < C; ++j) {
+                p[j] = x.nc.x * fmaf(-cp, p[j], q[j]);
+                const f2 np = f2_pack(-p[j], -p[j]);
+#pragma unroll
+                for (int i = 0; i < R2; ++i) S[j][i] = f2_fma(x.al[i], np, X[j][i]);
+            }
+            if constexpr (G > 2)
+#pragma unroll
+                for (int j = 0; j < C; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], 2);
+#pragma unroll
+            for (int j = 0; j < C; ++j) part[j] = dot(x.r, S[j]);
+#pragma unroll
+            for (int o = 4; o < G; o <<= 1)
+#pragma unroll
+                for (int j = 0; j < C; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], o);
+#pragma unroll
+            for (int j = 0; j < C; ++j) q[j] = d[j];
+#pragma unroll
+            for (int i = 0; i < R2; ++i) kc[i] = x.k[i];
+            cp = x.nc.y;
         };
         int tt = 0;
+        Token a;
+        fetch(a, 0);
         for (; tt + 8 <= n; tt += 8) {
-            float part[8];
+            float part[C][8];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) part[j] = token(tt + j);
-            lanes_sum8<G>(part, lane);
+            for (int i = 0; i < 8; ++i) {
+                Token b;
+                fetch(b, min(tt + i + 1, TC - 1));
+                float one[C];
+                token(a, one);
+                a = b;
+#pragma unroll
+                for (int j = 0; j < C; ++j) part[j][i] = one[j];
+            }
             constexpr int LEFT = G >= 8 ? 1 : 8 / G;
-            if ((G <= 8 || g < 8) && c < D) {
-                float* dst = o + (size_t)(tb + tt + eight_first<G>(lane)) * I + (size_t)h * D + c;
 #pragma unroll
-                for (int i = 0; i < LEFT; ++i) dst[(size_t)i * I] = part[i];
+            for (int j = 0; j < C; ++j) {
+                lanes_sum8<G>(part[j], lane);
+                if ((G <= 8 || g < 8) && c + j < D) {
+                    float* dst = o + (size_t)(tb + tt + eight_first<G>(lane)) * I + (size_t)h * D + c + j;
+#pragma unroll
+                    for (int i = 0; i < LEFT; ++i) dst[(size_t)i * I] = part[j][i];
+                }
             }
         }
         for (; tt < n; ++tt) {
-            const float part = lanes_sum<G>(token(tt));
-            if (g == 0 && c < D) o[(size_t)(tb + tt) * I + (size_t)h * D + c] = part;
+            float one[C];
+            fetch(a, tt);
+            token(a, one);
+#pragma unroll
+            for (int j = 0; j < C; ++j) {
+                one[j] = lanes_sum<G>(one[j]);
+                if (g == 0 && c + j < D) o[(size_t)(tb + tt) * I + (size_t)h * D + c + j] = one[j];
+            }
         }
         __syncthreads();
     }
-    if (c < D) {
+    pdl_launch_dependents();
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int d = ((i >> 2) * G + g) * 4 + (i & 3);
-            if (d < D) st[(size_t)d * D + c] = S[i];
+    for (int j = 0; j < C; ++j)
+#pragma unroll
+        for (int i = 0; i < R2; ++i) {
+            const int d = ((i >> 1) * G + g) * 4 + (i & 1) * 2;
+            float a, b;
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(S[j][i]));
+            if (c + j < D && d < D) st[(size_t)d * D + c + j] = a;
+            if (c + j < D && d + 1 < D) st[(size_t)(d + 1) * D + c + j] = b;
         }
-    }
 }
 
-template <int R, int G>
+template <int R, int G, int C, int NW>
 static int launch_delta(const float* proj, int ld, const float* w, const float2* sc, float* state, const int* slots,
                         const int* cu_q, float* o, int n_seqs, int H, int D, cudaStream_t stream) {
-    constexpr int DP = R * G, DVT = DL_WARPS * 32 / G;
+    constexpr int DP = R * G, DVT = NW * (32 / G) * C;
     const int per_token = (4 * DP + DVT + 2) * 4;
     int TC = 32;
-    while (TC > 8 && 2 * (TC * per_token + DP * 4) > 96 * 1024) TC -= 8;
+    while (TC > 8 && 2 * (TC * per_token + DP * 4) > 72 * 1024) TC -= 8;
     const size_t smem = 2 * ((size_t)TC * per_token + DP * 4);
     static AcvSmemConfig cfg;
     if (smem > 48 * 1024)
-        if (int e = acv_ensure_smem(cfg, delta_kernel<R, G>, (int)smem)) return e;
+        if (int e = acv_ensure_smem(cfg, delta_kernel<R, G, C, NW>, (int)smem)) return e;
     const int vec = D % 4 == 0 && ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)w & 15);
     const dim3 grid(n_seqs, H, (D + DVT - 1) / DVT);
     if (grid.y > 65535 || grid.z > 65535) return ACV_ERR_SIZE;
-    acv_launch(PDL_ATTN, delta_kernel<R, G>, grid, DL_WARPS * 32, smem, stream, proj, ld, w, sc, state, slots, cu_q, o, H, D, TC, vec);
+    acv_launch(PDL_ATTN, delta_kernel<R, G, C, NW>, grid, NW * 32, smem, stream, proj, ld, w, sc, state, slots, cu_q, o, H, D, TC, vec);
     return acv_launch_status();
 }
 
 // After acv_delta_prepare.  o: float [T][H*D]; state: float [slots][H][D][D]; heads of up to 512 channels.
+// form: 0 by the sizes; 1, 2, 3 (heads of 33 to 64 channels): one, two or four columns a thread.
 ACV_API int acv_delta(const float* proj, int ld, const float* w, const float* sc, float* state, const int* slots,
-                      const int* cu_q, float* o, int n_seqs, int H, int D, cudaStream_t stream) {
+                      const int* cu_q, float* o, int n_seqs, int H, int D, int form, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (H <= 0 || D <= 0 || D > 512) return ACV_ERR_SIZE;
-#define DL_CASE(RR, GG) \
-    if (D <= RR * GG) return launch_delta<RR, GG>(proj, ld, w, (const float2*)sc, state, slots, cu_q, o, n_seqs, H, D, stream);
-    DL_CASE(8, 1) DL_CASE(8, 2) DL_CASE(8, 4) DL_CASE(8, 8) DL_CASE(8, 16) DL_CASE(8, 32) DL_CASE(16, 32)
+#define DL_CASE(RR, GG, CC, WW) \
+    return launch_delta<RR, GG, CC, WW>(proj, ld, w, (const float2*)sc, state, slots, cu_q, o, n_seqs, H, D, stream);
+    if (D <= 8) DL_CASE(8, 1, 1, 4)
+    if (D <= 16) DL_CASE(8, 2, 1, 4)
+    if (D <= 32) DL_CASE(8, 4, 1, 4)
+    if (D <= 64) {
+        if (form == 1) DL_CASE(8, 8, 1, 4)
+        if (form == 3) DL_CASE(8, 8, 4, 2)
+        if (form == 4) DL_CASE(4, 16, 2, 4)
+        if (form == 5) DL_CASE(8, 8, 2, 4)
+        if (form == 6) DL_CASE(4, 16, 4, 2)
+        if (form == 7) DL_CASE(8, 8, 4, 1)
+        if (form == 8) DL_CASE(16, 4, 1, 2)
+        DL_CASE(8, 8, 2, 2)
+    }
+    if (D <= 128) {
+        if (form == 1) DL_CASE(8, 16, 1, 4)
+        if (form == 2) DL_CASE(8, 16, 4, 2)
+        if (form == 3) DL_CASE(16, 8, 2, 2)
+        DL_CASE(8, 16, 2, 4)
+    }
+    if (D <= 256) DL_CASE(8, 32, 1, 4)
+    DL_CASE(16, 32, 1, 4)
 #undef DL_CASE
-    return ACV_ERR_SIZE;
 }
 
 // ----------------------------------------------------------------------------- one token a request, everything

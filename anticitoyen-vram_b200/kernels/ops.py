@@ -91,7 +91,7 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_retention": [P, P, P, I, P, I, I, P, P, F, P, P, P, P, P, I, P, I, P, I, I, I, I, I, I, I, P],
         "acv_retention_gate": [P, I, P, I, P, I, I, I, I, F, F, I, P, I, I, I, P],
         "acv_delta_prepare": [P, I, P, P, P, P, I, I, I, I, P],
-        "acv_delta": [P, I, P, P, P, P, P, P, I, I, I, P],
+        "acv_delta": [P, I, P, P, P, P, P, P, I, I, I, I, P],
         "acv_delta_step_takes": [I, I],
         "acv_delta_step": [P, I, P, P, P, F, P, P, P, P, I, I, I, I, I, I, P],
         "acv_gemm_simt": [P, I, P, I, P, I, I, I, I, I, I, P],
@@ -1925,7 +1925,7 @@ def delta_prepare(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, deca
 
 
 def delta(proj: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
-          cu_q: torch.Tensor, num_seqs: int, out: torch.Tensor, num_heads: int, dim: int) -> torch.Tensor:
+          cu_q: torch.Tensor, num_seqs: int, out: torch.Tensor, num_heads: int, dim: int, form: int = 0) -> torch.Tensor:
     """S = diag(w) S - (a u) (u^T S) + k v^T, o = S^T r along each request's tokens, per head, after ``delta_prepare``;
     state float32 [slots, heads, dim, dim], out float32 [T, heads * dim].  Heads of up to 512 channels."""
     _need_cuda(proj, decay, scalars, state, out)
@@ -1933,7 +1933,7 @@ def delta(proj: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor, state:
             or state.shape[1:] != (num_heads, dim, dim) or out.shape != (proj.shape[0], num_heads * dim):
         raise KernelError("delta: a float32 state [slots, heads, dim, dim] and output [T, heads * dim] are wanted")
     _check(library().acv_delta(_p(proj), proj.stride(0), _p(decay), _p(scalars), _p(state), _p(slots), _p(cu_q), _p(out),
-                               num_seqs, num_heads, dim, _stream()), "delta")
+                               num_seqs, num_heads, dim, form, _stream()), "delta")
     return out
 
 
