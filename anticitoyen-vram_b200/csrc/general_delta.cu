@@ -7,112 +7,288 @@
 // A token's row of the input product is [r | k | v | z | g | x] (I = H*D each, then L): z the removal rate in front of its
 // sigmoid, g the output gate in front of its sigmoid, x the decay's inner values in front of their tanh.  All float.
 //
-//   acv_delta_prepare   w[t][c] = exp(-exp(-1/2) sigmoid(w0[c] + sum_j W2[c][j] tanh(x[t][j])));  z becomes
-//                       al = sigmoid(z) u in place;  per (token, head): 1 / sqrt(sum(k^2) + 1e-6), and <k_{t+1}, al_t>
-//   acv_delta           the recurrence for portions and single tokens, o float
+//   acv_delta_blocks    everything that does not need the state, for eight tokens of a request at a time
+//   acv_delta           the recurrence over those blocks, o float
 //   acv_delta_step      steps in which every request brings one token: all of the above, the head's norm, weight and gate
 //                       in one launch
 //
-// acv_delta.  A column of S is a recurrence of its own, S[:, c].  G lanes of a warp share a column (R rows each, in
-// registers); a block of four warps holds 4 * 32 / G columns and walks the tokens in chunks staged in shared memory, the next
-// chunk copied while one is computed.  What bounds a token's time is the chain product with u -> sum over the lanes
-// -> update -> next product; it is cut in half by looking one token ahead.  With X_t = diag(w_t) S_{t-1} + k_t v_t^T (known
-// before p_t = u_t^T S_{t-1} is):
+// Token by token the recurrence is a chain (product with u, a sum over the channels, an update, the next product) of some
+// 300 cycles a token.  Eight tokens at once the state enters linearly.  With W_i the product of the block's decays up to
+// token i (1..8, W_0 = 1; a decay is above 0.54, so W_8 is above 0.007 and may be divided by), al_i = a_i u_i, n_i the
+// inverse root, S the state in front of the block, and over the block's tokens i, j
 //
-//     S_t = X_t - al_t p_t,     p_{t+1} = n_{t+1} (k_{t+1}^T X_t - <k_{t+1}, al_t> p_t)       n = 1 / sqrt(sum(k^2) + 1e-6)
+//     k'_i = n_i W_{i-1} k_i    r'_i = W_i r_i      kd_j = k_j / W_j      ad_j = al_j / W_j
+//     K = low(k' kd^T)   A = low(k' ad^T)   (j < i)       P = low(r' kd^T)   Q = low(r' ad^T)   (j <= i)
 //
-// so the lanes' sum of k_{t+1}^T X_t runs beside token t's own update; <k_{t+1}, al_t> is a number per token and head.
+// the products p_i = u_i^T S_{i-1} obey p = k' S + K v - A p, and o = r' S + P v - Q p.  Solved for the state (I + A is
+// unit lower triangular; the solution is a forward substitution along the block's tokens, channel by channel):
+//
+//     kt = (I + A)^-1 k'    M = (I + A)^-1 K    rt = r' - Q kt    N = P - Q M
+//     p = kt S + M v        o = rt S + N v      S_8 = W_8 (S + sum_j kd_j v_j^T - ad_j p_j^T)
+//
+// A block's record (floats, channels padded to DP with zeros): kt [8][DP], rt [8][DP], W_8 kd [8][DP], -W_8 ad [8][DP],
+// W_8 [DP], M [8][8], N [8][8].  Tokens behind a portion's end are k = r = 0, w = 1: they change nothing.
 #include "mma_tiles.cuh"
 
-#define DL_WARPS 4
+#define DL_TOK 8
 #define DL_RATE 0.6065306597126334f         // exp(-1/2)
 #define DL_UNIT_EPS 1e-6f
 
 __device__ __forceinline__ float dl_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
-// ----------------------------------------------------------------------------- decays, removal vectors
-#define DP_TOK 8
-// grid (tiles of DP_TOK tokens, tiles of whole heads).  proj: rows of `ld` floats; w2t float [L][I].  Half of the block's
-// threads take the first four tokens' decays, half the others; then a warp a (token, head).
+// channels of a head as a record pads them
+static int delta_pad(int D) {
+    int p = 8;
+    while (p < D) p <<= 1;
+    return p;
+}
+static size_t delta_record(int DP) { return (size_t)33 * DP + 128; }
+
+// ----------------------------------------------------------------------------- the blocks' records
+// grid (blocks of tokens, tiles of `heads` whole heads); a thread owns NC channels (tid + 256 q).  proj: rows of `ld` floats; w2t
+// float [L][I]; rec: [items][H][record].
+template <int NC>
 __global__ void __launch_bounds__(256)
-delta_prepare_kernel(float* __restrict__ proj, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
-                     float* __restrict__ w, float2* __restrict__ sc, int T_tokens, int H, int D, int L, int heads_per) {
-    extern __shared__ __align__(16) float th[];         // [L][DP_TOK]
+delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
+                    const int* __restrict__ item_seq, const int* __restrict__ item_idx, const int* __restrict__ cu_q,
+                    float* __restrict__ rec, int H, int D, int DP, int L, int heads) {
+    extern __shared__ __align__(16) float sm[];
+    const int PD = (D + 3) & ~3;            // pitch of a row of channels
+    float* th = sm;                         // [L][8]
+    float* mA = th + L * DL_TOK;            // [heads][16][PD]: raw k, then k', r'
+    float* mB = mA + (size_t)heads * 16 * PD;       // [heads][16][PD]: kd, ad
+    float* gm = mB + (size_t)heads * 16 * PD;       // [heads][16][16]: [K A; P Q]
+    float* inv = gm + heads * 256;          // [heads][8]
     pdl_wait();
-    const int I = H * D;
-    const int t0 = blockIdx.x * DP_TOK;
-    const int n = min(DP_TOK, T_tokens - t0);
-    const int h0 = blockIdx.y * heads_per, h1 = min(H, h0 + heads_per);
-    for (int i = threadIdx.x; i < L * DP_TOK; i += blockDim.x) {
+    const int item = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int seq = item_seq[item], I = H * D;
+    const int t0 = cu_q[seq] + item_idx[item] * DL_TOK;
+    const int n = min(DL_TOK, cu_q[seq + 1] - t0);
+    const int h0 = blockIdx.y * heads, nh = min(heads, H - h0);
+    const float* base = proj + (size_t)t0 * ld;
+    for (int i = tid; i < L * DL_TOK; i += 256) {
         const int tt = i / L, j = i - tt * L;
-        th[j * DP_TOK + tt] = tt < n ? tanhf(proj[(size_t)(t0 + tt) * ld + 5 * (size_t)I + j]) : 0.f;
+        th[j * DL_TOK + tt] = tt < n ? tanhf(base[(size_t)tt * ld + 5 * (size_t)I + j]) : 0.f;
+    }
+    float k[NC][DL_TOK], r[NC][DL_TOK], z[NC][DL_TOK], w[NC][DL_TOK];
+#pragma unroll
+    for (int q = 0; q < NC; ++q) {
+        const int ch = tid + 256 * q, c = h0 * D + ch;
+        const bool in = ch < nh * D;
+#pragma unroll
+        for (int tt = 0; tt < DL_TOK; ++tt) {
+            const float* row = base + (size_t)tt * ld + c;
+            const bool there = in && tt < n;
+            r[q][tt] = there ? row[0] : 0.f;
+            k[q][tt] = there ? row[I] : 0.f;
+            z[q][tt] = there ? row[3 * (size_t)I] : 0.f;
+        }
+        if (in) {
+            const int hh = ch / D, e = ch - hh * D;
+#pragma unroll
+            for (int tt = 0; tt < DL_TOK; ++tt) mA[((size_t)hh * 16 + tt) * PD + e] = k[q][tt];
+        }
     }
     __syncthreads();
-    const int half = threadIdx.x >> 7;
-    for (int c = h0 * D + (threadIdx.x & 127); c < h1 * D; c += 128) {
-        const float z0 = w0[c];
-        float z[4] = {z0, z0, z0, z0};
-#pragma unroll 8
-        for (int j = 0; j < L; ++j) {
-            const float m = w2t[(size_t)j * I + c];
-            const float4 x = *reinterpret_cast<const float4*>(th + j * DP_TOK + half * 4);
-            z[0] = fmaf(m, x.x, z[0]); z[1] = fmaf(m, x.y, z[1]); z[2] = fmaf(m, x.z, z[2]); z[3] = fmaf(m, x.w, z[3]);
-        }
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-            if (half * 4 + i < n) w[(size_t)(t0 + half * 4 + i) * I + c] = expf(-DL_RATE * dl_sigmoid(z[i]));
-    }
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-    for (int u = warp; u < n * (h1 - h0); u += nw) {
-        const int tt = u / (h1 - h0), h = h0 + u - tt * (h1 - h0), t = t0 + tt;
-        const float* k = proj + (size_t)t * ld + I + (size_t)h * D;
-        const float* kn = t + 1 < T_tokens ? k + ld : k;        // (behind the last token: never used)
-        float* z = proj + (size_t)t * ld + 3 * (size_t)I + (size_t)h * D;
-        // one pass: the removal vector without its inverse root, and both sums
-        float ss = 0.f, dot = 0.f;
-        for (int e = lane; e < D; e += 32) {
-            const float kk = k[e], al = dl_sigmoid(z[e]) * kk;
-            ss = fmaf(kk, kk, ss);
-            dot = fmaf(kn[e], al, dot);
-        }
+    for (int u = warp; u < nh * DL_TOK; u += 8) {
+        const float* row = mA + ((size_t)(u >> 3) * 16 + (u & 7)) * PD;
+        float ss = 0.f;
+        for (int e = lane; e < D; e += 32) ss = fmaf(row[e], row[e], ss);
         ss = warp_sum(ss);
-        dot = warp_sum(dot);
-        const float inv = 1.f / sqrtf(ss + DL_UNIT_EPS);
-        for (int e = lane; e < D; e += 32) z[e] = dl_sigmoid(z[e]) * (k[e] * inv);
-        if (lane == 0) sc[(size_t)t * H + h] = make_float2(inv, dot * inv);
+        if (lane == 0) inv[u] = 1.f / sqrtf(ss + DL_UNIT_EPS);
     }
+#pragma unroll
+    for (int q = 0; q < NC; ++q) {
+        const int ch = tid + 256 * q, c = h0 * D + ch;
+        const bool in = ch < nh * D;
+        const float z0 = in ? w0[c] : 0.f;
+#pragma unroll
+        for (int tt = 0; tt < DL_TOK; ++tt) w[q][tt] = z0;
+        if (in) {
+#pragma unroll 4
+            for (int j = 0; j < L; ++j) {
+                const float m = w2t[(size_t)j * I + c];
+                const float4 a = *reinterpret_cast<const float4*>(th + j * DL_TOK), b = *reinterpret_cast<const float4*>(th + j * DL_TOK + 4);
+                w[q][0] = fmaf(m, a.x, w[q][0]); w[q][1] = fmaf(m, a.y, w[q][1]);
+                w[q][2] = fmaf(m, a.z, w[q][2]); w[q][3] = fmaf(m, a.w, w[q][3]);
+                w[q][4] = fmaf(m, b.x, w[q][4]); w[q][5] = fmaf(m, b.y, w[q][5]);
+                w[q][6] = fmaf(m, b.z, w[q][6]); w[q][7] = fmaf(m, b.w, w[q][7]);
+            }
+        }
+        float run = 1.f;                    // w becomes the running product W_i
+#pragma unroll
+        for (int tt = 0; tt < DL_TOK; ++tt) {
+            if (tt < n) run *= expf(-DL_RATE * dl_sigmoid(w[q][tt]));
+            w[q][tt] = run;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int q = 0; q < NC; ++q) {
+        const int ch = tid + 256 * q;
+        if (ch < nh * D) {
+            const int hh = ch / D, e = ch - hh * D;
+            float* a = mA + (size_t)hh * 16 * PD + e;
+            float* b = mB + (size_t)hh * 16 * PD + e;
+#pragma unroll
+            for (int tt = 0; tt < DL_TOK; ++tt) {
+                const float over = 1.f / w[q][tt], ni = inv[hh * DL_TOK + tt];
+                const float kp = ni * k[q][tt] * (tt ? w[q][tt - 1] : 1.f);
+                r[q][tt] *= w[q][tt];
+                z[q][tt] = dl_sigmoid(z[q][tt]) * (k[q][tt] * ni) * over;       // ad
+                k[q][tt] *= over;                                               // kd
+                a[tt * PD] = kp; a[(8 + tt) * PD] = r[q][tt];
+                b[tt * PD] = k[q][tt]; b[(8 + tt) * PD] = z[q][tt];
+            }
+        }
+    }
+    if (PD != D)                            // the channels that fill a row's last 16 bytes
+        for (int i = tid; i < nh * 32 * (PD - D); i += 256) {
+            const int row = i / (PD - D), e = D + i % (PD - D);
+            (row < nh * 16 ? mA + (size_t)row * PD : mB + (size_t)(row - nh * 16) * PD)[e] = 0.f;
+        }
+    __syncthreads();
+    // [k'; r'] [kd; ad]^T, 16 x 16 for every head: a warp four of its rows, eight lanes share the channels of a 4 x 4 tile
+    for (int u = warp; u < nh * 4; u += 8) {
+        const int hh = u >> 2, ti = u & 3, tj = lane >> 3, kg = lane & 7;
+        const float* a = mA + ((size_t)hh * 16 + ti * 4) * PD;
+        const float* b = mB + ((size_t)hh * 16 + tj * 4) * PD;
+        float acc[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) acc[i] = 0.f;
+        for (int e = kg * 4; e < PD; e += 32) {
+            float4 x[4], y[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                x[i] = *reinterpret_cast<const float4*>(a + (size_t)i * PD + e);
+                y[i] = *reinterpret_cast<const float4*>(b + (size_t)i * PD + e);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    float s = acc[i * 4 + j];
+                    s = fmaf(x[i].x, y[j].x, s); s = fmaf(x[i].y, y[j].y, s);
+                    s = fmaf(x[i].z, y[j].z, s); s = fmaf(x[i].w, y[j].w, s);
+                    acc[i * 4 + j] = s;
+                }
+        }
+        // the eight lanes' sums: every exchange halves the values that a lane still carries
+        int first = 0;
+#pragma unroll
+        for (int s = 0; s < 3; ++s) {
+            const int half = 8 >> s;
+            const bool up = lane & (1 << s);
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+                if (i < half) {
+                    const float keep = up ? acc[i + half] : acc[i], give = up ? acc[i] : acc[i + half];
+                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1 << s);
+                }
+            first += up ? half : 0;
+        }
+        float* dst = gm + hh * 256 + (ti * 4 + (first >> 2)) * 16 + tj * 4 + (first & 3);
+        dst[0] = acc[0];
+        dst[1] = acc[1];
+    }
+    __syncthreads();
+    // forward substitution, a thread a channel; behind the channels eight columns a head for M and N
+    float* out = rec + ((size_t)item * H + h0) * (33 * (size_t)DP + 128);
+    const size_t rs = 33 * (size_t)DP + 128;
+#pragma unroll
+    for (int q = 0; q < NC; ++q) {
+        const int ch = tid + 256 * q;
+        if (ch < nh * D) {
+            const int hh = ch / D, e = ch - hh * D;
+            const float* g = gm + hh * 256;
+            const float* a = mA + (size_t)hh * 16 * PD + e;
+            float* o = out + hh * rs + e;
+            const float last = w[q][DL_TOK - 1];
+            float kt[DL_TOK];
+#pragma unroll
+            for (int i = 0; i < DL_TOK; ++i) {
+                float s = a[i * PD], t = r[q][i];
+#pragma unroll
+                for (int j = 0; j < i; ++j) s = fmaf(-g[i * 16 + 8 + j], kt[j], s);
+                kt[i] = s;
+#pragma unroll
+                for (int j = 0; j <= i; ++j) t = fmaf(-g[(8 + i) * 16 + 8 + j], kt[j], t);
+                o[(size_t)i * DP] = s;
+                o[(size_t)(8 + i) * DP] = t;
+                o[(size_t)(16 + i) * DP] = k[q][i] * last;
+                o[(size_t)(24 + i) * DP] = -(z[q][i] * last);
+            }
+            o[(size_t)32 * DP] = last;
+        }
+    }
+    for (int u = tid; u < nh * 8; u += 256) {
+        const int hh = u >> 3, c = u & 7;
+        const float* g = gm + hh * 256;
+        float* o = out + hh * rs + 33 * (size_t)DP + c;
+        float m[DL_TOK];
+#pragma unroll
+        for (int i = 0; i < DL_TOK; ++i) {
+            float s = c < i ? g[i * 16 + c] : 0.f, t = c <= i ? g[(8 + i) * 16 + c] : 0.f;
+#pragma unroll
+            for (int j = 0; j < i; ++j) s = fmaf(-g[i * 16 + 8 + j], m[j], s);
+            m[i] = s;
+#pragma unroll
+            for (int j = 0; j <= i; ++j) t = fmaf(-g[(8 + i) * 16 + 8 + j], m[j], t);
+            o[i * 8] = s;
+            o[64 + i * 8] = t;
+        }
+    }
+    if (DP != D)
+        for (int i = tid; i < nh * 33 * (DP - D); i += 256) {
+            const int row = i / (DP - D), hh = row / 33;
+            out[hh * rs + (size_t)(row - hh * 33) * DP + D + i % (DP - D)] = 0.f;
+        }
     // the recurrence has few, long-lived blocks: begun while these blocks fill the SMs they would pile up on whichever
     // SMs have room first
     pdl_launch_dependents();
 }
 
-// proj: float [T][ld], rows [r | k | v | z | g | x]; w: float [T][H*D]; sc: float2 [T][H].
-ACV_API int acv_delta_prepare(float* proj, int ld, const float* w2t, const float* w0, float* w, float* sc, int T_tokens, int H,
-                              int D, int L, cudaStream_t stream) {
-    if (T_tokens <= 0) return 0;
-    if (H <= 0 || D <= 0 || L <= 0 || L > 1024 || ld < 5 * H * D + L) return ACV_ERR_SIZE;
-    int heads_per = 128 / D;
-    heads_per = heads_per < 1 ? 1 : (heads_per > H ? H : heads_per);
-    const dim3 grid((T_tokens + DP_TOK - 1) / DP_TOK, (H + heads_per - 1) / heads_per);
-    if (grid.y > 65535) return ACV_ERR_SIZE;
-    acv_launch(PDL_MISC, delta_prepare_kernel, grid, 256, (size_t)L * DP_TOK * sizeof(float), stream, proj, ld, w2t, w0, w,
-               (float2*)sc, T_tokens, H, D, L, heads_per);
+// proj: float [T][ld], rows [r | k | v | z | g | x]; the step's n_items blocks of up to eight tokens (item_seq: the request, item_idx:
+// the block's number in it); rec: float [n_items][H][33 pad(D) + 128].
+ACV_API int acv_delta_blocks(const float* proj, int ld, const float* w2t, const float* w0, const int* item_seq,
+                             const int* item_idx, const int* cu_q, float* rec, int n_items, int H, int D, int L,
+                             cudaStream_t stream) {
+    if (n_items <= 0) return 0;
+    if (H <= 0 || D <= 0 || D > 512 || L <= 0 || L > 1024 || ld < 5 * H * D + L) return ACV_ERR_SIZE;
+    int heads = 256 / D;
+    heads = heads < 1 ? 1 : (heads > 32 ? 32 : heads);
+    if (heads > H) heads = H;
+    const int PD = (D + 3) & ~3;
+    const size_t smem = ((size_t)L * DL_TOK + (size_t)heads * (32 * PD + 256 + DL_TOK)) * sizeof(float);
+    const dim3 grid(n_items, (H + heads - 1) / heads);
+    if (grid.y > 65535 || smem > 200 * 1024) return ACV_ERR_SIZE;
+#define DB_LAUNCH(N)                                                                                                          \
+    do {                                                                                                                      \
+        static AcvSmemConfig cfg;                                                                                             \
+        if (smem > 48 * 1024)                                                                                                 \
+            if (int e = acv_ensure_smem(cfg, delta_blocks_kernel<N>, (int)smem)) return e;                                    \
+        acv_launch(PDL_MISC, delta_blocks_kernel<N>, grid, 256, smem, stream, proj, ld, w2t, w0, item_seq, item_idx, cu_q,    \
+                   rec, H, D, delta_pad(D), L, heads);                                                                        \
+    } while (0)
+    if (D <= 256) DB_LAUNCH(1);
+    else DB_LAUNCH(2);
+#undef DB_LAUNCH
     return acv_launch_status();
 }
 
+ACV_API int acv_delta_record_floats(int D) { return (int)delta_record(delta_pad(D)); }
+
 // ----------------------------------------------------------------------------- the recurrence
-// two floats that one instruction works on
-typedef unsigned long long f2;
+// Columns of S are recurrences of their own.  A thread keeps R rows of C neighbouring columns in registers (pairs of rows,
+// two to an instruction), G lanes share a column, a block's NW warps hold NW * 32 / G * C columns and walk the request's
+// blocks of eight tokens; records and values are copied asynchronously, STAGES - 1 blocks ahead.
+typedef unsigned long long f2;              // two floats that one instruction works on
 __device__ __forceinline__ f2 f2_pack(float a, float b) {
     f2 r;
     asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
     return r;
 }
-__device__ __forceinline__ float f2_total(f2 x) {
-    float a, b;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(x));
-    return a + b;
-}
+__device__ __forceinline__ void f2_split(f2 x, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(x)); }
 __device__ __forceinline__ f2 f2_fma(f2 a, f2 b, f2 c) {
     f2 r;
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
@@ -124,16 +300,9 @@ __device__ __forceinline__ f2 f2_mul(f2 a, f2 b) {
     return r;
 }
 
-template <int G>
-__device__ __forceinline__ float lanes_sum(float v) {
-#pragma unroll
-    for (int o = 1; o < G; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-
-// The sums over the G lanes of a column of eight values each: every step halves the values that a lane still carries,
-// so eight sums cost 7 exchanges at G = 8.  Afterwards v[0 .. 8/min(G,8)) of a lane are the totals of the values
-// eight_first(lane) + i.
+// The sums over the G lanes of a column of eight values each (one for every token of the block): every exchange halves the
+// values that a lane still carries.  Afterwards v[0 .. LEFT) of a lane are the totals of the tokens first_of(lane) + i,
+// LEFT = G >= 8 ? 1 : 8 / G.
 template <int G>
 __device__ __forceinline__ void lanes_sum8(float (&v)[8], int lane) {
     if constexpr (G > 1) {
@@ -161,72 +330,54 @@ __device__ __forceinline__ void lanes_sum8(float (&v)[8], int lane) {
     for (int o = 8; o < G; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
 }
 template <int G>
-__device__ __forceinline__ int eight_first(int lane) {
+__device__ __forceinline__ int first_of(int lane) {
     return (G > 1 ? (lane & 1) * 4 : 0) + (G > 2 ? (lane & 2) : 0) + (G > 4 ? (lane & 4) >> 2 : 0);
 }
+// the lane (within its column's G) and the place at which token e's total lies
+template <int G>
+__device__ __forceinline__ constexpr int lane_of(int e) {
+    return (G > 1 ? (e >> 2) & 1 : 0) | (G > 2 ? ((e >> 1) & 1) << 1 : 0) | (G > 4 ? (e & 1) << 2 : 0);
+}
+template <int G>
+__device__ __forceinline__ constexpr int place_of(int e) { return G >= 8 ? 0 : e & (8 / G - 1); }
 
-// R rows and C neighbouring columns of S a thread, G lanes a column group, NW warps a block
-template <int R, int G, int C, int NW>
+template <int R, int G, int C, int NW, int STAGES>
 __global__ void __launch_bounds__(NW * 32)
-delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w, const float2* __restrict__ sc,
-             float* __restrict__ state, const int* __restrict__ slots, const int* __restrict__ cu_q, float* __restrict__ o,
-             int H, int D, int TC, int vec) {
-    constexpr int DP = R * G, DVT = NW * (32 / G) * C, R2 = R / 2;
+delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int ld, float* __restrict__ state,
+             const int* __restrict__ slots, const int* __restrict__ cu_q, const int* __restrict__ first_block,
+             float* __restrict__ o, int H, int D, int vec) {
+    constexpr int DP = R * G, DVT = NW * (32 / G) * C, R2 = R / 2, LEFT = G >= 8 ? 1 : 8 / G;
+    constexpr int REC = 33 * DP + 128, SET = REC + 8 * DVT, NT = NW * 32;
     extern __shared__ __align__(16) float sm[];
-    const int set = TC * (4 * DP + DVT + 2) + DP;       // floats of a staged chunk (k has one row more)
-    const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DVT;
-    const int tid = threadIdx.x, nthr = NW * 32, lane = tid & 31, warp = tid >> 5;
-    if (DP != D || c0 + DVT > D)                        // columns that no copy writes read as zeros
-        for (int i = tid; i < 2 * set; i += nthr) sm[i] = 0.f;
     pdl_wait();
+    const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DVT;
     const int t0 = cu_q[seq], t1 = cu_q[seq + 1];
     if (t1 <= t0) return;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int g = lane % G, cl = (warp * (32 / G) + lane / G) * C, c = c0 + cl;
-    const int I = H * D;
+    const int I = H * D, nb = (t1 - t0 + 7) >> 3;
     float* st = state + ((size_t)slots[seq] * H + h) * D * D;
-    const float* base = proj + (size_t)h * D;
+    const float* recs = rec + ((size_t)first_block[seq] * H + h) * REC;
+    const float* vals = proj + (size_t)t0 * ld + 2 * (size_t)I + (size_t)h * D + c0;
 
-    auto stage = [&](int tb, float* s) {
-        const int n = min(TC, t1 - tb);
-        float* rs = s; float* ws_ = rs + TC * DP; float* as_ = ws_ + TC * DP; float* ks = as_ + TC * DP;
-        float* vs = ks + (TC + 1) * DP; float* ss = vs + TC * DVT;
+    auto stage = [&](int b) {
+        float* s = sm + (b % STAGES) * SET;
+        const float* src = recs + (size_t)b * H * REC;
+        for (int i = tid * 4; i < REC; i += NT * 4) cp_async16(smem_u32(s + i), src + i, true);
+        float* vs = s + REC;
         if (vec) {
-            const int d4 = D >> 2;
-            for (int i = tid; i < (n + 1) * d4; i += nthr) {
-                const int tt = i / d4, e = (i - tt * d4) << 2, t = tb + tt;
-                const float* row = base + (size_t)t * ld + e;
-                const bool in = t < t1;
-                cp_async16(smem_u32(ks + tt * DP + e), in ? (const void*)(row + I) : (const void*)proj, in);
-                if (tt < n) {
-                    cp_async16(smem_u32(rs + tt * DP + e), row, true);
-                    cp_async16(smem_u32(as_ + tt * DP + e), row + 3 * (size_t)I, true);
-                    cp_async16(smem_u32(ws_ + tt * DP + e), w + (size_t)t * I + (size_t)h * D + e, true);
-                }
-            }
-            for (int i = tid; i < n * (DVT >> 2); i += nthr) {
-                const int tt = i / (DVT >> 2), e = (i - tt * (DVT >> 2)) << 2;
-                const bool in = c0 + e < D;
-                cp_async16(smem_u32(vs + tt * DVT + e), in ? (const void*)(base + (size_t)(tb + tt) * ld + 2 * (size_t)I + c0 + e) : (const void*)proj, in);
+            for (int i = tid * 4; i < 8 * DVT; i += NT * 4) {
+                const int tt = i / DVT, e = i % DVT, t = b * 8 + tt;
+                const bool in = t < t1 - t0 && c0 + e < D;
+                cp_async16(smem_u32(vs + i), in ? (const void*)(vals + (size_t)t * ld + e) : (const void*)proj, in);
             }
         } else {
-            for (int i = tid; i < (n + 1) * D; i += nthr) {
-                const int tt = i / D, e = i - tt * D, t = tb + tt;
-                const float* row = base + (size_t)t * ld + e;
-                ks[tt * DP + e] = t < t1 ? row[I] : 0.f;
-                if (tt < n) {
-                    rs[tt * DP + e] = row[0];
-                    as_[tt * DP + e] = row[3 * (size_t)I];
-                    ws_[tt * DP + e] = w[(size_t)t * I + (size_t)h * D + e];
-                }
-            }
-            for (int i = tid; i < n * DVT; i += nthr) {
-                const int tt = i / DVT, e = i - tt * DVT;
-                vs[i] = c0 + e < D ? base[(size_t)(tb + tt) * ld + 2 * (size_t)I + c0 + e] : 0.f;
+            for (int i = tid; i < 8 * DVT; i += NT) {
+                const int tt = i / DVT, e = i % DVT, t = b * 8 + tt;
+                vs[i] = t < t1 - t0 && c0 + e < D ? vals[(size_t)t * ld + e] : 0.f;
             }
         }
-        for (int tt = tid; tt < n; tt += nthr) reinterpret_cast<float2*>(ss)[tt] = sc[(size_t)(tb + tt) * H + h];
     };
-
     // a thread's rows: pairs of neighbours, four neighbours to a 16-byte piece, pieces G apart
     f2 S[C][R2];
 #pragma unroll
@@ -237,9 +388,11 @@ delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w
             const bool in = c + j < D;
             S[j][i] = f2_pack(in && d < D ? st[(size_t)d * D + c + j] : 0.f, in && d + 1 < D ? st[(size_t)(d + 1) * D + c + j] : 0.f);
         }
-    __syncthreads();            // (the zeros stand before the first copies)
-    stage(t0, sm);
-    cp_async_commit();
+#pragma unroll
+    for (int b = 0; b < STAGES - 1; ++b) {
+        if (b < nb) stage(b);
+        cp_async_commit();
+    }
     auto rows = [&](const float* row, f2 (&x)[R2]) {
 #pragma unroll
         for (int i = 0; i < R2; i += 2) {
@@ -251,116 +404,94 @@ delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w
         f2 a = f2_mul(x[0], y[0]);
 #pragma unroll
         for (int i = 1; i < R2; ++i) a = f2_fma(x[i], y[i], a);
-        return f2_total(a);
+        float lo, hi;
+        f2_split(a, lo, hi);
+        return lo + hi;
     };
-    f2 kc[R2];                  // the current token's key rows
-    float q[C], p[C], cp = 0.f;
-#pragma unroll
-    for (int j = 0; j < C; ++j) q[j] = p[j] = 0.f;
-    bool first = true;
-    int turn = 0;
-    for (int tb = t0; tb < t1; tb += TC, turn ^= 1) {
-        const int n = min(TC, t1 - tb);
-        float* s = sm + turn * set;
-        // (the other set was read in the turn before this one, whose last barrier every thread has passed)
-        if (tb + TC < t1) stage(tb + TC, sm + (turn ^ 1) * set);
+    for (int b = 0; b < nb; ++b) {
+        cp_async_wait<STAGES - 2>();
+        __syncthreads();                    // block b is there; everyone is done with block b - 1, whose buffer is filled next
+        if (b + STAGES - 1 < nb) stage(b + STAGES - 1);
         cp_async_commit();
-        cp_async_wait<1>();
-        __syncthreads();
-        const float* rs = s; const float* wsm = rs + TC * DP; const float* asm_ = wsm + TC * DP; const float* ks = asm_ + TC * DP;
-        const float* vs = ks + (TC + 1) * DP + cl; const float2* ss = reinterpret_cast<const float2*>(ks + (TC + 1) * DP + TC * DVT);
-        if (first) {
-            first = false;
-            rows(ks, kc);
+        const float* s = sm + (b % STAGES) * SET;
+        const float* mn = s + 33 * DP;
+        const float* vs = s + REC + cl;
+        float y[C][8], z[C][8], v[C][8];
+        f2 x[R2];
 #pragma unroll
-            for (int j = 0; j < C; ++j) q[j] = lanes_sum<G>(dot(kc, S[j]));
+        for (int i = 0; i < 8; ++i) {
+            rows(s + i * DP, x);
+#pragma unroll
+            for (int j = 0; j < C; ++j) y[j][i] = dot(x, S[j]);
         }
-        // a token's own vectors, read one token ahead of their use
-        struct Token { f2 w[R2], k[R2], al[R2], r[R2]; float v[C]; float2 nc; };
-        auto fetch = [&](Token& x, int tt) {
-            rows(wsm + tt * DP, x.w);
-            rows(ks + (tt + 1) * DP, x.k);          // the key of the token behind it
-            rows(asm_ + tt * DP, x.al);
-            rows(rs + tt * DP, x.r);
 #pragma unroll
-            for (int j = 0; j < C; ++j) x.v[j] = vs[tt * DVT + j];
-            x.nc = ss[tt];
-        };
-        // one token: from S_{t-1} and q = k_t^T X_{t-1} to S_t, this lane's part of o_t, and the next q, whose exchanges
-        // between the lanes are issued among the work that does not wait for them
-        auto token = [&](const Token& x, float (&part)[C]) {
-            f2 X[C][R2];
-            float d[C];
+        for (int j = 0; j < C; ++j) lanes_sum8<G>(y[j], lane);
 #pragma unroll
-            for (int j = 0; j < C; ++j) {
-                const f2 vv = f2_pack(x.v[j], x.v[j]);
+        for (int i = 0; i < 8; ++i) {
+            rows(s + (8 + i) * DP, x);
 #pragma unroll
-                for (int i = 0; i < R2; ++i) X[j][i] = f2_fma(x.w[i], S[j][i], f2_mul(kc[i], vv));
-            }
+            for (int j = 0; j < C; ++j) z[j][i] = dot(x, S[j]);
+        }
 #pragma unroll
-            for (int j = 0; j < C; ++j) d[j] = dot(x.k, X[j]);
-            if constexpr (G > 1)
+        for (int i = 0; i < 8; ++i)
 #pragma unroll
-                for (int j = 0; j < C; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], 1);
+            for (int j = 0; j < C; ++j) v[j][i] = vs[i * DVT + j];
+        // this lane's tokens: p (its sum over the values of the tokens before it), later o
+        const int e0 = first_of<G>(lane);
+#pragma unroll
+        for (int l = 0; l < LEFT; ++l) {
+            const float4 m0 = *reinterpret_cast<const float4*>(mn + (e0 + l) * 8), m1 = *reinterpret_cast<const float4*>(mn + (e0 + l) * 8 + 4);
 #pragma unroll
             for (int j = 0; j < C; ++j) {
-                p[j] = x.nc.x * fmaf(-cp, p[j], q[j]);
-                const f2 np = f2_pack(-p[j], -p[j]);
-#pragma unroll
-                for (int i = 0; i < R2; ++i) S[j][i] = f2_fma(x.al[i], np, X[j][i]);
+                float a = fmaf(m0.x, v[j][0], y[j][l]), d = m0.y * v[j][1];
+                a = fmaf(m0.z, v[j][2], a); d = fmaf(m0.w, v[j][3], d);
+                a = fmaf(m1.x, v[j][4], a); d = fmaf(m1.y, v[j][5], d);
+                y[j][l] = fmaf(m1.z, v[j][6], a) + d;
             }
-            if constexpr (G > 2)
+        }
+        rows(s + 32 * DP, x);
 #pragma unroll
-                for (int j = 0; j < C; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], 2);
+        for (int j = 0; j < C; ++j)
 #pragma unroll
-            for (int j = 0; j < C; ++j) part[j] = dot(x.r, S[j]);
+            for (int i = 0; i < R2; ++i) S[j][i] = f2_mul(x[i], S[j][i]);
 #pragma unroll
-            for (int o = 4; o < G; o <<= 1)
-#pragma unroll
-                for (int j = 0; j < C; ++j) d[j] += __shfl_xor_sync(0xffffffffu, d[j], o);
-#pragma unroll
-            for (int j = 0; j < C; ++j) q[j] = d[j];
-#pragma unroll
-            for (int i = 0; i < R2; ++i) kc[i] = x.k[i];
-            cp = x.nc.y;
-        };
-        int tt = 0;
-        Token a;
-        fetch(a, 0);
-        for (; tt + 8 <= n; tt += 8) {
-            float part[C][8];
-#pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                Token b;
-                fetch(b, min(tt + i + 1, TC - 1));
-                float one[C];
-                token(a, one);
-                a = b;
-#pragma unroll
-                for (int j = 0; j < C; ++j) part[j][i] = one[j];
-            }
-            constexpr int LEFT = G >= 8 ? 1 : 8 / G;
+        for (int i = 0; i < 8; ++i) {
+            rows(s + (16 + i) * DP, x);
 #pragma unroll
             for (int j = 0; j < C; ++j) {
-                lanes_sum8<G>(part[j], lane);
-                if ((G <= 8 || g < 8) && c + j < D) {
-                    float* dst = o + (size_t)(tb + tt + eight_first<G>(lane)) * I + (size_t)h * D + c + j;
+                const f2 vv = f2_pack(v[j][i], v[j][i]);
 #pragma unroll
-                    for (int i = 0; i < LEFT; ++i) dst[(size_t)i * I] = part[j][i];
+                for (int q = 0; q < R2; ++q) S[j][q] = f2_fma(x[q], vv, S[j][q]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            rows(s + (24 + i) * DP, x);
+#pragma unroll
+            for (int j = 0; j < C; ++j) {
+                const float p = G > 1 ? __shfl_sync(0xffffffffu, y[j][place_of<G>(i)], lane_of<G>(i), G) : y[j][i];
+                const f2 pp = f2_pack(p, p);
+#pragma unroll
+                for (int q = 0; q < R2; ++q) S[j][q] = f2_fma(x[q], pp, S[j][q]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < C; ++j) lanes_sum8<G>(z[j], lane);
+        if (G <= 8 || g < 8) {
+#pragma unroll
+            for (int l = 0; l < LEFT; ++l) {
+                const float4 m0 = *reinterpret_cast<const float4*>(mn + 64 + (e0 + l) * 8), m1 = *reinterpret_cast<const float4*>(mn + 64 + (e0 + l) * 8 + 4);
+                const int t = t0 + b * 8 + e0 + l;
+#pragma unroll
+                for (int j = 0; j < C; ++j) {
+                    float a = fmaf(m0.x, v[j][0], z[j][l]), d = m0.y * v[j][1];
+                    a = fmaf(m0.z, v[j][2], a); d = fmaf(m0.w, v[j][3], d);
+                    a = fmaf(m1.x, v[j][4], a); d = fmaf(m1.y, v[j][5], d);
+                    a = fmaf(m1.z, v[j][6], a); d = fmaf(m1.w, v[j][7], d);
+                    if (t < t1 && c + j < D) o[(size_t)t * I + (size_t)h * D + c + j] = a + d;
                 }
             }
         }
-        for (; tt < n; ++tt) {
-            float one[C];
-            fetch(a, tt);
-            token(a, one);
-#pragma unroll
-            for (int j = 0; j < C; ++j) {
-                one[j] = lanes_sum<G>(one[j]);
-                if (g == 0 && c + j < D) o[(size_t)(tb + tt) * I + (size_t)h * D + c + j] = one[j];
-            }
-        }
-        __syncthreads();
     }
     pdl_launch_dependents();
 #pragma unroll
@@ -369,59 +500,60 @@ delta_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w
         for (int i = 0; i < R2; ++i) {
             const int d = ((i >> 1) * G + g) * 4 + (i & 1) * 2;
             float a, b;
-            asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(S[j][i]));
+            f2_split(S[j][i], a, b);
             if (c + j < D && d < D) st[(size_t)d * D + c + j] = a;
             if (c + j < D && d + 1 < D) st[(size_t)(d + 1) * D + c + j] = b;
         }
 }
 
-template <int R, int G, int C, int NW>
-static int launch_delta(const float* proj, int ld, const float* w, const float2* sc, float* state, const int* slots,
-                        const int* cu_q, float* o, int n_seqs, int H, int D, cudaStream_t stream) {
-    constexpr int DP = R * G, DVT = NW * (32 / G) * C;
-    const int per_token = (4 * DP + DVT + 2) * 4;
-    int TC = 32;
-    while (TC > 8 && 2 * (TC * per_token + DP * 4) > 72 * 1024) TC -= 8;
-    const size_t smem = 2 * ((size_t)TC * per_token + DP * 4);
+template <int R, int G, int C, int NW, int STAGES>
+static int launch_delta(const float* rec, const float* proj, int ld, float* state, const int* slots, const int* cu_q,
+                        const int* first_block, float* o, int n_seqs, int H, int D, cudaStream_t stream) {
+    constexpr int DVT = NW * (32 / G) * C;
+    constexpr size_t smem = (size_t)STAGES * (33 * R * G + 128 + 8 * DVT) * sizeof(float);
+    static_assert(smem <= 227 * 1024 && DVT % 4 == 0, "a block's stages fit, values come in 16-byte pieces");
     static AcvSmemConfig cfg;
     if (smem > 48 * 1024)
-        if (int e = acv_ensure_smem(cfg, delta_kernel<R, G, C, NW>, (int)smem)) return e;
-    const int vec = D % 4 == 0 && ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)w & 15);
+        if (int e = acv_ensure_smem(cfg, delta_kernel<R, G, C, NW, STAGES>, (int)smem)) return e;
+    const int vec = D % 4 == 0 && ld % 4 == 0 && !((uintptr_t)proj & 15);
     const dim3 grid(n_seqs, H, (D + DVT - 1) / DVT);
     if (grid.y > 65535 || grid.z > 65535) return ACV_ERR_SIZE;
-    acv_launch(PDL_ATTN, delta_kernel<R, G, C, NW>, grid, NW * 32, smem, stream, proj, ld, w, sc, state, slots, cu_q, o, H, D, TC, vec);
+    acv_launch(PDL_ATTN, delta_kernel<R, G, C, NW, STAGES>, grid, NW * 32, smem, stream, rec, proj, ld, state, slots, cu_q,
+               first_block, o, H, D, vec);
     return acv_launch_status();
 }
 
-// After acv_delta_prepare.  o: float [T][H*D]; state: float [slots][H][D][D]; heads of up to 512 channels.
-// form: 0 by the sizes; 1, 2, 3 (heads of 33 to 64 channels): one, two or four columns a thread.
-ACV_API int acv_delta(const float* proj, int ld, const float* w, const float* sc, float* state, const int* slots,
-                      const int* cu_q, float* o, int n_seqs, int H, int D, int form, cudaStream_t stream) {
+// After acv_delta_blocks.  first_block: the number of each request's first block among the step's items; o: float [T][H*D];
+// state: float [slots][H][D][D]; heads of up to 512 channels.  form: 0, or a choice among the shapes of a block (timing).
+ACV_API int acv_delta(const float* rec, const float* proj, int ld, float* state, const int* slots, const int* cu_q,
+                      const int* first_block, float* o, int n_seqs, int H, int D, int form, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (H <= 0 || D <= 0 || D > 512) return ACV_ERR_SIZE;
-#define DL_CASE(RR, GG, CC, WW) \
-    return launch_delta<RR, GG, CC, WW>(proj, ld, w, (const float2*)sc, state, slots, cu_q, o, n_seqs, H, D, stream);
-    if (D <= 8) DL_CASE(8, 1, 1, 4)
-    if (D <= 16) DL_CASE(8, 2, 1, 4)
-    if (D <= 32) DL_CASE(8, 4, 1, 4)
+    if ((uintptr_t)rec & 15) return ACV_ERR_ALIGN;
+#define DL_CASE(RR, GG, CC, WW, SS) \
+    return launch_delta<RR, GG, CC, WW, SS>(rec, proj, ld, state, slots, cu_q, first_block, o, n_seqs, H, D, stream);
+    if (D <= 8) DL_CASE(8, 1, 1, 1, 3)
+    if (D <= 16) DL_CASE(8, 2, 1, 1, 3)
+    if (D <= 32) DL_CASE(8, 4, 1, 4, 3)
     if (D <= 64) {
-        if (form == 1) DL_CASE(8, 8, 1, 4)
-        if (form == 3) DL_CASE(8, 8, 4, 2)
-        if (form == 4) DL_CASE(4, 16, 2, 4)
-        if (form == 5) DL_CASE(8, 8, 2, 4)
-        if (form == 6) DL_CASE(4, 16, 4, 2)
-        if (form == 7) DL_CASE(8, 8, 4, 1)
-        if (form == 8) DL_CASE(16, 4, 1, 2)
-        DL_CASE(8, 8, 2, 2)
+        if (form == 1) DL_CASE(8, 8, 1, 4, 3)
+        if (form == 2) DL_CASE(8, 8, 2, 2, 3)
+        if (form == 3) DL_CASE(8, 8, 4, 2, 3)
+        if (form == 4) DL_CASE(4, 16, 2, 4, 3)
+        if (form == 5) DL_CASE(8, 8, 2, 4, 3)
+        if (form == 6) DL_CASE(4, 16, 4, 2, 3)
+        if (form == 7) DL_CASE(8, 8, 4, 1, 3)
+        if (form == 8) DL_CASE(4, 16, 4, 4, 3)
+        DL_CASE(8, 8, 2, 2, 3)
     }
     if (D <= 128) {
-        if (form == 1) DL_CASE(8, 16, 1, 4)
-        if (form == 2) DL_CASE(8, 16, 4, 2)
-        if (form == 3) DL_CASE(16, 8, 2, 2)
-        DL_CASE(8, 16, 2, 4)
+        if (form == 1) DL_CASE(8, 16, 1, 4, 3)
+        if (form == 2) DL_CASE(8, 16, 4, 2, 3)
+        if (form == 3) DL_CASE(4, 32, 4, 4, 3)
+        DL_CASE(8, 16, 2, 4, 3)
     }
-    if (D <= 256) DL_CASE(8, 32, 1, 4)
-    DL_CASE(16, 32, 1, 4)
+    if (D <= 256) DL_CASE(8, 32, 1, 4, 3)
+    DL_CASE(16, 32, 1, 4, 2)
 #undef DL_CASE
 }
 

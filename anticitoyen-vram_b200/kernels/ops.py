@@ -90,8 +90,9 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_gated_scan": [P, P, P, I, P, P, P, P, P, P, I, P, I, P, I, I, I, I, I, P],
         "acv_retention": [P, P, P, I, P, I, I, P, P, F, P, P, P, P, P, I, P, I, P, I, I, I, I, I, I, I, P],
         "acv_retention_gate": [P, I, P, I, P, I, I, I, I, F, F, I, P, I, I, I, P],
-        "acv_delta_prepare": [P, I, P, P, P, P, I, I, I, I, P],
-        "acv_delta": [P, I, P, P, P, P, P, P, I, I, I, I, P],
+        "acv_delta_blocks": [P, I, P, P, P, P, P, P, I, I, I, I, P],
+        "acv_delta_record_floats": [I],
+        "acv_delta": [P, P, I, P, P, P, P, P, I, I, I, I, P],
         "acv_delta_step_takes": [I, I],
         "acv_delta_step": [P, I, P, P, P, F, P, P, P, P, I, I, I, I, I, I, P],
         "acv_gemm_simt": [P, I, P, I, P, I, I, I, I, I, I, P],
@@ -1908,42 +1909,62 @@ def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, u: t
 
 
 # ----------------------------------------------------------------------------- a generalized delta rule
-def delta_prepare(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor,
-                  num_heads: int, dim: int) -> None:
-    """What enters the delta recurrence, from a token's row of the input product [r | k | v | z | g | x] (float32 [T, >=
-    5 I + L], I = heads * dim, L rows of ``w2_t`` [L, I]): ``decay`` [T, I] = exp(-exp(-1/2) sigmoid(w0 + tanh(x) w2_t));
-    z in place becomes sigmoid(z) u, u = k / sqrt(sum(k^2) + 1e-6) per head; ``scalars`` [T, heads, 2]: that inverse root,
-    and the product of the next token's k with the new z (csrc/general_delta.cu)."""
-    _need_cuda(proj, w2_t, w0, decay, scalars)
-    T, (L, I) = proj.shape[0], w2_t.shape
-    if any(t.dtype != torch.float32 for t in (proj, w2_t, w0, decay, scalars)) or I != num_heads * dim or proj.stride(1) != 1 \
-            or proj.shape[1] < 5 * I + L or not all(t.is_contiguous() for t in (w2_t, w0, decay, scalars)) \
-            or decay.shape != (T, I) or scalars.shape != (T, num_heads, 2):
-        raise KernelError("delta_prepare: float32 rows [r | k | v | z | g | x], w2_t [L, I], w0 [I], decay [T, I] and scalars [T, heads, 2] are wanted")
-    _check(library().acv_delta_prepare(_p(proj), proj.stride(0), _p(w2_t), _p(w0), _p(decay), _p(scalars), T, num_heads, dim, L,
-                                       _stream()), "delta_prepare")
+DELTA_TOKENS = 8        # tokens of a request that the delta recurrence takes at once
 
 
-def delta(proj: torch.Tensor, decay: torch.Tensor, scalars: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
-          cu_q: torch.Tensor, num_seqs: int, out: torch.Tensor, num_heads: int, dim: int, form: int = 0) -> torch.Tensor:
-    """S = diag(w) S - (a u) (u^T S) + k v^T, o = S^T r along each request's tokens, per head, after ``delta_prepare``;
-    state float32 [slots, heads, dim, dim], out float32 [T, heads * dim].  Heads of up to 512 channels."""
-    _need_cuda(proj, decay, scalars, state, out)
+def delta_work(q_lens) -> tuple[dict, dict]:
+    """The step's blocks of up to ``DELTA_TOKENS`` tokens: int32 arrays (the request and the block's number in it for every
+    block; the number of each request's first block), and how many there are."""
+    import numpy as np
+    arrays, values = segment_work(q_lens, DELTA_TOKENS)
+    n = np.asarray([max(1, -(-int(q) // DELTA_TOKENS)) for q in q_lens], dtype=np.int64)
+    first = np.concatenate([np.zeros(1, np.int64), np.cumsum(n)[:-1]]) if len(n) else np.zeros(0, np.int64)
+    return {**arrays, "first_block": first.astype(np.int32)}, {"n_items": values["n_items"]}
+
+
+def delta_work_decode(padded: int) -> tuple[dict, dict]:
+    """The same for a batch of ``padded`` requests with one token each."""
+    return delta_work([1] * padded)
+
+
+def delta_blocks(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, cu_q: torch.Tensor, num_heads: int, dim: int,
+                 work: dict) -> torch.Tensor:
+    """Everything in the delta recurrence that does not need the state, for every block of ``delta_work``: from a token's row
+    of the input product [r | k | v | z | g | x] (float32 [T, >= 5 I + L], I = heads * dim, L rows of ``w2_t`` [L, I]) the
+    block's record (csrc/general_delta.cu), float32 [blocks, heads, record]."""
+    _need_cuda(proj, w2_t, w0)
+    L, I = w2_t.shape
+    if any(t.dtype != torch.float32 for t in (proj, w2_t, w0)) or I != num_heads * dim or proj.stride(1) != 1 \
+            or proj.shape[1] < 5 * I + L or not w2_t.is_contiguous() or not w0.is_contiguous():
+        raise KernelError("delta_blocks: float32 rows [r | k | v | z | g | x], w2_t [L, I] and w0 [I] are wanted")
+    lib = library()
+    rec = torch.empty((work["n_items"], num_heads, lib.acv_delta_record_floats(dim)), device=proj.device, dtype=torch.float32)
+    _check(lib.acv_delta_blocks(_p(proj), proj.stride(0), _p(w2_t), _p(w0), _p(work["seg_seq"]), _p(work["seg_idx"]), _p(cu_q),
+                                _p(rec), work["n_items"], num_heads, dim, L, _stream()), "delta_blocks")
+    return rec
+
+
+def delta(rec: torch.Tensor, proj: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor, num_seqs: int,
+          out: torch.Tensor, num_heads: int, dim: int, work: dict, form: int = 0) -> torch.Tensor:
+    """S = diag(w) S - (a u) (u^T S) + k v^T, o = S^T r along each request's tokens, per head, over the records of
+    ``delta_blocks`` (and the values in ``proj``); state float32 [slots, heads, dim, dim], out float32 [T, heads * dim].
+    Heads of up to 512 channels.  ``form``: a choice among the kernel's block shapes (0: by the sizes)."""
+    _need_cuda(rec, proj, state, out)
     if state.dtype != torch.float32 or not state.is_contiguous() or out.dtype != torch.float32 or not out.is_contiguous() \
-            or state.shape[1:] != (num_heads, dim, dim) or out.shape != (proj.shape[0], num_heads * dim):
+            or state.shape[1:] != (num_heads, dim, dim) or out.shape != (proj.shape[0], num_heads * dim) or not rec.is_contiguous():
         raise KernelError("delta: a float32 state [slots, heads, dim, dim] and output [T, heads * dim] are wanted")
-    _check(library().acv_delta(_p(proj), proj.stride(0), _p(decay), _p(scalars), _p(state), _p(slots), _p(cu_q), _p(out),
+    _check(library().acv_delta(_p(rec), _p(proj), proj.stride(0), _p(state), _p(slots), _p(cu_q), _p(work["first_block"]), _p(out),
                                num_seqs, num_heads, dim, form, _stream()), "delta")
     return out
 
 
 def general_delta(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, weight: torch.Tensor, eps: float,
                   state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor, num_seqs: int, max_q_len: int,
-                  out: torch.Tensor, num_heads: int, dim: int, rank: int) -> torch.Tensor:
-    """From the input product (``delta_prepare``; z is changed in place) to the gated heads: every head's o of the
-    recurrence to unit RMS (``eps``), times ``weight`` (float32 [heads * dim]), times sigmoid(g), into ``out`` (a view
-    [T, heads * dim] with dense rows).  Steps in which every request brings one token are one launch; others prepare,
-    recurrence and gate."""
+                  out: torch.Tensor, num_heads: int, dim: int, rank: int, work: dict | None) -> torch.Tensor:
+    """From the input product (``delta_blocks``) to the gated heads: every head's o of the recurrence to unit RMS
+    (``eps``), times ``weight`` (float32 [heads * dim]), times sigmoid(g), into ``out`` (a view [T, heads * dim] with dense
+    rows).  Steps in which every request brings one token are one launch; others blocks, recurrence and gate (``work``:
+    the step's ``delta_work``)."""
     _need_cuda(proj, w2_t, w0, weight, state, out)
     T, I = out.shape
     if weight.dtype != torch.float32 or weight.numel() != I or not weight.is_contiguous() or out.stride(1) != 1:
@@ -1957,9 +1978,7 @@ def general_delta(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, weig
                                   _p(cu_q), _p(out), out.stride(0), num_seqs, num_heads, dim, rank, dtype_code(out.dtype),
                                   _stream()), "delta_step")
         return out
-    decay = torch.empty((T, I), device=proj.device, dtype=torch.float32)
-    scalars = torch.empty((T, num_heads, 2), device=proj.device, dtype=torch.float32)
-    delta_prepare(proj, w2_t, w0, decay, scalars, num_heads, dim)
+    rec = delta_blocks(proj, w2_t, w0, cu_q, num_heads, dim, work)
     o = torch.empty((T, I), device=proj.device, dtype=torch.float32)
-    delta(proj, decay, scalars, state, slots, cu_q, num_seqs, o, num_heads, dim)
+    delta(rec, proj, state, slots, cu_q, num_seqs, o, num_heads, dim, work)
     return retention_gate(o, proj[:, 4 * I:5 * I], out, num_heads, dim, eps, weight=weight, gate_fn="sigmoid")

@@ -347,6 +347,7 @@ class GeneralDelta(Mixer):
     whatever the file holds."""
 
     NAMES = {n: n for n in ("r", "k", "v", "a", "a.b", "g", "w1", "w2", "w0", "norm", "o")}
+    metadata_key = "delta_blocks"       # the recurrence takes a request's tokens in blocks (``ops.delta_work``)
 
     def __init__(self, hidden_size: int, num_heads: int, dim: int, norm_eps: float, prefix: str = "mix.",
                  names: dict | None = None) -> None:
@@ -359,6 +360,12 @@ class GeneralDelta(Mixer):
 
     def _n(self, role: str) -> str:
         return self.prefix + self.names[role]
+
+    def step_metadata(self, q_lens, kv_lens, cu_q) -> StepMetadata:
+        return StepMetadata(*ops.delta_work(q_lens))
+
+    def decode_metadata(self, padded: int, max_kv: int) -> StepMetadata:
+        return StepMetadata(*ops.delta_work_decode(padded))
 
     def cache_need(self):
         return StateNeed((self.num_heads, self.dim, self.dim), "float32")
@@ -410,7 +417,8 @@ class GeneralDelta(Mixer):
     def inner(self, h, ctx, cache: CacheView, out) -> None:
         proj = self.qkv(h, out_dtype=torch.float32)
         ops.general_delta(proj, self.w2_t, self.w0, self.norm_weight, self.norm_eps, cache.state, ctx.state_slots[cache.group],
-                          ctx.cu_q, ctx.num_seqs, ctx.max_q_len, out, self.num_heads, self.dim, self.rank)
+                          ctx.cu_q, ctx.num_seqs, ctx.max_q_len, out, self.num_heads, self.dim, self.rank,
+                          ctx.work.get(self.metadata_key))
 
     def forward(self, h, ctx, cache: CacheView):
         out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)

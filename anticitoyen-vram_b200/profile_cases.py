@@ -295,7 +295,7 @@ def retention_case(q_len: int, batch: int, reps: int, H: int = 16, D: int = 64, 
 
 
 def delta_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, rank: int = 32) -> dict:
-    """The delta recurrence behind its input product: prepare, recurrence and gate of ``batch`` portions of ``q_len`` tokens,
+    """The delta recurrence behind its input product: blocks, recurrence and gate of ``batch`` portions of ``q_len`` tokens,
     or the one launch of steps of single tokens."""
     T, I = q_len * batch, H * D
     dev = "cuda:0"
@@ -306,17 +306,19 @@ def delta_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, rank
     slots = torch.arange(batch, dtype=torch.int32, device=dev)
     cu = torch.arange(0, T + 1, q_len, dtype=torch.int32, device=dev)
     out = torch.empty(T, I, device=dev, dtype=torch.bfloat16)
-    decay, scalars, o = torch.empty(T, I, device=dev), torch.empty(T, H, 2, device=dev), torch.empty(T, I, device=dev)
-    us_all = _time(lambda i: ops.general_delta(proj, w2_t, w0, weight, 1e-6, state, slots, cu, batch, q_len, out, H, D, rank), reps)
-    us_prep = _time(lambda i: ops.delta_prepare(proj, w2_t, w0, decay, scalars, H, D), reps)
-    proj[:, 3 * I:4 * I] *= 0.1
-    us = _time(lambda i: ops.delta(proj, decay, scalars, state, slots, cu, batch, o, H, D), reps)
+    o = torch.empty(T, I, device=dev)
+    arrays, values = ops.delta_work([q_len] * batch)
+    work = {**{k: torch.as_tensor(v).to(dev) for k, v in arrays.items()}, **values}
+    us_all = _time(lambda i: ops.general_delta(proj, w2_t, w0, weight, 1e-6, state, slots, cu, batch, q_len, out, H, D, rank, work), reps)
+    rec = ops.delta_blocks(proj, w2_t, w0, cu, H, D, work)
+    us_prep = _time(lambda i: ops.delta_blocks(proj, w2_t, w0, cu, H, D, work), reps)
+    us = _time(lambda i: ops.delta(rec, proj, state, slots, cu, batch, o, H, D, work), reps)
     us_gate = _time(lambda i: ops.retention_gate(o, proj[:, 4 * I:5 * I], out, H, D, 1e-6, weight=weight, gate_fn="sigmoid"), reps)
     flops = 10.0 * H * D * D * T        # five multiply-adds a state element and token
     print(f"delta q_len={q_len} batch={batch} heads={H} of {D}x{D}: all {us_all:.1f} us, recurrence {us:.1f} us ({flops / us / 1e6:.2f} "
-          f"TFLOP/s float, state {2 * batch * H * D * D * 4 / us / 1e3:.0f} GB/s), prepare {us_prep:.1f} us, gate {us_gate:.1f} us; "
+          f"TFLOP/s float, state {2 * batch * H * D * D * 4 / us / 1e3:.0f} GB/s), blocks {us_prep:.1f} us, gate {us_gate:.1f} us; "
           f"all: state {2 * batch * H * D * D * 4 / us_all / 1e3:.0f} GB/s")
-    return {"kernel": "delta", "q_len": q_len, "batch": batch, "us": us, "us_all": us_all, "us_prepare": us_prep, "us_gate": us_gate,
+    return {"kernel": "delta", "q_len": q_len, "batch": batch, "us": us, "us_all": us_all, "us_blocks": us_prep, "us_gate": us_gate,
             "tflops_f32": flops / us / 1e6}
 
 

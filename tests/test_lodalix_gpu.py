@@ -149,7 +149,7 @@ def test_decoding_token_by_token(folders, which, dtype):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("which", ["A", "B", "C", "D"])
 def test_portions_of_any_size(folders, which, dtype):
-    """Portions down to two tokens, longer than a chunk of the recurrence kernel (70 tokens), and single tokens between
+    """Portions down to two tokens, longer than a block of the recurrence kernel (8 tokens) and no multiple of it, and single tokens between
     them (which take the step's kernel for portions or the one for single tokens)."""
     f = folders[which]
     runner = make_runner(f, dtype)

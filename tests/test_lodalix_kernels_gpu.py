@@ -36,6 +36,12 @@ def delta_proj(h, W, pad):
     return dev(np.concatenate(cols, axis=1))
 
 
+def blocks(q_lens):
+    from acvram_b200.kernels import ops
+    arrays, values = ops.delta_work(q_lens)
+    return {**{k: i32(v) for k, v in arrays.items()}, **values}
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,D,L", [(2, 8, 3), (1, 4, 1), (3, 10, 5), (2, 16, 8), (3, 20, 7), (2, 32, 16), (5, 48, 4), (2, 64, 32),
                                    (1, 100, 9), (2, 128, 12), (1, 200, 6), (1, 300, 5)])
@@ -59,7 +65,7 @@ def test_delta_over_steps(H, D, L, dtype):
             T = proj.shape[0]
             wide = torch.full((T, I + 5), 7.0, device=DEV, dtype=DT[dtype])       # the heads land in columns of wider rows
             ops.general_delta(proj, w2t, w0, nw, 1e-5, state, i32([slots_of[r] for r, _, _ in step]), cu, len(step),
-                              max(c for _, _, c in step), wide[:, :I], H, D, L)
+                              max(c for _, _, c in step), wide[:, :I], H, D, L, blocks([c for _, _, c in step]))
             assert bool((wide[:, I:] == 7.0).all())
             at = 0
             for r, a0, c in step:
@@ -73,8 +79,8 @@ def test_delta_over_steps(H, D, L, dtype):
 
 @pytest.mark.parametrize("D", [12, 64])
 def test_a_long_portion_equals_token_by_token(D):
-    """300 tokens of one request as one portion (many chunks of the kernel), one by one (the one-launch kernel) and cut
-    around a single token; decays close to 1 and few removals, so that the first tokens still weigh at the end."""
+    """300 tokens of one request as one portion (many blocks of the kernel), one by one (the one-launch kernel) and cut
+    around a single token (blocks of eight tokens begin anywhere); decays close to 1 and few removals, so that the first tokens still weigh at the end."""
     from acvram_b200.kernels import ops
     rng = np.random.default_rng(D)
     n, H, L, width = 300, 2, 4, 32
@@ -91,7 +97,7 @@ def test_a_long_portion_equals_token_by_token(D):
         at = 0
         for c in cuts:
             proj = delta_proj(h[at:at + c], W, 0)
-            ops.general_delta(proj, w2t, w0, nw, 1e-5, state, i32([1]), i32([0, c]), 1, c, got[at:at + c], H, D, L)
+            ops.general_delta(proj, w2t, w0, nw, 1e-5, state, i32([1]), i32([0, c]), 1, c, got[at:at + c], H, D, L, blocks([c]))
             at += c
         close(got, want, 2e-4, f"cuts {cuts[:3]}")
 
