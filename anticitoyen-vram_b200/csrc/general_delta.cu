@@ -34,7 +34,8 @@
 #define DL_RATE 0.6065306597126334f         // exp(-1/2)
 #define DL_UNIT_EPS 1e-6f
 
-__device__ __forceinline__ float dl_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+// (the quotient within two units in the last place; a denominator past 2^126 gives 0)
+__device__ __forceinline__ float dl_sigmoid(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
 
 // channels of a head as a record pads them
 static int delta_pad(int D) {
@@ -48,7 +49,7 @@ static size_t delta_record(int DP) { return (size_t)33 * DP + 128; }
 // grid (blocks of tokens, tiles of `heads` whole heads); a thread owns NC channels (tid + 256 q).  proj: rows of `ld` floats; w2t
 // float [L][I]; rec: [items][H][record].
 template <int NC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, NC == 1 ? 3 : 1)
 delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w2t, const float* __restrict__ w0,
                     const int* __restrict__ item_seq, const int* __restrict__ item_idx, const int* __restrict__ cu_q,
                     float* __restrict__ rec, int H, int D, int DP, int L, int heads) {
@@ -105,7 +106,7 @@ delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restr
 #pragma unroll
         for (int tt = 0; tt < DL_TOK; ++tt) w[q][tt] = z0;
         if (in) {
-#pragma unroll 4
+#pragma unroll 8
             for (int j = 0; j < L; ++j) {
                 const float m = w2t[(size_t)j * I + c];
                 const float4 a = *reinterpret_cast<const float4*>(th + j * DL_TOK), b = *reinterpret_cast<const float4*>(th + j * DL_TOK + 4);
@@ -132,7 +133,7 @@ delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restr
             float* b = mB + (size_t)hh * 16 * PD + e;
 #pragma unroll
             for (int tt = 0; tt < DL_TOK; ++tt) {
-                const float over = 1.f / w[q][tt], ni = inv[hh * DL_TOK + tt];
+                const float over = __fdividef(1.f, w[q][tt]), ni = inv[hh * DL_TOK + tt];
                 const float kp = ni * k[q][tt] * (tt ? w[q][tt - 1] : 1.f);
                 r[q][tt] *= w[q][tt];
                 z[q][tt] = dl_sigmoid(z[q][tt]) * (k[q][tt] * ni) * over;       // ad
@@ -192,6 +193,10 @@ delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restr
         dst[1] = acc[1];
     }
     __syncthreads();
+    auto row8 = [](const float* p, float (&x)[DL_TOK]) {
+        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+    };
     // forward substitution, a thread a channel; behind the channels eight columns a head for M and N
     float* out = rec + ((size_t)item * H + h0) * (33 * (size_t)DP + 128);
     const size_t rs = 33 * (size_t)DP + 128;
@@ -207,12 +212,14 @@ delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restr
             float kt[DL_TOK];
 #pragma unroll
             for (int i = 0; i < DL_TOK; ++i) {
-                float s = a[i * PD], t = r[q][i];
+                float s = a[i * PD], t = r[q][i], gr[DL_TOK], gq[DL_TOK];
+                row8(g + i * 16 + 8, gr);
+                row8(g + (8 + i) * 16 + 8, gq);
 #pragma unroll
-                for (int j = 0; j < i; ++j) s = fmaf(-g[i * 16 + 8 + j], kt[j], s);
+                for (int j = 0; j < i; ++j) s = fmaf(-gr[j], kt[j], s);
                 kt[i] = s;
 #pragma unroll
-                for (int j = 0; j <= i; ++j) t = fmaf(-g[(8 + i) * 16 + 8 + j], kt[j], t);
+                for (int j = 0; j <= i; ++j) t = fmaf(-gq[j], kt[j], t);
                 o[(size_t)i * DP] = s;
                 o[(size_t)(8 + i) * DP] = t;
                 o[(size_t)(16 + i) * DP] = k[q][i] * last;
@@ -300,32 +307,19 @@ __device__ __forceinline__ f2 f2_mul(f2 a, f2 b) {
     return r;
 }
 
-// The sums over the G lanes of a column of eight values each (one for every token of the block): every exchange halves the
-// values that a lane still carries.  Afterwards v[0 .. LEFT) of a lane are the totals of the tokens first_of(lane) + i,
-// LEFT = G >= 8 ? 1 : 8 / G.
+// The sums over the G lanes of a column of eight values each, one for every token of the block.  A lane keeps token i ^ m in
+// v[i], m = first_of(lane): the half that it gives away at an exchange is then the half that its partner keeps, and an
+// exchange halves what a lane still carries (7 exchanges at G = 8).  Afterwards v[0 .. LEFT) are the totals of the tokens
+// m + i, LEFT = G >= 8 ? 1 : 8 / G.
 template <int G>
-__device__ __forceinline__ void lanes_sum8(float (&v)[8], int lane) {
-    if constexpr (G > 1) {
-        const bool up = lane & 1;
+__device__ __forceinline__ void lanes_sum8(float (&v)[8]) {
+    if constexpr (G > 1)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const float keep = up ? v[i + 4] : v[i], give = up ? v[i] : v[i + 4];
-            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-        }
-    }
-    if constexpr (G > 2) {
-        const bool up = lane & 2;
+        for (int i = 0; i < 4; ++i) v[i] += __shfl_xor_sync(0xffffffffu, v[i + 4], 1);
+    if constexpr (G > 2)
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const float keep = up ? v[i + 2] : v[i], give = up ? v[i] : v[i + 2];
-            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
-        }
-    }
-    if constexpr (G > 4) {
-        const bool up = lane & 4;
-        const float keep = up ? v[1] : v[0], give = up ? v[0] : v[1];
-        v[0] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
-    }
+        for (int i = 0; i < 2; ++i) v[i] += __shfl_xor_sync(0xffffffffu, v[i + 2], 2);
+    if constexpr (G > 4) v[0] += __shfl_xor_sync(0xffffffffu, v[1], 4);
 #pragma unroll
     for (int o = 8; o < G; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
 }
@@ -347,6 +341,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
              const int* __restrict__ slots, const int* __restrict__ cu_q, const int* __restrict__ first_block,
              float* __restrict__ o, int H, int D, int vec) {
     constexpr int DP = R * G, DVT = NW * (32 / G) * C, R2 = R / 2, LEFT = G >= 8 ? 1 : 8 / G;
+    constexpr int PF = R < 4 ? 1 : 2;       // pairs in a piece that one load brings
     constexpr int REC = 33 * DP + 128, SET = REC + 8 * DVT, NT = NW * 32;
     extern __shared__ __align__(16) float sm[];
     pdl_wait();
@@ -356,6 +351,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int g = lane % G, cl = (warp * (32 / G) + lane / G) * C, c = c0 + cl;
     const int I = H * D, nb = (t1 - t0 + 7) >> 3;
+    const int e0 = first_of<G>(lane);
     float* st = state + ((size_t)slots[seq] * H + h) * D * D;
     const float* recs = rec + ((size_t)first_block[seq] * H + h) * REC;
     const float* vals = proj + (size_t)t0 * ld + 2 * (size_t)I + (size_t)h * D + c0;
@@ -378,13 +374,13 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
             }
         }
     };
-    // a thread's rows: pairs of neighbours, four neighbours to a 16-byte piece, pieces G apart
+    // a thread's rows: pairs of neighbours, PF pairs to a piece, pieces G apart
     f2 S[C][R2];
 #pragma unroll
     for (int j = 0; j < C; ++j)
 #pragma unroll
         for (int i = 0; i < R2; ++i) {
-            const int d = ((i >> 1) * G + g) * 4 + (i & 1) * 2;
+            const int d = ((i / PF) * G + g) * PF * 2 + (i % PF) * 2;
             const bool in = c + j < D;
             S[j][i] = f2_pack(in && d < D ? st[(size_t)d * D + c + j] : 0.f, in && d + 1 < D ? st[(size_t)(d + 1) * D + c + j] : 0.f);
         }
@@ -395,9 +391,13 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
     }
     auto rows = [&](const float* row, f2 (&x)[R2]) {
 #pragma unroll
-        for (int i = 0; i < R2; i += 2) {
-            const ulonglong2 q = reinterpret_cast<const ulonglong2*>(row)[(i >> 1) * G + g];
-            x[i] = q.x; x[i + 1] = q.y;
+        for (int i = 0; i < R2; i += PF) {
+            if constexpr (PF == 2) {
+                const ulonglong2 q = reinterpret_cast<const ulonglong2*>(row)[(i >> 1) * G + g];
+                x[i] = q.x; x[i + 1] = q.y;
+            } else {
+                x[i] = reinterpret_cast<const f2*>(row)[i * G + g];
+            }
         }
     };
     auto dot = [&](const f2 (&x)[R2], const f2 (&y)[R2]) {
@@ -420,15 +420,15 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
         f2 x[R2];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            rows(s + i * DP, x);
+            rows(s + (i ^ e0) * DP, x);
 #pragma unroll
             for (int j = 0; j < C; ++j) y[j][i] = dot(x, S[j]);
         }
 #pragma unroll
-        for (int j = 0; j < C; ++j) lanes_sum8<G>(y[j], lane);
+        for (int j = 0; j < C; ++j) lanes_sum8<G>(y[j]);
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            rows(s + (8 + i) * DP, x);
+            rows(s + (8 + (i ^ e0)) * DP, x);
 #pragma unroll
             for (int j = 0; j < C; ++j) z[j][i] = dot(x, S[j]);
         }
@@ -437,7 +437,6 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
 #pragma unroll
             for (int j = 0; j < C; ++j) v[j][i] = vs[i * DVT + j];
         // this lane's tokens: p (its sum over the values of the tokens before it), later o
-        const int e0 = first_of<G>(lane);
 #pragma unroll
         for (int l = 0; l < LEFT; ++l) {
             const float4 m0 = *reinterpret_cast<const float4*>(mn + (e0 + l) * 8), m1 = *reinterpret_cast<const float4*>(mn + (e0 + l) * 8 + 4);
@@ -476,7 +475,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
             }
         }
 #pragma unroll
-        for (int j = 0; j < C; ++j) lanes_sum8<G>(z[j], lane);
+        for (int j = 0; j < C; ++j) lanes_sum8<G>(z[j]);
         if (G <= 8 || g < 8) {
 #pragma unroll
             for (int l = 0; l < LEFT; ++l) {
@@ -498,7 +497,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
     for (int j = 0; j < C; ++j)
 #pragma unroll
         for (int i = 0; i < R2; ++i) {
-            const int d = ((i >> 1) * G + g) * 4 + (i & 1) * 2;
+            const int d = ((i / PF) * G + g) * PF * 2 + (i % PF) * 2;
             float a, b;
             f2_split(S[j][i], a, b);
             if (c + j < D && d < D) st[(size_t)d * D + c + j] = a;
@@ -535,22 +534,18 @@ ACV_API int acv_delta(const float* rec, const float* proj, int ld, float* state,
     if (D <= 8) DL_CASE(8, 1, 1, 1, 3)
     if (D <= 16) DL_CASE(8, 2, 1, 1, 3)
     if (D <= 32) DL_CASE(8, 4, 1, 4, 3)
+    // few columns for the device: four warps to sixteen columns; more: two warps, then one (fewer instructions a column)
+    const long long tiles = (long long)n_seqs * H * ((D + 15) / 16);
     if (D <= 64) {
-        if (form == 1) DL_CASE(8, 8, 1, 4, 3)
-        if (form == 2) DL_CASE(8, 8, 2, 2, 3)
-        if (form == 3) DL_CASE(8, 8, 4, 2, 3)
-        if (form == 4) DL_CASE(4, 16, 2, 4, 3)
-        if (form == 5) DL_CASE(8, 8, 2, 4, 3)
-        if (form == 6) DL_CASE(4, 16, 4, 2, 3)
-        if (form == 7) DL_CASE(8, 8, 4, 1, 3)
-        if (form == 8) DL_CASE(4, 16, 4, 4, 3)
-        DL_CASE(8, 8, 2, 2, 3)
+        if (!form) form = tiles <= 180 ? 1 : tiles <= 600 ? 2 : 3;
+        if (form == 1) DL_CASE(4, 16, 2, 4, 3)
+        if (form == 2) DL_CASE(4, 16, 4, 2, 3)
+        DL_CASE(8, 8, 4, 1, 3)
     }
     if (D <= 128) {
-        if (form == 1) DL_CASE(8, 16, 1, 4, 3)
-        if (form == 2) DL_CASE(8, 16, 4, 2, 3)
-        if (form == 3) DL_CASE(4, 32, 4, 4, 3)
-        DL_CASE(8, 16, 2, 4, 3)
+        if (!form) form = tiles <= 600 ? 1 : 2;
+        if (form == 1) DL_CASE(8, 16, 2, 4, 3)
+        DL_CASE(8, 16, 4, 2, 3)
     }
     if (D <= 256) DL_CASE(8, 32, 1, 4, 3)
     DL_CASE(16, 32, 1, 4, 2)

@@ -315,12 +315,77 @@ __global__ void retention_gate_kernel(const float* __restrict__ o, int ldo, cons
     }
 }
 
+// The same with four neighbouring elements to a thread: a head of 4 n elements (n a power of two up to 32) is n
+// neighbouring lanes of a warp, so a warp takes 32 / n heads of a token at a time.
+__device__ __forceinline__ float4 gate_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 gate_ld4(const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void gate_st4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void gate_st4(bf16* p, const float (&v)[4]) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&lo);
+    u.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = u;
+}
+template <typename TG, typename T>
+__global__ void __launch_bounds__(256)
+retention_gate4_kernel(const float* __restrict__ o, int ldo, const TG* __restrict__ gate, int ldg, T* __restrict__ out, int ld_out,
+                       int width, int group, const float* __restrict__ w, int gate_kind, float eps, float out_scale,
+                       int T_tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int per_row = width >> 2, lanes = group >> 2;
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const int t = (int)(i / per_row), e = (int)(i - (long long)t * per_row) << 2;
+    const bool in = t < T_tokens;           // (whole heads are in or out: the exchanges stay among lanes of one head)
+    const float4 x = in ? gate_ld4(o + (size_t)t * ldo + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 z = in ? gate_ld4(gate + (size_t)t * ldg + e) : x;
+    float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
+    for (int s = 1; s < lanes; s <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+    if (!in) return;
+    const float inv = out_scale / sqrtf(ss / (float)group + eps);
+    const float4 wv = w ? *reinterpret_cast<const float4*>(w + e) : make_float4(1.f, 1.f, 1.f, 1.f);
+    const float xs[4] = {x.x * wv.x, x.y * wv.y, x.z * wv.z, x.w * wv.w}, zs[4] = {z.x, z.y, z.z, z.w};
+    float v[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float sg = 1.f / (1.f + expf(-zs[j]));
+        v[j] = xs[j] * inv * (gate_kind == 1 ? sg : zs[j] * sg);
+    }
+    gate_st4(out + (size_t)t * ld_out + e, v);
+}
+
 ACV_API int acv_retention_gate(const float* o, int ldo, const void* gate, int ldg, void* out, int ld_out, int T_tokens,
                                int H, int DV, float eps, float out_scale, int dtype, const float* weight, int joint,
                                int gate_kind, int gate_dtype, cudaStream_t stream) {
     if (T_tokens <= 0) return 0;
     const int warps = 8;
     const int groups = joint ? 1 : H, group = joint ? H * DV : DV;
+    // whole heads in 16-byte pieces (8 bytes of bfloat16): the vector form
+    const int lanes = group / 4;
+    auto pieces = [](const void* p, int ld, int dt) { return !((uintptr_t)p & (dt == ACV_F32 ? 15 : 7)) && ld % 4 == 0; };
+    if (group % 4 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 && pieces(o, ldo, ACV_F32) && pieces(gate, ldg, gate_dtype) &&
+        pieces(out, ld_out, dtype) && (!weight || !((uintptr_t)weight & 15)) && (gate_dtype == dtype || gate_dtype == ACV_F32)) {
+        const int width = groups * group;
+        const long long threads = (long long)T_tokens * (width / 4);
+        const int g4 = (int)((threads + 255) / 256);
+        if (dtype == ACV_F32)
+            acv_launch(PDL_MISC, retention_gate4_kernel<float, float>, g4, 256, 0, stream, o, ldo, (const float*)gate, ldg,
+                       (float*)out, ld_out, width, group, weight, gate_kind, eps, out_scale, T_tokens);
+        else if (dtype == ACV_BF16 && gate_dtype == ACV_F32)
+            acv_launch(PDL_MISC, retention_gate4_kernel<float, bf16>, g4, 256, 0, stream, o, ldo, (const float*)gate, ldg,
+                       (bf16*)out, ld_out, width, group, weight, gate_kind, eps, out_scale, T_tokens);
+        else if (dtype == ACV_BF16)
+            acv_launch(PDL_MISC, retention_gate4_kernel<bf16, bf16>, g4, 256, 0, stream, o, ldo, (const bf16*)gate, ldg,
+                       (bf16*)out, ld_out, width, group, weight, gate_kind, eps, out_scale, T_tokens);
+        else
+            return ACV_ERR_DTYPE;
+        return acv_launch_status();
+    }
     const int grid = (T_tokens * groups + warps - 1) / warps;
     if (dtype == ACV_F32 && gate_dtype == ACV_F32)
         acv_launch(PDL_MISC, retention_gate_kernel<float, float>, grid, warps * 32, 0, stream, o, ldo, (const float*)gate, ldg,
