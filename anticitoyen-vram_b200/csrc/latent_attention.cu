@@ -38,7 +38,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* 
                                       const float* __restrict__ cos_sin, int rot, int table_rows,
                                       const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                                       const int* __restrict__ block_table, int bt_stride, const int* __restrict__ bt_rows,
-                                      T* __restrict__ pages, int page_size, int num_pages, int H, int D, int R, int KR, int halves) {
+                                      T* __restrict__ pages, int page_size, int num_pages, int H, int D, int R, int KR, int halves, int full) {
     extern __shared__ float sm[];           // [KR + R] the kv row, then [H * R] the heads' rotated parts
     __shared__ float red[32];
     pdl_launch_dependents();
@@ -64,7 +64,15 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* 
     }
     ss = block_sum(ss, red);                // (meets the block: row and qr are whole)
     const float inv = 1.f / sqrtf(ss / (float)KR + eps);
-    for (int i = tid; i < H * R; i += nthr) {
+    if (full) {         // whole heads [plain | rotated | zeros] of `full` elements
+        for (int i = tid; i < H * full; i += nthr) {
+            const int h = i / full, e = i - h * full;
+            float v = 0.f;
+            if (e < D) v = to_f32(q[(size_t)t * q_stride + (size_t)h * (D + R) + e]);
+            else if (e < D + R) v = rot_pairs(qr + h * R, e - D, rot, cs, halves);
+            q_out[(size_t)t * qo_stride + i] = from_f32<T>(v);
+        }
+    } else for (int i = tid; i < H * R; i += nthr) {
         const int h = i / R, e = i - h * R;
         q_out[(size_t)t * qo_stride + (size_t)h * (KR + R) + KR + e] = from_f32<T>(rot_pairs(qr + h * R, e, rot, cs, halves));
     }
@@ -79,13 +87,14 @@ __global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* 
 
 // q: rows of H*(D+R) at q_stride; q_out: rows of H*(KR+R) at qo_stride; kv: rows of KR+R at kv_stride; w float [KR];
 // cos_sin float [table_rows][rot]; pages [num_pages][1][page_size][KR+R] (null: nothing is kept, queries only).
+// full > 0: q_out is rows of H heads of `full` elements, [plain | rotated | zeros] (queries for keys that are written out).
 ACV_API int acv_latent_prepare(const void* q, int q_stride, void* q_out, int qo_stride, const void* kv, int kv_stride,
                                const float* w, float eps, const float* cos_sin, int rot, int table_rows,
                                const int* positions, const int* seq_of_token, const int* block_table, int bt_stride,
                                const int* bt_rows, void* pages, int page_size, int num_pages, int T_tokens, int H, int D,
-                               int R, int KR, int dtype, int halves, cudaStream_t stream) {
+                               int R, int KR, int dtype, int halves, int full, cudaStream_t stream) {
     if (T_tokens <= 0) return 0;
-    if (H <= 0 || D < 0 || R <= 0 || KR <= 0 || rot < 0 || rot > R || (rot & 1) || (rot && (!cos_sin || table_rows <= 0)))
+    if (H <= 0 || D < 0 || R <= 0 || KR <= 0 || rot < 0 || rot > R || (rot & 1) || (full && full < D + R) || (rot && (!cos_sin || table_rows <= 0)))
         return ACV_ERR_SIZE;
     const size_t smem = (size_t)(KR + R + H * R) * sizeof(float);
     if (smem > 200 * 1024) return ACV_ERR_SIZE;
@@ -99,7 +108,7 @@ ACV_API int acv_latent_prepare(const void* q, int q_stride, void* q_out, int qo_
         }                                                                                                               \
         acv_launch(PDL_ROPE, latent_prepare_kernel<T>, T_tokens, threads, smem, stream, (const T*)q, q_stride, (T*)q_out, \
                    qo_stride, (const T*)kv, kv_stride, w, eps, cos_sin, rot, table_rows, positions, seq_of_token,       \
-                   block_table, bt_stride, bt_rows, (T*)pages, page_size, num_pages, H, D, R, KR, halves);                      \
+                   block_table, bt_stride, bt_rows, (T*)pages, page_size, num_pages, H, D, R, KR, halves, full);                      \
     } while (0)
     if (dtype == ACV_F32) LP_LAUNCH(float);
     else if (dtype == ACV_BF16) LP_LAUNCH(bf16);

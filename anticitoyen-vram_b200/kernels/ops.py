@@ -107,7 +107,11 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_cast_rows_f32": [P, I, P, I, I, I, I, P],
         "acv_activation": [P, P, LL, I, F, F, I, P],
         "acv_rmsnorm_rows": [P, I, P, F, P, I, I, I, I, P],
-        "acv_latent_prepare": [P, I, P, I, P, I, P, F, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, P],
+        "acv_latent_prepare": [P, I, P, I, P, I, P, F, P, I, I, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, P],
+        "acv_latent_context": [P, P, P, P, P, I, P, P, I, I, I, I, P],
+        "acv_latent_pack": [P, I, P, I, P, P, I, I, I, I, I, I, I, P],
+        "acv_latent_pick": [P, I, P, P, P, I, I, I, I, I, P],
+        "acv_heads_gated": [P, I, P, I, P, P, I, I, I, I, P],
         "acv_attention_latent_tc_takes": [I, I, I],
         "acv_attention_latent_tc": [P, I, P, I, P, P, P, I, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, P, P, P, P],
         "acv_gemm_tc_qkv": [P, I, P, I, P, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, I, I, I, P, P, F, P, I, P, P, P, I, P, P, P, I, I, P],
@@ -1700,12 +1704,12 @@ def gemm_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torc
 def latent_prepare(q: torch.Tensor, q_out: torch.Tensor, kv: torch.Tensor | None, weight: torch.Tensor | None, eps: float,
                    cos_sin: torch.Tensor | None, positions: torch.Tensor, seq_of_token: torch.Tensor,
                    block_table: torch.Tensor | None, pages: torch.Tensor | None, num_heads: int, dim: int, rot_dim: int,
-                   rank: int, table_rows: torch.Tensor | None = None, rotate_half: bool = False) -> None:
+                   rank: int, table_rows: torch.Tensor | None = None, rotate_half: bool = False, whole: int = 0) -> None:
     """The kept row of every token, [normed latent | rotated shared key part], into its page, and every head's rotated
     query part into ``q_out[:, h, rank:]`` (csrc/latent_attention.cu).  q: [T, heads*(dim+rot_dim)]; q_out:
     [T, heads*(rank+rot_dim)]; kv: [T, rank+rot_dim], or None for a layer that reads rows kept by another one (queries
     only); pages [num_pages, 1, page_size, rank+rot_dim] or None.  Rotated pairs are (2i, 2i+1), with ``rotate_half``
-    (i, i + rot/2)."""
+    (i, i + rot/2).  ``whole`` > 0: q_out gets whole heads of that many elements instead, [plain | rotated | zeros]."""
     _need_cuda(q, q_out)
     if q.stride(1) != 1 or q_out.stride(1) != 1 or q_out.dtype != q.dtype or (kv is not None and (kv.stride(1) != 1 or q.dtype != kv.dtype)):
         raise KernelError("latent_prepare: q, q_out and kv have dense rows and one type")
@@ -1716,7 +1720,7 @@ def latent_prepare(q: torch.Tensor, q_out: torch.Tensor, kv: torch.Tensor | None
         cos_sin.shape[0] if cos_sin is not None else 0, _p(positions), _p(seq_of_token), _p(block_table),
         block_table.stride(0) if block_table is not None else 0, _p(table_rows), _p(pages),
         pages.shape[2] if pages is not None else 1, pages.shape[0] if pages is not None else 0, q.shape[0], num_heads, dim,
-        rot_dim, rank, dtype_code(q.dtype), 1 if rotate_half else 0, _stream()), "latent_prepare")
+        rot_dim, rank, dtype_code(q.dtype), 1 if rotate_half else 0, int(whole), _stream()), "latent_prepare")
 
 
 def attention_latent_tc_takes(dtype: torch.dtype, num_heads: int, row: int, rank: int) -> bool:
@@ -1759,6 +1763,86 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ct
         return out
     return attention_generic(q, out, pages, pages, ctx.positions, ctx.seq_of_token, block_table, num_heads, 1, row, scale,
                              window, table_rows=rows, value_dim=rank, sinks=sinks)
+
+
+LATENT_PAGE = 128               # tokens of a page of written-out keys and values (csrc/latent_expand.cu)
+LATENT_EXPAND_QUERIES = 32      # queries a context row must meet on average for its keys and values to be written out
+LATENT_EXPAND_ROWS = 1 << 17    # most context rows that a step writes out
+
+
+def latent_context_work(q_lens, kv_lens) -> tuple[dict, dict]:
+    """Which contexts a step with portions of prompts writes out as keys and values: those of all its portions (requests
+    with more than one token), if their rows meet enough queries; ``n_pages`` 0: none.  Arrays: request and number of
+    every page of ``LATENT_PAGE`` tokens; a block table over those pages (``width`` columns, one row a request of the
+    step); 0 .. one-token requests - 1."""
+    import numpy as np
+    portions = [i for i, q in enumerate(q_lens) if q > 1]
+    rows = sum(int(kv_lens[i]) for i in portions)
+    pairs = sum(int(q_lens[i]) * (2 * int(kv_lens[i]) - int(q_lens[i]) + 1) // 2 for i in portions)
+    empty = np.zeros(0, np.int32)
+    if not portions or rows > LATENT_EXPAND_ROWS or pairs < LATENT_EXPAND_QUERIES * rows:
+        return {"page_seq": empty, "page_idx": empty, "table": empty, "order": empty}, {"n_pages": 0, "width": 0}
+    n = [-(-int(kv_lens[i]) // LATENT_PAGE) for i in portions]
+    width = max(n)
+    table = np.full((len(q_lens), width), -1, np.int32)
+    at = 0
+    for i, k in zip(portions, n):
+        table[i, :k] = np.arange(at, at + k)
+        at += k
+    return ({"page_seq": np.repeat(np.asarray(portions, np.int32), n), "page_idx": np.concatenate([np.arange(k, dtype=np.int32) for k in n]),
+             "table": table.reshape(-1), "order": np.arange(len(q_lens) - len(portions), dtype=np.int32)},
+            {"n_pages": at, "width": width})
+
+
+def latent_context(pages: torch.Tensor, ctx, block_table: torch.Tensor, work: dict, row: int) -> torch.Tensor:
+    """The kept rows of the step's written-out contexts, [n_pages * 128, row], zeros behind a request's last token."""
+    _need_cuda(pages)
+    if pages.dtype != torch.bfloat16 or not pages.is_contiguous() or pages.shape[3] != row:
+        raise KernelError("latent_context: contiguous bfloat16 pages of kept rows are wanted")
+    out = torch.empty((work["n_pages"] * LATENT_PAGE, row), device=pages.device, dtype=pages.dtype)
+    _check(library().acv_latent_context(_p(pages), _p(work["page_seq"]), _p(work["page_idx"]), _p(ctx.kv_len), _p(block_table),
+                                        block_table.stride(0), _p(getattr(ctx, "table_rows", None)), _p(out), work["n_pages"], row,
+                                        pages.shape[2], pages.shape[0], _stream()), "latent_context")
+    return out
+
+
+def latent_pack(kv: torch.Tensor, rows: torch.Tensor, num_heads: int, dim: int, rot_dim: int, value_dim: int, rank: int,
+                head: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """(key pages, value pages) [n_pages, heads, 128, head]: keys [kv's plain part | the row's rotated part | zeros], values
+    [kv's | zeros]; kv [n_pages * 128, heads * (dim + value_dim)], rows [n_pages * 128, rank + rot_dim]."""
+    _need_cuda(kv, rows)
+    if kv.dtype != torch.bfloat16 or rows.dtype != torch.bfloat16 or kv.stride(1) != 1 or not rows.is_contiguous() or len(rows) % LATENT_PAGE:
+        raise KernelError("latent_pack: bfloat16 products and kept rows in whole pages are wanted")
+    n = len(rows) // LATENT_PAGE
+    k, v = (torch.empty((n, num_heads, LATENT_PAGE, head), device=kv.device, dtype=kv.dtype) for _ in range(2))
+    _check(library().acv_latent_pack(_p(kv), kv.stride(0), _p(rows), rows.shape[1], _p(k), _p(v), n, num_heads, dim, rot_dim,
+                                     value_dim, rank, head, _stream()), "latent_pack")
+    return k, v
+
+
+def latent_pick(q: torch.Tensor, head: int, rows: torch.Tensor, n: int, met: torch.Tensor, num_heads: int, dim: int, rot_dim: int,
+                rank: int) -> torch.Tensor:
+    """Of the listed rows of q ([T, heads * head], heads [plain | rotated | ...]): the plain parts [n, heads, dim] (returned), the
+    rotated parts into ``met`` [n, heads * (rank + rot_dim)] behind the latent part's place."""
+    _need_cuda(q, met)
+    out = torch.empty((n, num_heads, dim), device=q.device, dtype=q.dtype)
+    if q.dtype != torch.bfloat16 or not q.is_contiguous() or not met.is_contiguous() or met.dtype != q.dtype:
+        raise KernelError("latent_pick: contiguous bfloat16 queries are wanted")
+    _check(library().acv_latent_pick(_p(q), head, _p(rows), _p(out), _p(met), n, num_heads, dim, rot_dim, rank, _stream()), "latent_pick")
+    return out
+
+
+def heads_gated(x: torch.Tensor, head: int, gate: torch.Tensor | None, rows: torch.Tensor | None, out: torch.Tensor,
+                num_heads: int, value_dim: int) -> torch.Tensor:
+    """out[rows[i]] = the first ``value_dim`` elements of x's heads (x [n, heads * head]), times sigmoid(gate[rows[i]]) if
+    there is a gate (a view like out); ``rows`` None: row i."""
+    _need_cuda(x, out)
+    if x.dtype != torch.bfloat16 or not x.is_contiguous() or out.dtype != x.dtype or out.stride(1) != 1 or \
+            (gate is not None and (gate.dtype != x.dtype or gate.stride(1) != 1)):
+        raise KernelError("heads_gated: bfloat16 heads, gate and output with dense rows are wanted")
+    _check(library().acv_heads_gated(_p(x), head, _p(gate), gate.stride(0) if gate is not None else 0, _p(rows), _p(out),
+                                     out.stride(0), x.shape[0], num_heads, value_dim, _stream()), "heads_gated")
+    return out
 
 
 def rmsnorm_rows(x: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor) -> torch.Tensor:

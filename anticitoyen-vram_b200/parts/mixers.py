@@ -568,10 +568,29 @@ class LatentAttention(Mixer):
     (csrc/latent_attention.cu): the query that meets the kept rows is [W_uk,h^T q_plain | q_rot], and the weighted sum
     of latents is projected by W_uv,h afterwards; both are one batched product over the heads.
 
+    In bfloat16 steps whose portions of prompts bring enough queries for a context row, the portions' keys and values are
+    written out instead (csrc/latent_expand.cu) and the tensor-core attention for portions runs over them, a key/value
+    head for every query head; one-token requests of the same step go on over the kept rows.
+
     Tensors behind ``prefix``: dq, dq.norm, uq, dkv, dkv.norm, uk, uv, o (``names`` renames them); no biases."""
 
     NAMES = {n: n for n in ("dq", "dq.norm", "uq", "dkv", "dkv.norm", "uk", "uv", "o")}
     metadata_key = "attention"      # the work lists of the attention kernels serve this layer as well
+    EXPAND = "latent_context"       # and, for portions of prompts, which contexts to write out
+
+    class _Context:
+        """Provider of the step's list of written-out contexts."""
+
+        @staticmethod
+        def step_metadata(q_lens, kv_lens, cu_q) -> StepMetadata:
+            return StepMetadata(*ops.latent_context_work(q_lens, kv_lens))
+
+        @staticmethod
+        def decode_metadata(padded: int, max_kv: int) -> StepMetadata:
+            return StepMetadata(*ops.latent_context_work([1] * padded, [1] * padded))
+
+    def metadata_providers(self) -> dict:
+        return {self.metadata_key: self, self.EXPAND: self._Context()}
 
     def step_metadata(self, q_lens, kv_lens, cu_q) -> StepMetadata:
         return StepMetadata(*ops.attention_work(q_lens, kv_lens, cu_q))
@@ -642,6 +661,10 @@ class LatentAttention(Mixer):
         # per head: W_uk,h^T as the weight [rank, dim] of q_plain -> latent space; W_uv,h [value_dim, rank] as it is
         self.uk_t = w("uk").view(H, D, KR).transpose(1, 2).contiguous()
         self.uv = w("uv").view(H, DV, KR).contiguous()
+        # keys and values written out: heads of 64 or 128 elements (padded with zeros)
+        wide = max(D + self.rot_dim, DV)
+        self.head = (64 if wide <= 64 else 128) if rt.dtype == torch.bfloat16 and wide <= 128 else 0
+        self.ukv = Linear.stacked([w("uk"), w("uv")]) if self.head else None
         self.position.load({}, rt)
         if self.position.rotary_table() is None:
             raise ValueError("latent_attention takes a position encoding that offers a rotary table")
@@ -683,6 +706,12 @@ class LatentAttention(Mixer):
         cq = torch.empty((T, self.q_rank), device=h.device, dtype=h.dtype)
         ops.rmsnorm_rows(down[:, :self.q_rank], self.q_norm, self.norm_eps, cq)
         q = self.uq(cq)                                         # [T, H, dim + rot_dim]
+        gate = down[:, gate_at:gate_at + self.inner_size] if self.gate is not None else None
+        expand = ctx.work.get(self.EXPAND)
+        if self.head and expand is not None and expand["n_pages"] and (
+                not ctx.work[self.metadata_key]["n_dec"] or ops.attention_latent_tc_takes(h.dtype, H, self.row, KR)):
+            self._written_out(q, down[:, kv_at:kv_at + self.row] if self.own_kv else None, gate, ctx, cache, table, expand, out)
+            return
         met = torch.empty((T, H * self.row), device=h.device, dtype=h.dtype)      # the queries that meet the kept rows
         ops.latent_prepare(q, met, down[:, kv_at:kv_at + self.row] if self.own_kv else None, self.kv_norm, self.norm_eps,
                            self.position.rotary_table(), ctx.positions, ctx.seq_of_token, table if self.own_kv else None,
@@ -692,8 +721,36 @@ class LatentAttention(Mixer):
         lat = torch.empty((T, H * KR), device=h.device, dtype=h.dtype)            # weighted sums of latents
         ops.attention_latent(met, lat, cache.k_pages, ctx, table, H, self.row, KR, self.scale, self.window,
                              work=ctx.work.get(self.metadata_key), sinks=self.sinks)
-        gate = down[:, gate_at:gate_at + self.inner_size].unflatten(1, (H, DV)) if self.gate is not None else None
-        ops.gemm_batched(lat.view(T, H, KR), self.uv, out.unflatten(1, (H, DV)), gate=gate)
+        ops.gemm_batched(lat.view(T, H, KR), self.uv, out.unflatten(1, (H, DV)),
+                         gate=gate.unflatten(1, (H, DV)) if gate is not None else None)
+
+    def _written_out(self, q, kv, gate, ctx, cache: CacheView, table, expand, out) -> None:
+        """The same from the queries on, for a step whose portions' contexts are written out as keys and values."""
+        H, D, R, DV, KR, HD = self.num_heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank, self.head
+        T, dev, work = q.shape[0], q.device, ctx.work[self.metadata_key]
+        qx = torch.empty((T, H * HD), device=dev, dtype=q.dtype)         # whole queries, a head padded to HD
+        ops.latent_prepare(q, qx, kv, self.kv_norm, self.norm_eps, self.position.rotary_table(), ctx.positions, ctx.seq_of_token,
+                           table if self.own_kv else None, cache.k_pages if self.own_kv else None, H, D, R, KR,
+                           table_rows=ctx.table_rows, rotate_half=self.rotate_half, whole=HD)
+        rows = ops.latent_context(cache.k_pages, ctx, table, expand, self.row)
+        keys, values = ops.latent_pack(self.ukv(rows[:, :KR]), rows, H, D, R, DV, KR, HD)
+        direct = gate is None and HD == DV and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+        o = out if direct else torch.empty((T, H * HD), device=dev, dtype=q.dtype)
+        ops.attention_tc(qx, o, keys, values, work["tile_seq"], work["tile_q0"], work["n_tiles"], ctx.cu_q, ctx.kv_len,
+                         expand["table"].view(-1, expand["width"]), H, H, HD, self.scale, self.window, sinks=self.sinks)
+        if not direct:
+            ops.heads_gated(o, HD, gate, None, out, H, DV)
+        n = work["n_dec"]
+        if n:       # one-token requests of the step, over the kept rows
+            met = torch.empty((n, H * self.row), device=dev, dtype=q.dtype)
+            plain = ops.latent_pick(qx, HD, work["dec_tokens"], n, met, H, D, R, KR)
+            ops.gemm_batched(plain, self.uk_t, met.view(n, H, self.row)[:, :, :KR])
+            lat = torch.empty((n, H * KR), device=dev, dtype=q.dtype)
+            ops.attention_latent(met, lat, cache.k_pages, ctx, table, H, self.row, KR, self.scale, self.window,
+                                 work={**work, "dec_tokens": expand["order"], "n_tiles": 0}, sinks=self.sinks)
+            heads = torch.empty((n, H * DV), device=dev, dtype=q.dtype)
+            ops.gemm_batched(lat.view(n, H, KR), self.uv, heads.view(n, H, DV))
+            ops.heads_gated(heads, DV, gate, work["dec_tokens"], out, H, DV)
 
     def forward(self, h, ctx, cache: CacheView):
         out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
