@@ -614,6 +614,7 @@ class LatentAttention(Mixer):
         self.names = {**self.NAMES, **(names or {})}
         self.position = build("position", position, hidden_size)
         self.row = kv_rank + rot_dim            # elements of a kept row, and of a query that meets it
+        self.head = 0                           # size of a written-out head (0: none are written out), known when loaded
         self.inner_size = num_heads * value_dim # columns in front of the output projection
 
     def _n(self, role: str) -> str:
@@ -687,8 +688,17 @@ class LatentAttention(Mixer):
         return float(sum(min(self.window, p + 1) for p in range(kv - q, kv)))
 
     def mixing_flops(self, q_lens, kv_lens) -> float:
-        # scores over the kept rows, weighted sums over their latents
-        return 2.0 * self.num_heads * (self.row + self.kv_rank) * sum(self._seen(q, kv) for q, kv in zip(q_lens, kv_lens))
+        # scores over the kept rows, weighted sums over their latents; where keys and values are written out: scores and sums
+        # over those, and the products that write out what the portion's own tokens (counted in ``flops``) do not
+        H, out = self.num_heads, 0.0
+        written = self.head and ops.latent_context_work(q_lens, kv_lens)[1]["n_pages"] > 0
+        for q, kv in zip(q_lens, kv_lens):
+            if written and q > 1:
+                out += 2.0 * H * (self.dim + self.rot_dim + self.value_dim) * self._seen(q, kv)
+                out += 2.0 * H * (kv - q) * self.kv_rank * (self.dim + self.value_dim)
+            else:
+                out += 2.0 * H * (self.row + self.kv_rank) * self._seen(q, kv)
+        return out
 
     def cache_bytes_read(self, q_lens, kv_lens, itemsize: int) -> int:
         keys = sum(min(kv, self.window + q - 1) if self.window > 0 else kv for q, kv in zip(q_lens, kv_lens))
