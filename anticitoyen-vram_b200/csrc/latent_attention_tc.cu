@@ -8,7 +8,7 @@
 // weights there as bfloat16; then each multiplies all BN weights with its own slice of NDV*16 value columns.  So no
 // score is computed twice, and the accumulators of a row (KR floats) are spread over S warps.
 //
-//   barrier A   tile t has arrived (cp.async), and everyone is done with tile t-1: fetch tile t+1 into the other buffer
+//   barrier A   tile t has arrived, and everyone is done with tile t-1: fetch the tile NB - 1 further on into its buffer
 //   scores      q . k over ROW, * scale * log2(e), masked (causal, window)
 //   barrier B   row maxima of the S warps are there (S > 1)
 //   weights     p = 2^(s - m); running maximum and sum; accumulators rescaled; p into shared memory
@@ -18,9 +18,12 @@
 // One token with 16 heads is one row group (the decode step's shape); a portion takes as many tokens as 16 warps and
 // the shared memory hold.  Rows are padded by 16 bytes instead of swizzled, so ROW and KR need only be multiples of 8.
 #include "mma_tiles.cuh"
+#include "tc_ptx.cuh"
 
 #define LT_LOG2E 1.4426950408889634f
 #define LT_TILE_TOKENS 128      // query tokens in a tile of the step's work list
+#define LT_MAX_BUFFERS 4
+#define LT_STATUS 21            // a wait for kept rows ran out
 
 struct LatentArgs {
     const bf16* q; int q_stride; bf16* out; int out_stride;
@@ -34,6 +37,8 @@ struct LatentArgs {
     int TOK;                // query tokens of a unit (divides 16)
     int HPC, HB;            // heads of a CTA, head blocks (HPC * HB == NH)
     int RG;                 // row groups of a CTA = ceil(TOK * HPC / 16)
+    int NB;                 // buffers of key tiles (2..LT_MAX_BUFFERS)
+    int* status;            // gets a code when a bounded wait for a tile runs out
     int n_split;            // CTAs that share the rows of a one-token request (1: none)
     float* part_acc;        // n_split > 1: [n_dec][n_split][NH][KR] unnormalised sums
     float* part_ml;         //              [n_dec][n_split][NH][2] running maximum (in powers of two) and sum
@@ -53,8 +58,10 @@ attn_latent_tc_kernel(const LatentArgs a) {
     constexpr int PP = (BN + 8) * 2;        // bytes of a row of weights
 
     unsigned char* q_s = smem;                                      // [RG * 16][QP]
-    unsigned char* k_s = q_s + (size_t)RG * 16 * QP;                // [2][BN][QP]
-    unsigned char* p_s = k_s + (size_t)2 * BN * QP;                 // [RG][16][PP]
+    unsigned char* k_s = q_s + (size_t)RG * 16 * QP;                // [NB][BN][QP]
+    unsigned char* p_s = k_s + (size_t)a.NB * BN * QP;              // [RG][16][PP]
+    __shared__ __align__(8) uint64_t full_s[LT_MAX_BUFFERS];
+    __shared__ int abort_s;
     float* mx_s = reinterpret_cast<float*>(p_s + (size_t)RG * 16 * PP);     // [RG][S][16]
     float* l_s = mx_s + (size_t)RG * S * 16;                        // [RG][S][16]
 
@@ -119,24 +126,49 @@ attn_latent_tc_kernel(const LatentArgs a) {
                                                 (size_t)(h_first + R % HPC) * ROW + c * 8);
         *reinterpret_cast<uint4*>(q_s + (size_t)R * QP + c * 16) = v;
     }
+    // A tile's rows: one bulk copy each, counted at the buffer's barrier, at which every thread arrives with the bytes of
+    // its own rows.  Rows that no query sees (or without a page) become zeros: their weights are zero, and nothing that is
+    // no number may stand beside them.
+    const uint32_t full0 = gt_smem(full_s);
+    if (DP > ROW)                                // a row's last 16 bytes, which no copy brings
+        for (int r = tid; r < a.NB * BN; r += nthr) *reinterpret_cast<uint4*>(k_s + (size_t)r * QP + ROW * 2) = make_uint4(0, 0, 0, 0);
+    if (tid == 0) {
+        abort_s = 0;
+        for (int i = 0; i < a.NB; ++i) mbar_init(full0 + 8 * i, nthr);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
     auto load_keys = [&](int t) {
-        const int j0 = j_first + t * BN;
-        unsigned char* dst = k_s + (size_t)(t & 1) * BN * QP;
-        for (int id = tid; id < BN * CH; id += nthr) {
-            const int c = id % CH, r = id / CH;
-            const int j = j0 + r;
-            bool ok = j <= hi && j >= lo && c * 8 < ROW;
-            size_t off = 0;
-            if (ok) {
-                const int pg = bt[j / a.page_size];
-                ok = pg >= 0 && pg < a.num_pages;
-                off = ((size_t)pg * a.page_size + (j % a.page_size)) * ROW + c * 8;
+        const int j0 = j_first + t * BN, buf = (t - t_first) % a.NB;
+        unsigned char* dst = k_s + (size_t)buf * BN * QP;
+        const uint32_t bar = full0 + 8 * buf;
+        auto page_of = [&](int j) {
+            if (j > hi || j < lo) return -1;
+            const int pg = bt[j / a.page_size];
+            return pg < a.num_pages ? pg : -1;
+        };
+        uint32_t bytes = 0;
+        bool zeroed = false;
+        for (int r = tid; r < BN; r += nthr) {
+            if (page_of(j0 + r) >= 0) {
+                bytes += ROW * 2;
+            } else {
+                for (int c = 0; c < ROW / 8; ++c) *reinterpret_cast<uint4*>(dst + (size_t)r * QP + c * 16) = make_uint4(0, 0, 0, 0);
+                zeroed = true;
             }
-            cp_async16(smem_u32(dst + (size_t)r * QP + c * 16), ok ? (const void*)(a.pages + off) : (const void*)a.pages, ok);
         }
+        if (zeroed) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");    // (this thread's copies may follow there)
+        mbar_expect_tx(bar, bytes);         // (arrives)
+        if (bytes)
+            for (int r = tid; r < BN; r += nthr) {
+                const int j = j0 + r, pg = page_of(j);
+                if (pg < 0) continue;
+                const bf16* src = a.pages + ((size_t)pg * a.page_size + (j % a.page_size)) * ROW;
+                asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                             ::"r"(smem_u32(dst + (size_t)r * QP)), "l"(src), "r"(ROW * 2), "r"(bar) : "memory");
+            }
     };
-    load_keys(t_first);
-    cp_async_commit();
+    for (int t = t_first; t < n_t && t < t_first + a.NB - 1; ++t) load_keys(t);
 
     const int mi = lane >> 3, lr = lane & 7;
     const int r_lo = lane >> 2, c_lo = (lane & 3) * 2;
@@ -158,11 +190,17 @@ attn_latent_tc_kernel(const LatentArgs a) {
 
     for (int t = t_first; t < n_t; ++t) {
         const int j0 = j_first + t * BN;
-        cp_async_wait<0>();
-        __syncthreads();                                            // A
-        if (t + 1 < n_t) load_keys(t + 1);
-        cp_async_commit();
-        const uint32_t kb = smem_u32(k_s + (size_t)(t & 1) * BN * QP);
+        const int turn = t - t_first;
+        const bool there = mbar_wait(full0 + 8 * (turn % a.NB), (turn / a.NB) & 1, &abort_s);
+        if (!__syncthreads_and(there)) {                            // A
+            if (tid == 0) atomicExch(a.status, LT_STATUS);
+            // the copies that are under way end before the block does (bounded again)
+            for (int u = t; u < n_t && u < t + a.NB - 1; ++u)
+                mbar_wait(full0 + 8 * ((u - t_first) % a.NB), ((u - t_first) / a.NB) & 1, &abort_s);
+            return;
+        }
+        if (t + a.NB - 1 < n_t) load_keys(t + a.NB - 1);
+        const uint32_t kb = smem_u32(k_s + (size_t)(turn % a.NB) * BN * QP);
         const int key0 = sl * KPW;
         float s[NT][4];
 #pragma unroll
@@ -258,7 +296,6 @@ attn_latent_tc_kernel(const LatentArgs a) {
             }
         }
     }
-    cp_async_wait<0>();
 
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
@@ -345,15 +382,15 @@ __global__ void attn_latent_merge_kernel(const float* __restrict__ part_acc, con
 }
 
 struct LatentShape {
-    int S, NDV, TOK, HPC, HB, RG, BN;
+    int S, NDV, TOK, HPC, HB, RG, BN, NB;
     size_t smem;
 };
 
 #define LT_SMEM_LIMIT (200 * 1024)
 
-static size_t latent_tc_smem(int ROW, int RG, int S, int BN) {
+static size_t latent_tc_smem(int ROW, int RG, int S, int BN, int NB) {
     const size_t QP = ((ROW + 15) & ~15) * 2 + 16, PP = (BN + 8) * 2;
-    return (size_t)RG * 16 * QP + (size_t)2 * BN * QP + (size_t)RG * 16 * PP + (size_t)2 * RG * S * 16 * 4;
+    return (size_t)RG * 16 * QP + (size_t)NB * BN * QP + (size_t)RG * 16 * PP + (size_t)2 * RG * S * 16 * 4;
 }
 
 // how a launch is cut for these sizes (portions: as many tokens a unit as fit; one-token requests alone: one); 0 if not at all
@@ -369,11 +406,13 @@ static int latent_tc_shape(int NH, int ROW, int KR, bool portions, LatentShape& 
     for (int tok = portions ? 16 : 1; tok >= 1; tok /= 2) {
         const int rg = (tok * sh.HPC + 15) / 16;
         if (rg > max_rg) continue;
-        for (int bn = 64; bn >= 32; bn /= 2) {
-            if (bn / sh.S < 8) continue;
-            const size_t smem = latent_tc_smem(ROW, rg, sh.S, bn);
+        // one-token requests wait for memory: small tiles, several on their way; portions for the tensor cores: large ones
+        static const int forms[2][4][2] = {{{32, 4}, {32, 3}, {64, 2}, {32, 2}}, {{64, 3}, {64, 2}, {32, 3}, {32, 2}}};
+        for (const auto& f : forms[portions]) {
+            if (f[0] / sh.S < 8) continue;
+            const size_t smem = latent_tc_smem(ROW, rg, sh.S, f[0], f[1]);
             if (smem <= LT_SMEM_LIMIT) {
-                sh.TOK = tok; sh.RG = rg; sh.BN = bn; sh.smem = smem;
+                sh.TOK = tok; sh.RG = rg; sh.BN = f[0]; sh.NB = f[1]; sh.smem = smem;
                 return 1;
             }
         }
@@ -408,7 +447,7 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
                                     const int* dec_seqs, int n_dec, const int* cu_q, const int* kv_len,
                                     const int* block_table, int bt_stride, const int* bt_rows, int NH, int ROW, int KR,
                                     int page_size, int num_pages, float scale, int window, int n_split, float* part_acc,
-                                    float* part_ml, const float* sinks, cudaStream_t stream) {
+                                    float* part_ml, const float* sinks, int* status, cudaStream_t stream) {
     if (n_split < 1 || (n_split > 1 && (!part_acc || !part_ml))) return ACV_ERR_SIZE;
     if (n_tiles < 0) n_tiles = 0;
     if (n_dec < 0) n_dec = 0;
@@ -419,7 +458,7 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
         return ACV_ERR_ALIGN;
     LatentArgs a = {(const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)pages, tile_seq, tile_q0, n_tiles,
                     dec_tokens, dec_seqs, n_dec, cu_q, kv_len, block_table, bt_stride, bt_rows, NH, ROW, KR, page_size,
-                    num_pages, scale, window, sh.TOK, sh.HPC, sh.HB, sh.RG, n_split, part_acc, part_ml, sinks};
+                    num_pages, scale, window, sh.TOK, sh.HPC, sh.HB, sh.RG, sh.NB, status, n_split, part_acc, part_ml, sinks};
 #define LT_CASE(B, SS, N) if (sh.BN == B && sh.S == SS && sh.NDV == N) return launch_latent_tc<B, SS, N>(a, sh, stream);
     LT_CASE(64, 1, 4) LT_CASE(64, 1, 8) LT_CASE(64, 2, 8) LT_CASE(64, 4, 8)
     LT_CASE(32, 1, 4) LT_CASE(32, 1, 8) LT_CASE(32, 2, 8) LT_CASE(32, 4, 8)

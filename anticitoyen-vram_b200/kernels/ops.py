@@ -113,7 +113,7 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_latent_pick": [P, I, P, P, P, I, I, I, I, I, P],
         "acv_heads_gated": [P, I, P, I, P, P, I, I, I, I, P],
         "acv_attention_latent_tc_takes": [I, I, I],
-        "acv_attention_latent_tc": [P, I, P, I, P, P, P, I, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, P, P, P, P],
+        "acv_attention_latent_tc": [P, I, P, I, P, P, P, I, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, P, P, P, P, P],
         "acv_gemm_tc_qkv": [P, I, P, I, P, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, I, I, I, P, P, F, P, I, P, P, P, I, P, P, P, I, I, P],
         "acv_gemm_tc": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P],
         "acv_gemm_tc_bias": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P, F, F, P],
@@ -1759,7 +1759,7 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ct
             _p(q), q.stride(0), _p(out), out.stride(0), _p(pages), _p(work["tile_seq"]), _p(work["tile_q0"]),
             work["n_tiles"], _p(work["dec_tokens"]), _p(work["dec_seqs"]), work["n_dec"], _p(ctx.cu_q), _p(ctx.kv_len),
             _p(block_table), block_table.stride(0), _p(rows), num_heads, row, rank, pages.shape[2], pages.shape[0],
-            float(scale), int(window), n_split, _p(acc), _p(ml), _p(sinks), _stream()), "attention_latent_tc")
+            float(scale), int(window), n_split, _p(acc), _p(ml), _p(sinks), _p(status_word(q.device)), _stream()), "attention_latent_tc")
         return out
     return attention_generic(q, out, pages, pages, ctx.positions, ctx.seq_of_token, block_table, num_heads, 1, row, scale,
                              window, table_rows=rows, value_dim=rank, sinks=sinks)
