@@ -381,6 +381,8 @@ __global__ void attn_latent_merge_kernel(const float* __restrict__ part_acc, con
     }
 }
 
+#include "latent_attention_dec.cuh"
+
 struct LatentShape {
     int S, NDV, TOK, HPC, HB, RG, BN, NB;
     size_t smem;
@@ -452,13 +454,31 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
     if (n_tiles < 0) n_tiles = 0;
     if (n_dec < 0) n_dec = 0;
     if (n_tiles == 0 && n_dec == 0) return 0;
-    LatentShape sh;
-    if (!latent_tc_shape(NH, ROW, KR, n_tiles > 0, sh)) return ACV_ERR_SIZE;
+    LatentShape sh = {};
+    // one-token requests have a kernel of their own where its sizes allow; portions beside them are then a launch of their own
+    const bool dec_own = n_dec > 0 && latent_dec_takes(ROW, KR);
+    if ((n_tiles > 0 || !dec_own) && !latent_tc_shape(NH, ROW, KR, n_tiles > 0, sh)) return ACV_ERR_SIZE;
     if (((uintptr_t)q & 15) || ((size_t)q_stride * 2) % 16 || ((uintptr_t)pages & 15) || ((uintptr_t)out & 3) || (out_stride & 1))
         return ACV_ERR_ALIGN;
     LatentArgs a = {(const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)pages, tile_seq, tile_q0, n_tiles,
                     dec_tokens, dec_seqs, n_dec, cu_q, kv_len, block_table, bt_stride, bt_rows, NH, ROW, KR, page_size,
                     num_pages, scale, window, sh.TOK, sh.HPC, sh.HB, sh.RG, sh.NB, status, n_split, part_acc, part_ml, sinks};
+    if (dec_own) {
+        LatentArgs d = a;
+        d.n_tiles = 0;
+        d.HB = (NH + 15) / 16;
+        int rc;
+        if (ROW <= 192 && KR <= 128) rc = launch_latent_dec<12, 1>(d, stream);
+        else if (ROW <= 320 && KR <= 256) rc = launch_latent_dec<20, 2>(d, stream);
+        else rc = launch_latent_dec<36, 4>(d, stream);
+        if (rc) return rc;
+        if (n_split > 1)
+            acv_launch(PDL_ATTN, attn_latent_merge_kernel, dim3(n_dec * NH), dim3(128), 0, stream, (const float*)part_acc,
+                       (const float*)part_ml, dec_tokens, a.out, out_stride, n_split, NH, KR, sinks);
+        if (n_tiles == 0) return acv_launch_status();
+        a.n_dec = 0;
+        a.n_split = 1;
+    }
 #define LT_CASE(B, SS, N) if (sh.BN == B && sh.S == SS && sh.NDV == N) return launch_latent_tc<B, SS, N>(a, sh, stream);
     LT_CASE(64, 1, 4) LT_CASE(64, 1, 8) LT_CASE(64, 2, 8) LT_CASE(64, 4, 8)
     LT_CASE(32, 1, 4) LT_CASE(32, 1, 8) LT_CASE(32, 2, 8) LT_CASE(32, 4, 8)

@@ -1746,12 +1746,12 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ct
     if work is not None and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and pages.is_contiguous() and \
             attention_latent_tc_takes(q.dtype, num_heads, row, rank):
         # a step of one-token requests alone: a CTA a request leaves SMs idle, so the rows of a request are shared among
-        # several (each at least MIXED_SPLIT_KEYS), and a second small launch merges their partial results
+        # several (each at least LATENT_SPLIT_KEYS), and a second small launch merges their partial results
         n_dec, n_split, acc, ml = work["n_dec"], 1, None, None
         if n_dec and not work["n_tiles"]:
             seen = min(work["max_dec_kv"], window) if window > 0 else work["max_dec_kv"]
-            room = max(1, sm_count(q.device) // (n_dec * ((num_heads + 63) // 64)))
-            n_split = max(1, min(room, seen // MIXED_SPLIT_KEYS, 16))
+            room = max(1, sm_count(q.device) // (n_dec * ((num_heads + 15) // 16)))
+            n_split = max(1, min(room, seen // LATENT_SPLIT_KEYS, 16))
             if n_split > 1:
                 parts = n_dec * n_split * num_heads
                 acc, ml, _ = _decode_scratch(q.device, parts * rank, parts * 2, 0)
@@ -1765,6 +1765,7 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ct
                              window, table_rows=rows, value_dim=rank, sinks=sinks)
 
 
+LATENT_SPLIT_KEYS = 128         # no share of a one-token request's kept rows is shorter than this
 LATENT_PAGE = 128               # tokens of a page of written-out keys and values (csrc/latent_expand.cu)
 LATENT_EXPAND_QUERIES = 32      # queries a context row must meet on average for its keys and values to be written out
 LATENT_EXPAND_ROWS = 1 << 17    # most context rows that a step writes out

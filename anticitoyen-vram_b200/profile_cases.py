@@ -486,6 +486,8 @@ CASES = {
     "latent_attention_prefill": lambda r: latent_attention_case(2048, 1, 2048, r),
     "latent_attention_prefill_small": lambda r: latent_attention_case(512, 1, 512, r, window=256),
     "latent_attention_decode_b64": lambda r: latent_attention_case(1, 64, 2048, r),
+    "latent_attention_decode_b64_full": lambda r: latent_attention_case(1, 64, 2048, r, window=0),
+    "latent_attention_decode_b8_full": lambda r: latent_attention_case(1, 8, 2048, r, window=0),
     "retention_prefill": lambda r: retention_case(2048, 1, r),
     "retention_decode_b64": lambda r: retention_case(1, 64, r),
     "delta_prefill": lambda r: delta_case(2048, 1, r),
