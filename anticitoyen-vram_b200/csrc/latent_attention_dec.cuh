@@ -1,8 +1,8 @@
 // One-token requests over kept latent rows (see latent_attention_tc.cu, whose arguments and merge they share).
 //
 // A CTA is one request (or a share of its rows) with up to 16 heads: the 16 rows of mma.sync m16n8k16.  Eight warps; the
-// queries' fragments stay in registers for the whole walk (NK steps of 16 elements), key tiles of 64 rows come by bulk
-// copies, two tiles ahead.  For a tile each warp makes the scores of eight keys (four chains of products), the warps
+// queries' fragments stay in registers for the whole walk (NK steps of 16 elements), key tiles of 64 rows come by TMA, two
+// tiles ahead: a box is 64 elements (one 128-byte swizzle row) of a page's rows, or of 64 of them.  For a tile each warp makes the scores of eight keys (four chains of products), the warps
 // exchange their row maxima and weights through shared memory, and each multiplies all 64 weights with its own
 // NDV * 16 value columns.
 #pragma once
@@ -10,19 +10,22 @@
 #define LD_BN 64
 #define LD_NB 3
 #define LD_THREADS 256
+#define LD_ATOM (LD_BN * 128)    // bytes of 64 elements of a tile's rows
 
-template <int NK, int NDV>
+// EXACT: rows of NK * 16 elements with latents of NDV * 128 (sizes known when compiled); otherwise up to that
+template <int NK, int NDV, bool EXACT>
 __global__ void __launch_bounds__(LD_THREADS, 1)
-attn_latent_dec_kernel(const LatentArgs a) {
-    extern __shared__ __align__(128) unsigned char smem[];
+attn_latent_dec_kernel(const __grid_constant__ CUtensorMap rows, const LatentArgs a) {
+    extern __shared__ unsigned char smem_raw[];
+    unsigned char* smem = smem_raw + ((1024u - (gt_smem(smem_raw) & 1023u)) & 1023u);
     __shared__ __align__(8) uint64_t full_s[LD_NB];
     __shared__ int abort_s;
-    const int ROW = a.ROW, KR = a.KR;
+    const int ROW = EXACT ? NK * 16 : a.ROW, KR = EXACT ? NDV * 128 : a.KR;
     const int DP = (ROW + 15) & ~15, KRP = (KR + 15) & ~15, nk = DP >> 4;
-    const int QP = DP * 2 + 16;                 // bytes of a padded row
+    const int NA = (ROW + 63) >> 6;             // 64-element pieces of a row
     constexpr int PP = (LD_BN + 8) * 2;
-    unsigned char* k_s = smem;                                      // [LD_NB][LD_BN][QP]
-    unsigned char* p_s = k_s + (size_t)LD_NB * LD_BN * QP;          // [16][PP]
+    unsigned char* k_s = smem;                                      // [LD_NB][NA][LD_BN][128 bytes, swizzled]
+    unsigned char* p_s = k_s + (size_t)LD_NB * NA * LD_ATOM;        // [16][PP]
     float* mx_s = reinterpret_cast<float*>(p_s + 16 * PP);          // [16][8]
     float* l_s = mx_s + 16 * 8;                                     // [16][8]
 
@@ -54,10 +57,9 @@ attn_latent_dec_kernel(const LatentArgs a) {
     const int t_first = split * per_split, n_t = min(n_all, t_first + per_split);
 
     const uint32_t full0 = gt_smem(full_s);
-    if (DP > ROW)                               // a row's last 16 bytes, which no copy brings
-        for (int r = tid; r < LD_NB * LD_BN; r += LD_THREADS) *reinterpret_cast<uint4*>(k_s + (size_t)r * QP + ROW * 2) = make_uint4(0, 0, 0, 0);
     // the queries wait in the last buffer until their fragments are read
-    unsigned char* q_s = k_s + (size_t)(LD_NB - 1) * LD_BN * QP;
+    const int QP = DP * 2 + 16;
+    unsigned char* q_s = k_s + (size_t)(LD_NB - 1) * NA * LD_ATOM;
     const int CH = DP / 8;
     for (int id = tid; id < 16 * CH; id += LD_THREADS) {
         const int c = id % CH, R = id / CH;
@@ -69,28 +71,29 @@ attn_latent_dec_kernel(const LatentArgs a) {
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");        // (copies follow where these writes are)
     if (tid == 0) {
         abort_s = 0;
-        for (int b = 0; b < LD_NB; ++b) mbar_init(full0 + 8 * b, LD_BN);
+        for (int b = 0; b < LD_NB; ++b) mbar_init(full0 + 8 * b, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
-    // a thread a row: a bulk copy counted at the buffer's barrier, or zeros where no query sees the row (or it has no page)
+    // Warp 0 loads: a lane a page of the tile (or 64 rows of one), looked up a tile earlier.  A page that is not there is a
+    // place outside the pool, which reads as zeros; rows behind the last token of a page hold older, finite numbers.
+    const int box = min(a.page_size, LD_BN), n_box = LD_BN / box;
+    auto row_of = [&](int t) {                  // the box's first row in the pool
+        const int j = j_first + t * LD_BN + lane * box;
+        if (warp || lane >= n_box || t >= n_t || j > pos || j + box <= lo) return -LD_BN;
+        const int pg = bt[j / a.page_size];
+        return pg >= 0 && pg < a.num_pages ? pg * a.page_size + j % a.page_size : -LD_BN;
+    };
+    int row = row_of(t_first);
     auto load_keys = [&](int t) {
-        if (tid >= LD_BN) return;
-        const int j = j_first + t * LD_BN + tid, buf = (t - t_first) % LD_NB;
-        unsigned char* dst = k_s + ((size_t)buf * LD_BN + tid) * QP;
-        const uint32_t bar = full0 + 8 * buf;
-        int pg = -1;
-        if (j <= pos && j >= lo) pg = bt[j / a.page_size];
-        if (pg >= 0 && pg < a.num_pages) {
-            const bf16* src = a.pages + ((size_t)pg * a.page_size + (j % a.page_size)) * ROW;
-            mbar_expect_tx(bar, ROW * 2);       // (arrives)
-            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                         ::"r"(smem_u32(dst)), "l"(src), "r"(ROW * 2), "r"(bar) : "memory");
-        } else {
-            for (int c = 0; c < ROW / 8; ++c) *reinterpret_cast<uint4*>(dst + c * 16) = make_uint4(0, 0, 0, 0);
-            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-            mbar_arrive(bar);
-        }
+        if (warp) return;
+        const int buf = (t - t_first) % LD_NB, next = row_of(t + 1);
+        const uint32_t dst = smem_u32(k_s) + buf * NA * LD_ATOM, bar = full0 + 8 * buf;
+        if (lane == 0) mbar_expect_tx(bar, NA * LD_ATOM);
+        __syncwarp();
+        if (lane < n_box)
+            for (int c = 0; c < NA; ++c) tma_load_2d(dst + c * LD_ATOM + lane * box * 128, &rows, bar, c * 64, row);
+        row = next;
     };
     for (int t = t_first; t < n_t && t < t_first + LD_NB - 1; ++t) load_keys(t);
 
@@ -99,7 +102,7 @@ attn_latent_dec_kernel(const LatentArgs a) {
     uint32_t qf[NK][4];
 #pragma unroll
     for (int kd = 0; kd < NK; ++kd) {
-        if (kd < nk) ldmatrix_x4(qf[kd], smem_u32(q_s) + ((mi & 1) * 8 + lr) * QP + (kd * 2 + (mi >> 1)) * 16);
+        if (EXACT || kd < nk) ldmatrix_x4(qf[kd], smem_u32(q_s) + ((mi & 1) * 8 + lr) * QP + (kd * 2 + (mi >> 1)) * 16);
         else qf[kd][0] = qf[kd][1] = qf[kd][2] = qf[kd][3] = 0u;
     }
     const float sc_log2 = a.scale * LT_LOG2E;
@@ -121,21 +124,21 @@ attn_latent_dec_kernel(const LatentArgs a) {
             return;
         }
         if (t + LD_NB - 1 < n_t) load_keys(t + LD_NB - 1);
-        const uint32_t kb = smem_u32(k_s + (size_t)buf * LD_BN * QP);
+        const uint32_t kb = smem_u32(k_s) + buf * NA * LD_ATOM;
         // scores of keys warp*8 .. +7: four chains
         float s4[4][4];
 #pragma unroll
         for (int c = 0; c < 4; ++c)
 #pragma unroll
             for (int e = 0; e < 4; ++e) s4[c][e] = 0.f;
-        const uint32_t krow = kb + (warp * 8 + lr) * QP + mi * 16;
+        const uint32_t krow = kb + (warp * 8 + lr) * 128, kx[2] = {(uint32_t)(mi ^ lr) << 4, (uint32_t)((4 + mi) ^ lr) << 4};
 #pragma unroll
         for (int k2 = 0; k2 < NK / 2; ++k2) {
-            if (2 * k2 < nk) {
+            if (EXACT || 2 * k2 < nk) {
                 uint32_t b[4];                  // eight keys, two steps of 16 elements
-                ldmatrix_x4(b, krow + k2 * 64);
+                ldmatrix_x4(b, krow + (k2 >> 1) * LD_ATOM + kx[k2 & 1]);
                 mma_bf16(s4[(2 * k2) & 3], qf[2 * k2], b[0], b[1]);
-                if (2 * k2 + 1 < nk) mma_bf16(s4[(2 * k2 + 1) & 3], qf[2 * k2 + 1], b[2], b[3]);
+                if (EXACT || 2 * k2 + 1 < nk) mma_bf16(s4[(2 * k2 + 1) & 3], qf[2 * k2 + 1], b[2], b[3]);
             }
         }
         const int key = warp * 8 + c_lo, j = j_first + t * LD_BN + key;
@@ -180,9 +183,10 @@ attn_latent_dec_kernel(const LatentArgs a) {
 #pragma unroll
             for (int nd = 0; nd < NDV; ++nd) {
                 const int c16 = warp * NDV + nd;
-                if (c16 * 16 < KRP) {
+                if (EXACT || c16 * 16 < KRP) {
                     uint32_t b[4];
-                    ldmatrix_x4_trans(b, kb + (kp * 16 + (mi & 1) * 8 + lr) * QP + (c16 * 2 + (mi >> 1)) * 16);
+                    const int ch = c16 * 2 + (mi >> 1);
+                    ldmatrix_x4_trans(b, kb + (ch >> 3) * LD_ATOM + (kp * 16 + (mi & 1) * 8 + lr) * 128 + (((ch & 7) ^ lr) << 4));
                     mma_bf16(acc[2 * nd], pa, b[0], b[1]);
                     mma_bf16(acc[2 * nd + 1], pa, b[2], b[3]);
                 }
@@ -230,17 +234,21 @@ attn_latent_dec_kernel(const LatentArgs a) {
 }
 
 static size_t latent_dec_smem(int ROW) {
-    const size_t QP = ((ROW + 15) & ~15) * 2 + 16;
-    return (size_t)LD_NB * LD_BN * QP + 16 * (LD_BN + 8) * 2 + 2 * 16 * 8 * sizeof(float);
+    return (size_t)LD_NB * ((ROW + 63) / 64) * LD_ATOM + 16 * (LD_BN + 8) * 2 + 2 * 16 * 8 * sizeof(float) + 1024;
 }
-static bool latent_dec_takes(int ROW, int KR) { return ROW % 8 == 0 && KR % 8 == 0 && KR <= ROW && KR <= 512 && ROW <= 576; }
+static bool latent_dec_takes(int ROW, int KR, int page_size, int num_pages) {
+    return ROW % 8 == 0 && KR % 8 == 0 && KR <= ROW && KR <= 512 && ROW <= 576 && page_size >= 8 && page_size <= 1024 &&
+           !(page_size & (page_size - 1)) && (long long)num_pages * page_size <= 0x7fffffffLL;
+}
 
 // a.HB, a.n_dec, a.n_split and the rest of the arguments are set; the merge follows by the caller
-template <int NK, int NDV>
+template <int NK, int NDV, bool EXACT>
 static int launch_latent_dec(const LatentArgs& a, cudaStream_t stream) {
     static AcvSmemConfig cfg;
     const size_t smem = latent_dec_smem(a.ROW);
-    if (int rc = acv_ensure_smem(cfg, attn_latent_dec_kernel<NK, NDV>, (int)smem)) return rc;
-    acv_launch(PDL_ATTN, attn_latent_dec_kernel<NK, NDV>, dim3(a.n_dec * a.n_split * a.HB), dim3(LD_THREADS), smem, stream, a);
+    if (int rc = acv_ensure_smem(cfg, attn_latent_dec_kernel<NK, NDV, EXACT>, (int)smem)) return rc;
+    CUtensorMap rows;
+    if (int rc = make_map(&rows, a.pages, a.num_pages * a.page_size, a.ROW, a.ROW, a.page_size < LD_BN ? a.page_size : LD_BN)) return rc;
+    acv_launch(PDL_ATTN, attn_latent_dec_kernel<NK, NDV, EXACT>, dim3(a.n_dec * a.n_split * a.HB), dim3(LD_THREADS), smem, stream, rows, a);
     return 0;
 }

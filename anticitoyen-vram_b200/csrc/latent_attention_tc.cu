@@ -19,6 +19,7 @@
 // the shared memory hold.  Rows are padded by 16 bytes instead of swizzled, so ROW and KR need only be multiples of 8.
 #include "mma_tiles.cuh"
 #include "tc_ptx.cuh"
+#include "tensor_map.h"
 
 #define LT_LOG2E 1.4426950408889634f
 #define LT_TILE_TOKENS 128      // query tokens in a tile of the step's work list
@@ -456,7 +457,7 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
     if (n_tiles == 0 && n_dec == 0) return 0;
     LatentShape sh = {};
     // one-token requests have a kernel of their own where its sizes allow; portions beside them are then a launch of their own
-    const bool dec_own = n_dec > 0 && latent_dec_takes(ROW, KR);
+    const bool dec_own = n_dec > 0 && latent_dec_takes(ROW, KR, page_size, num_pages);
     if ((n_tiles > 0 || !dec_own) && !latent_tc_shape(NH, ROW, KR, n_tiles > 0, sh)) return ACV_ERR_SIZE;
     if (((uintptr_t)q & 15) || ((size_t)q_stride * 2) % 16 || ((uintptr_t)pages & 15) || ((uintptr_t)out & 3) || (out_stride & 1))
         return ACV_ERR_ALIGN;
@@ -468,9 +469,10 @@ ACV_API int acv_attention_latent_tc(const void* q, int q_stride, void* out, int 
         d.n_tiles = 0;
         d.HB = (NH + 15) / 16;
         int rc;
-        if (ROW <= 192 && KR <= 128) rc = launch_latent_dec<12, 1>(d, stream);
-        else if (ROW <= 320 && KR <= 256) rc = launch_latent_dec<20, 2>(d, stream);
-        else rc = launch_latent_dec<36, 4>(d, stream);
+        if (ROW == 576 && KR == 512) rc = launch_latent_dec<36, 4, true>(d, stream);
+        else if (ROW <= 192 && KR <= 128) rc = launch_latent_dec<12, 1, false>(d, stream);
+        else if (ROW <= 320 && KR <= 256) rc = launch_latent_dec<20, 2, false>(d, stream);
+        else rc = launch_latent_dec<36, 4, false>(d, stream);
         if (rc) return rc;
         if (n_split > 1)
             acv_launch(PDL_ATTN, attn_latent_merge_kernel, dim3(n_dec * NH), dim3(128), 0, stream, (const float*)part_acc,
