@@ -70,6 +70,22 @@ def test_plan_and_what_every_layer_keeps():
     assert set(names) == set(lu.random_weights(lu.config("A"), 0))
 
 
+def test_blocks_and_contexts_of_a_step():
+    from acvram_b200.kernels import ops
+    arrays, values = ops.delta_work([1, 17, 8, 9])
+    assert values == {"n_items": 7}
+    assert arrays["seg_seq"].tolist() == [0, 1, 1, 1, 2, 3, 3] and arrays["seg_idx"].tolist() == [0, 0, 1, 2, 0, 0, 1]
+    assert arrays["first_block"].tolist() == [0, 1, 4, 5]
+    # portions that bring few queries for a long context leave it as it is; one-token requests never count
+    assert ops.latent_context_work([1, 1], [500, 900])[1]["n_pages"] == 0
+    assert ops.latent_context_work([2, 1], [500, 900])[1]["n_pages"] == 0
+    assert ops.latent_context_work([2, 100], [100000, 100000])[1]["n_pages"] == 0        # more rows than a step writes out
+    arrays, values = ops.latent_context_work([1, 100, 128], [500, 129, 128])
+    assert values == {"n_pages": 3, "width": 2} and arrays["order"].tolist() == [0]
+    assert arrays["page_seq"].tolist() == [1, 1, 2] and arrays["page_idx"].tolist() == [0, 1, 0]
+    assert arrays["table"].reshape(3, 2).tolist() == [[-1, -1], [0, 1], [2, -1]]
+
+
 def test_rotation_by_hand():
     x = np.arange(8.0).reshape(2, 4)                        # positions 0 and 1, one vector each
     r = lu.rot(100.0, 4)

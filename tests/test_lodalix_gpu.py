@@ -211,6 +211,21 @@ def test_mixed_batches_in_a_small_pool(folders, which, dtype):
     assert all(g.num_free == 3 for g in runner.manager.state_groups)
 
 
+@pytest.mark.parametrize("which", ["A", "B", "C", "D"])
+def test_portions_with_written_out_keys_beside_decoded_tokens(folders, which):
+    """Long portions (whose contexts are written out as keys and values) in one step with single tokens (which go on over
+    the kept rows), the portions in the middle of their requests, and then the other way round."""
+    from acvram_b200.kernels import ops
+    f = folders[which]
+    requests = {"a": ids_of(f, 47, 61), "b": ids_of(f, 330, 62), "c": ids_of(f, 290, 63)}
+    assert ops.latent_context_work([1, 200, 150], [41, 230, 150])[1]["n_pages"] > 0
+    runner = make_runner(f, "bfloat16", pages=64)
+    steps = [{"a": 40, "b": 30}, {"a": 1, "b": 200, "c": 150}, {"a": 1, "b": 1, "c": 137}, {"a": 1, "b": 97, "c": 1}]
+    steps += [{"a": 2, "b": 1, "c": 1}, {"a": 2, "b": 1, "c": 1}]
+    got = play(runner, requests, steps)
+    agree(f, requests, got, "bfloat16", "written out")
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_a_far_key_decides(tmp_path, dtype):
     """One layer of each latent kind alone with a sharp softmax: position 600 must find the keys of the first tokens.  The

@@ -143,6 +143,9 @@ SINK_CASES = [
     (16, 576, 512, 64, [400, 300, 64], [150, 1, 1]),            # four warps share a row group
     (80, 320, 256, 16, [60, 40], [9, 1]),                       # head blocks
     (16, 144, 128, 16, [900, 40, 1300], [1, 1, 1]),             # one-token requests whose rows several CTAs share
+    (20, 576, 512, 64, [700, 64, 65, 3], [1, 1, 1, 1]),         # more heads than a CTA's 16, a tile's edge, a few keys
+    (5, 72, 48, 8, [130, 9], [1, 1]),                           # small pages; rows that end inside a 64-element piece
+    (6, 200, 136, 128, [300, 129], [1, 1]),                     # pages of two tiles
 ]
 
 
@@ -182,6 +185,83 @@ def test_sinks_over_kept_rows(case):
     out = torch.full((T, NH * KR), 7.0, device=DEV, dtype=torch.bfloat16)
     ops.attention_latent(q, out, k, ctx, table, NH, ROW, KR, scale, work=work, sinks=sd)
     assert float(np.abs(out.cpu().double().numpy().reshape(T, NH, KR) - want).max()) < 2e-2 * plain
+
+
+@pytest.mark.parametrize("window", [0, 70])
+def test_one_token_requests_over_kept_rows_under_a_window(window):
+    """The kernel for one-token requests beside a padded slot of a captured batch (no context): zeros come out, and the
+    others are as the dense sums say, with and without a window."""
+    from acvram_b200.kernels import ops
+    NH, ROW, KR, page, lens = 7, 144, 128, 16, [200, 71, 70, 1]
+    ctx, work, table, k, _, T = paged_case(1, ROW, 8, page, lens, [1, 1, 1, 1], 8, torch.bfloat16)
+    q = torch.randn(T, NH * ROW, generator=torch.Generator().manual_seed(4)).to(torch.bfloat16).to(DEV)
+    ctx.kv_len[3] = 0
+    out = torch.full((T, NH * KR), 7.0, device=DEV, dtype=torch.bfloat16)
+    ops.attention_latent(q, out, k, ctx, table, NH, ROW, KR, 0.1, window, work=work)
+    assert float(out[3].abs().max()) == 0.0
+    for b, n in enumerate(lens[:3]):
+        js = torch.arange(max(0, n - window) if window else 0, n)
+        rows = k.cpu().double()[table[b].long().cpu()[js // page], 0, js % page].numpy()
+        s = q[b].cpu().double().view(NH, ROW).numpy() @ rows.T * 0.1
+        w = np.exp(s - s.max(-1, keepdims=True))
+        close(out[b].view(NH, KR), (w / w.sum(-1, keepdims=True)) @ rows[:, :KR], 2e-2, f"request {b}")
+
+
+@pytest.mark.parametrize("H,D,R,DV,KR,page,gated", [(3, 16, 8, 24, 48, 16, True), (4, 64, 64, 128, 128, 64, False), (2, 7, 2, 9, 33, 8, True),
+                                                    (5, 32, 32, 64, 64, 16, False)])
+def test_written_out_keys_and_values(H, D, R, DV, KR, page, gated):
+    """A step of two portions and a one-token request, the portions' contexts longer than their tokens: keys and values
+    written out from the pages (pages in any order), attention over them, the heads gated into columns of wider rows, the
+    one-token request picked out of the queries.  One key at a page's end is planted so that its score stands out."""
+    from acvram_b200.kernels import ops
+    rng = np.random.default_rng(H * 10 + D)
+    HD, ROW = (64 if max(D + R, DV) <= 64 else 128), KR + R
+    lens, q_lens = [190, 33, 260], [150, 1, 77]
+    ctx, work, table, pages, _, T = paged_case(1, ROW, 8, page, lens, q_lens, 3 + H, torch.bfloat16)
+    arrays, values = ops.latent_context_work(q_lens, lens)
+    assert values["n_pages"] == 2 + 3 and arrays["table"].reshape(3, -1).tolist() == [[0, 1, -1], [-1, -1, -1], [2, 3, 4]]
+    ex = {**{k: i32(v) for k, v in arrays.items()}, **values}
+    uk, uv = bf(rng.standard_normal((H, D, KR)) / math.sqrt(KR)), bf(rng.standard_normal((H, DV, KR)) / math.sqrt(KR))
+    q = bf(rng.standard_normal((T, H, D + R)))
+    rows = [pages.cpu().double()[table[b].long().cpu()[torch.arange(n) // page], 0, torch.arange(n) % page].numpy() for b, n in enumerate(lens)]
+    place = lens[2] // page * page - 1
+    rows[2][place, KR:] = q[-1, 0, D:] * 3.0 / math.sqrt(R)
+    pages[table[2, place // page].item(), 0, place % page] = dev(rows[2][place], torch.bfloat16)
+    rows[2][place] = pages[table[2, place // page].item(), 0, place % page].cpu().double().numpy()
+    scale = 1.5 * (D + R) ** -0.5
+    z, sinks = bf(rng.standard_normal((T, H * DV))), bf(rng.standard_normal(H))
+    want = np.zeros((T, H, DV))
+    t0 = 0
+    for b, (n, ql) in enumerate(zip(lens, q_lens)):
+        for h in range(H):
+            keys = np.concatenate([rows[b][:, :KR] @ uk[h].T, rows[b][:, KR:]], axis=1)
+            s = np.zeros((n, n))
+            s[n - ql:] = q[t0:t0 + ql, h] @ keys.T * scale
+            want[t0:t0 + ql, h] = pl.causal_weights(s, float(sinks[h]))[n - ql:] @ (rows[b][:, :KR] @ uv[h].T)
+        t0 += ql
+    want = want.reshape(T, -1) * (pl.sigmoid(z) if gated else 1.0)
+    qx = torch.zeros((T, H, HD), device=DEV, dtype=torch.bfloat16)
+    qx[:, :, :D + R] = dev(q, torch.bfloat16)
+    qx = qx.view(T, -1)
+    got_rows = ops.latent_context(pages, ctx, table, ex, ROW)
+    assert torch.equal(got_rows[:lens[0]].double().cpu(), torch.as_tensor(rows[0])) and float(got_rows[lens[0]:256].abs().max()) == 0.0
+    w = torch.cat([dev(uk.reshape(-1, KR), torch.bfloat16), dev(uv.reshape(-1, KR), torch.bfloat16)])
+    kv = got_rows[:, :KR] @ w.t()
+    kp, vp = ops.latent_pack(kv, got_rows, H, D, R, DV, KR, HD)
+    o = torch.full((T, H * HD), 7.0, device=DEV, dtype=torch.bfloat16)
+    sd = dev(sinks)
+    ops.attention_tc(qx, o, kp, vp, work["tile_seq"], work["tile_q0"], work["n_tiles"], ctx.cu_q, ctx.kv_len,
+                     ex["table"].view(-1, ex["width"]), H, H, HD, scale, 0, sinks=sd)
+    out = torch.full((T, H * DV + 5), 7.0, device=DEV, dtype=torch.bfloat16)
+    gate = dev(z, torch.bfloat16) if gated else None
+    ops.heads_gated(o, HD, gate, None, out[:, :H * DV], H, DV)
+    met = torch.zeros((1, H * ROW), device=DEV, dtype=torch.bfloat16)
+    plain = ops.latent_pick(qx, HD, work["dec_tokens"], 1, met, H, D, R, KR)
+    assert torch.equal(plain[0].double().cpu(), torch.as_tensor(q[150, :, :D])) and torch.equal(met.view(H, ROW)[:, KR:].double().cpu(), torch.as_tensor(q[150, :, D:]))
+    one = dev(want[150:151].reshape(1, -1) if not gated else (want[150:151] / pl.sigmoid(z[150:151])).reshape(1, -1), torch.bfloat16)
+    ops.heads_gated(one, DV, gate, work["dec_tokens"], out[:, :H * DV], H, DV)
+    close(out[:, :H * DV], want, 2.5e-2, "heads")
+    assert bool((out[:, H * DV:] == 7.0).all())
 
 
 # --------------------------------------------------------------------------- gated per-head products, the clamped unit, the block
