@@ -20,69 +20,71 @@
 // rot on pass unchanged.  A layer that reads rows kept by another one gives no kv: queries only.
 #include "common.cuh"
 
-__device__ __forceinline__ float rot_pairs(const float* x, int e, int rot, const float* cs, int halves) {
-    if (e >= rot) return x[e];
-    if (halves) {
-        const int m = rot >> 1, i = e < m ? e : e - m;
-        const float c = cs[i], s = cs[m + i];
-        return e < m ? fmaf(x[e], c, -x[e + m] * s) : fmaf(x[e], c, x[e - m] * s);
-    }
-    const int i = e >> 1;
-    const float c = cs[i], s = cs[(rot >> 1) + i];
-    return (e & 1) ? fmaf(x[e], c, x[e - 1] * s) : fmaf(x[e], c, -x[e + 1] * s);
-}
-
 template <typename T>
-__global__ void latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ q_out, int qo_stride,
-                                      const T* __restrict__ kv, int kv_stride, const float* __restrict__ w, float eps,
-                                      const float* __restrict__ cos_sin, int rot, int table_rows,
-                                      const int* __restrict__ positions, const int* __restrict__ seq_of_token,
-                                      const int* __restrict__ block_table, int bt_stride, const int* __restrict__ bt_rows,
-                                      T* __restrict__ pages, int page_size, int num_pages, int H, int D, int R, int KR, int halves, int full) {
-    extern __shared__ float sm[];           // [KR + R] the kv row, then [H * R] the heads' rotated parts
+__global__ void __launch_bounds__(256)
+latent_prepare_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ q_out, int qo_stride,
+                      const T* __restrict__ kv, int kv_stride, const float* __restrict__ w, float eps,
+                      const float* __restrict__ cos_sin, int rot, int table_rows, const int* __restrict__ positions,
+                      const int* __restrict__ seq_of_token, const int* __restrict__ block_table, int bt_stride,
+                      const int* __restrict__ bt_rows, T* __restrict__ pages, int page_size, int num_pages, int H, int D, int R,
+                      int KR, int halves, int full, int vec) {
+    extern __shared__ float row[];          // [KR] the latent part of the kv row
     __shared__ float red[32];
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, tid = threadIdx.x, nthr = blockDim.x;
-    int pos = positions[t];
-    if (pos >= table_rows) pos = table_rows - 1;
+    const int warp = tid >> 5, lane = tid & 31, nw = nthr >> 5, half = rot >> 1;
+    const int at = positions[t], pos = min(at, table_rows - 1);
     const float* cs = cos_sin + (size_t)pos * rot;
-    float* row = sm;
-    float* qr = sm + KR + R;
+    float c0 = 1.f, s0 = 0.f;               // the lane's first pair
+    if (lane < half) { c0 = cs[lane]; s0 = cs[half + lane]; }
+    int pg = -1;
+    if (pages && kv) {
+        const int seq = seq_of_token[t];
+        pg = block_table[(size_t)(bt_rows ? bt_rows[seq] : seq) * bt_stride + at / page_size];
+    }
+    // R elements turned, by a warp: a lane a pair
+    auto turn = [&](const T* src, T* dst) {
+        for (int i = lane; i < half; i += 32) {
+            const float c = i == lane ? c0 : cs[i], s = i == lane ? s0 : cs[half + i];
+            const int a = halves ? i : 2 * i, b = halves ? i + half : 2 * i + 1;
+            const float u = to_f32(src[a]), v = to_f32(src[b]);
+            dst[a] = from_f32<T>(fmaf(u, c, -v * s));
+            dst[b] = from_f32<T>(fmaf(v, c, u * s));
+        }
+        for (int e = rot + lane; e < R; e += 32) dst[e] = src[e];
+    };
+    const T* kvr = kv + (size_t)t * kv_stride;
     float ss = 0.f;
-    if (kv) {
-        const T* kvr = kv + (size_t)t * kv_stride;
-        for (int e = tid; e < KR + R; e += nthr) {
+    if (kv)
+        for (int e = tid; e < KR; e += nthr) {
             const float v = to_f32(kvr[e]);
             row[e] = v;
-            if (e < KR) ss = fmaf(v, v, ss);
+            ss = fmaf(v, v, ss);
+        }
+    for (int h = warp; h < H; h += nw) {
+        const T* src = q + (size_t)t * q_stride + (size_t)h * (D + R);
+        if (full) {             // whole heads [plain | rotated | zeros] of `full` elements
+            T* dst = q_out + (size_t)t * qo_stride + (size_t)h * full;
+            constexpr int P = 8 / (int)sizeof(T);
+            if (vec) {          // plain parts in 8-byte pieces
+                for (int e = lane * P; e < D; e += 32 * P) *reinterpret_cast<uint2*>(dst + e) = *reinterpret_cast<const uint2*>(src + e);
+            } else {
+                for (int e = lane; e < D; e += 32) dst[e] = src[e];
+            }
+            turn(src + D, dst + D);
+            for (int e = D + R + lane; e < full; e += 32) dst[e] = from_f32<T>(0.f);
+        } else {
+            turn(src + D, q_out + (size_t)t * qo_stride + (size_t)h * (KR + R) + KR);
         }
     }
-    for (int i = tid; i < H * R; i += nthr) {
-        const int h = i / R, e = i - h * R;
-        qr[i] = to_f32(q[(size_t)t * q_stride + (size_t)h * (D + R) + D + e]);
-    }
-    ss = block_sum(ss, red);                // (meets the block: row and qr are whole)
-    const float inv = 1.f / sqrtf(ss / (float)KR + eps);
-    if (full) {         // whole heads [plain | rotated | zeros] of `full` elements
-        for (int i = tid; i < H * full; i += nthr) {
-            const int h = i / full, e = i - h * full;
-            float v = 0.f;
-            if (e < D) v = to_f32(q[(size_t)t * q_stride + (size_t)h * (D + R) + e]);
-            else if (e < D + R) v = rot_pairs(qr + h * R, e - D, rot, cs, halves);
-            q_out[(size_t)t * qo_stride + i] = from_f32<T>(v);
-        }
-    } else for (int i = tid; i < H * R; i += nthr) {
-        const int h = i / R, e = i - h * R;
-        q_out[(size_t)t * qo_stride + (size_t)h * (KR + R) + KR + e] = from_f32<T>(rot_pairs(qr + h * R, e, rot, cs, halves));
-    }
-    if (!pages || !kv) return;
-    const int seq = seq_of_token[t];
-    const int pg = block_table[(size_t)(bt_rows ? bt_rows[seq] : seq) * bt_stride + positions[t] / page_size];
+    if (!kv) return;
+    ss = block_sum(ss, red);                // (meets the block: row is whole)
     if (pg < 0 || pg >= num_pages) return;
-    T* dst = pages + ((size_t)pg * page_size + (positions[t] % page_size)) * (KR + R);
+    const float inv = 1.f / sqrtf(ss / (float)KR + eps);
+    T* dst = pages + ((size_t)pg * page_size + at % page_size) * (KR + R);
     for (int e = tid; e < KR; e += nthr) dst[e] = from_f32<T>(row[e] * inv * w[e]);
-    for (int e = tid; e < R; e += nthr) dst[KR + e] = from_f32<T>(rot_pairs(row + KR, e, rot, cs, halves));
+    if (warp == nw - 1) turn(kvr + KR, dst + KR);
 }
 
 // q: rows of H*(D+R) at q_stride; q_out: rows of H*(KR+R) at qo_stride; kv: rows of KR+R at kv_stride; w float [KR];
@@ -96,9 +98,12 @@ ACV_API int acv_latent_prepare(const void* q, int q_stride, void* q_out, int qo_
     if (T_tokens <= 0) return 0;
     if (H <= 0 || D < 0 || R <= 0 || KR <= 0 || rot < 0 || rot > R || (rot & 1) || (full && full < D + R) || (rot && (!cos_sin || table_rows <= 0)))
         return ACV_ERR_SIZE;
-    const size_t smem = (size_t)(KR + R + H * R) * sizeof(float);
+    const size_t smem = (size_t)KR * sizeof(float);
     if (smem > 200 * 1024) return ACV_ERR_SIZE;
     const int threads = 256;
+    const int piece = dtype == ACV_F32 ? 2 : 4;         // elements of 8 bytes
+    const int vec = D % piece == 0 && R % piece == 0 && full % piece == 0 && q_stride % piece == 0 && qo_stride % piece == 0 &&
+                    !(((uintptr_t)q | (uintptr_t)q_out) & 7);
 #define LP_LAUNCH(T)                                                                                                    \
     do {                                                                                                                \
         if (smem > 48 * 1024) {                                                                                         \
@@ -108,7 +113,7 @@ ACV_API int acv_latent_prepare(const void* q, int q_stride, void* q_out, int qo_
         }                                                                                                               \
         acv_launch(PDL_ROPE, latent_prepare_kernel<T>, T_tokens, threads, smem, stream, (const T*)q, q_stride, (T*)q_out, \
                    qo_stride, (const T*)kv, kv_stride, w, eps, cos_sin, rot, table_rows, positions, seq_of_token,       \
-                   block_table, bt_stride, bt_rows, (T*)pages, page_size, num_pages, H, D, R, KR, halves, full);                      \
+                   block_table, bt_stride, bt_rows, (T*)pages, page_size, num_pages, H, D, R, KR, halves, full, vec);                      \
     } while (0)
     if (dtype == ACV_F32) LP_LAUNCH(float);
     else if (dtype == ACV_BF16) LP_LAUNCH(bf16);
