@@ -1768,7 +1768,7 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, ct
 LATENT_SPLIT_KEYS = 128         # no share of a one-token request's kept rows is shorter than this
 LATENT_PAGE = 128               # tokens of a page of written-out keys and values (csrc/latent_expand.cu)
 LATENT_EXPAND_QUERIES = 32      # queries a context row must meet on average for its keys and values to be written out
-LATENT_EXPAND_ROWS = 1 << 17    # most context rows that a step writes out
+LATENT_EXPAND_ROWS = 1 << 16    # most context rows that a step writes out
 
 
 def latent_context_work(q_lens, kv_lens) -> tuple[dict, dict]:
