@@ -13,7 +13,8 @@
 // positions: nothing is shifted).
 // s = scale * q.k - slope_h * (p - j) (slopes: one per query head, or none); with sinks (one number per query head) the
 // softmax's denominator also holds exp(sink_h), which has no key and no value.  Softmax over the visible keys with a running maximum and sum in
-// 32-bit (acvram/kernels/acvram_kernels.cu:993-1146 has the same recurrence).
+// 32-bit (acvram/kernels/acvram_kernels.cu:993-1146 has the same recurrence).  With a gate (rows like the result's) the
+// result is multiplied by sigmoid(gate) before it is rounded.
 #include "common.cuh"
 
 #define AG_WARPS 4
@@ -24,7 +25,8 @@ __global__ void attn_generic_kernel(const T* __restrict__ q, int q_stride, T* __
                                     const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                                     const int* __restrict__ block_table, int bt_stride, const int* __restrict__ bt_rows, int NH, int NKV, int D, int DV,
                                     int page_size, int num_pages, float scale, int window, int keep_first, int v_row,
-                                    const float* __restrict__ sinks, const float* __restrict__ slopes) {
+                                    const float* __restrict__ sinks, const float* __restrict__ slopes,
+                                    const T* __restrict__ gate, int gate_stride) {
     extern __shared__ float sm_all[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y * AG_WARPS + warp;
@@ -115,7 +117,10 @@ __global__ void attn_generic_kernel(const T* __restrict__ q, int q_stride, T* __
 #pragma unroll
     for (int r = 0; r < NR; ++r) {
         const int e = lane + 32 * r;
-        if (e < DV) orow[e] = from_f32<T>(acc[r] * inv_l);
+        if (e >= DV) continue;
+        float o = acc[r] * inv_l;
+        if (gate) o *= 1.f / (1.f + expf(-to_f32(gate[(size_t)t * gate_stride + (size_t)h * DV + e])));
+        orow[e] = from_f32<T>(o);
     }
 }
 
@@ -123,7 +128,8 @@ template <typename T>
 static int launch_generic(const void* q, int q_stride, void* out, int out_stride, const void* k_pages,
                           const void* v_pages, const int* positions, const int* seq_of_token, const int* block_table,
                           int bt_stride, const int* bt_rows, int T_tokens, int NH, int NKV, int D, int DV, int page_size, int num_pages,
-                          float scale, int window, int keep_first, int v_row, const float* sinks, const float* slopes, cudaStream_t stream) {
+                          float scale, int window, int keep_first, int v_row, const float* sinks, const float* slopes, const void* gate, int gate_stride,
+                          cudaStream_t stream) {
     dim3 grid(T_tokens, (NH + AG_WARPS - 1) / AG_WARPS);
     const size_t smem = (size_t)AG_WARPS * D * sizeof(float);
     const int nr = (DV + 31) / 32;
@@ -131,7 +137,8 @@ static int launch_generic(const void* q, int q_stride, void* out, int out_stride
     case N:                                                                                                          \
         attn_generic_kernel<T, N><<<grid, AG_WARPS * 32, smem, stream>>>(                                            \
             (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pages, (const T*)v_pages, positions,             \
-            seq_of_token, block_table, bt_stride, bt_rows, NH, NKV, D, DV, page_size, num_pages, scale, window, keep_first, v_row, sinks, slopes);                \
+            seq_of_token, block_table, bt_stride, bt_rows, NH, NKV, D, DV, page_size, num_pages, scale, window, keep_first, v_row, sinks, slopes, \
+            (const T*)gate, gate_stride);                                                                            \
         break;
     switch (nr) {
         AG_CASE(1) AG_CASE(2) AG_CASE(3) AG_CASE(4) AG_CASE(5) AG_CASE(6) AG_CASE(7) AG_CASE(8)
@@ -146,7 +153,8 @@ ACV_API int acv_attention_generic(const void* q, int q_stride, void* out, int ou
                                   const void* v_pages, const int* positions, const int* seq_of_token,
                                   const int* block_table, int bt_stride, const int* bt_rows, int T_tokens, int NH, int NKV, int D,
                                   int page_size, int num_pages, float scale, int window, int dtype,
-                                  int value_dim, int keep_first, const float* sinks, const float* slopes, cudaStream_t stream) {
+                                  int value_dim, int keep_first, const float* sinks, const float* slopes, const void* gate,
+                                  int gate_stride, cudaStream_t stream) {
     if (T_tokens <= 0) return 0;
     const int DV = value_dim > 0 ? value_dim : D;
     if (D <= 0 || D > 1024 || DV > 512 || NKV <= 0 || NH % NKV) return ACV_ERR_SIZE;
@@ -156,10 +164,10 @@ ACV_API int acv_attention_generic(const void* q, int q_stride, void* out, int ou
     if (dtype == ACV_F32)
         return launch_generic<float>(q, q_stride, out, out_stride, k_pages, v_pages, positions, seq_of_token,
                                      block_table, bt_stride, bt_rows, T_tokens, NH, NKV, D, DV, page_size, num_pages, scale, window,
-                                     keep_first, v_row, sinks, slopes, stream);
+                                     keep_first, v_row, sinks, slopes, gate, gate_stride, stream);
     if (dtype == ACV_BF16)
         return launch_generic<bf16>(q, q_stride, out, out_stride, k_pages, v_pages, positions, seq_of_token,
                                     block_table, bt_stride, bt_rows, T_tokens, NH, NKV, D, DV, page_size, num_pages, scale, window,
-                                    keep_first, v_row, sinks, slopes, stream);
+                                    keep_first, v_row, sinks, slopes, gate, gate_stride, stream);
     return ACV_ERR_DTYPE;
 }

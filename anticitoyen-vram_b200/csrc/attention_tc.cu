@@ -55,6 +55,8 @@ struct AttnTcParams {
     float scale;
     int* status;
     const float* sinks;     // [NH] or null: exp(sink_h) joins the softmax's denominator (a score with no key and no value)
+    const bf16* gate;       // or null: rows like the result's, 16-byte pieces: the result is multiplied by sigmoid(gate) in float
+    int gate_stride;
     const float* slopes;    // [NH] or null: the score of query i and key j loses slope_h (i - j)
 };
 
@@ -365,6 +367,16 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 #pragma unroll
                     for (int c = 0; c < 32; c += 8) {
                         uint4 pk;
+                        if (p.gate) {
+                            const uint4 g = *reinterpret_cast<const uint4*>(p.gate + (size_t)(tok0 + r) * p.gate_stride + (size_t)head * D + c0 + c);
+                            const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const float ga = __uint_as_float(gw[e] << 16), gb = __uint_as_float(gw[e] & 0xffff0000u);
+                                o[c + 2 * e] = __float_as_uint(__uint_as_float(o[c + 2 * e]) * __fdividef(1.f, 1.f + __expf(-ga)));
+                                o[c + 2 * e + 1] = __float_as_uint(__uint_as_float(o[c + 2 * e + 1]) * __fdividef(1.f, 1.f + __expf(-gb)));
+                            }
+                        }
                         pk.x = pack_bf16x2(__uint_as_float(o[c]) * inv, __uint_as_float(o[c + 1]) * inv);
                         pk.y = pack_bf16x2(__uint_as_float(o[c + 2]) * inv, __uint_as_float(o[c + 3]) * inv);
                         pk.z = pack_bf16x2(__uint_as_float(o[c + 4]) * inv, __uint_as_float(o[c + 5]) * inv);
@@ -405,7 +417,8 @@ ACV_API int acv_attention_tc(const void* q, int q_stride, int T, void* out, int 
                              const void* v_pages, const int* tile_seq, const int* tile_q0, int n_tiles, const int* cu_q,
                              const int* kv_len, const int* block_table, int bt_stride, const int* bt_rows, int NH, int NKV,
                              int D, int page_size, int num_pages, float scale, int window, int chunk, int out_f32, int* status,
-                             int keep_first, const float* sinks, const float* slopes, cudaStream_t stream) {
+                             int keep_first, const float* sinks, const float* slopes, const void* gate, int gate_stride,
+                             cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (NKV <= 0 || NH % NKV || NH > 65535 || (D != 64 && D != 128)) return ACV_ERR_SIZE;
     if ((long long)n_tiles * NH > 0x7fffffffLL) return ACV_ERR_SIZE;
@@ -432,6 +445,9 @@ ACV_API int acv_attention_tc(const void* q, int q_stride, int T, void* out, int 
     p.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
     p.sinks = sinks;
     p.slopes = slopes;
+    p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
+    if (gate && (((uintptr_t)gate & 15) || (gate_stride % 8))) return ACV_ERR_ALIGN;
+    if (gate && out_f32) return ACV_ERR_SIZE;
     if (slopes && !(scale > 0.f)) return ACV_ERR_SIZE;
     p.status = status;
     if (D == 64) return launch_attn_tc<64>(mq, mk, mv, p, n_tiles, stream);

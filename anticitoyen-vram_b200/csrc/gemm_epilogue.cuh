@@ -17,10 +17,10 @@ struct GemmParams {
     int out_f32;
     int act;                // 1: output features come in (gate, up) pairs and C[:, n/2] = silu(gate) * up
                             // 2: the same pairs through a clamped gated unit, scaled by the row first (tokens on rows only):
-                            //    g = min(w gate, limit), u = clamp(w up, +-limit), C = g * sigmoid(alpha g) * (u + 1)
+                            //    g = min(w gate, limit), u = clamp(w up, +-limit), C = g * sigmoid(alpha g) * (u + shift)
     const float* bias;      // float [N]: added to the product's feature n before anything else is made of it (null: none)
     const float* row_scale; // act 2, and act 0 with tokens on rows: w of each row of A (null: 1)
-    float glu_limit, glu_alpha;
+    float glu_limit, glu_alpha, glu_shift;
     int gate_fn;            // act 1: what the pair becomes: 0 silu(gate) * up (with the roundings of the unfused path), 1 the
                             // tanh form of gelu instead (in float on the accumulators, the product rounded once), 2 the
                             // clamped gated unit of act 2 without a row scale (tokens on rows or on columns)
@@ -88,14 +88,14 @@ __device__ __forceinline__ float unary_act(float z, int kind) {
 }
 
 // The clamped gated unit of act 2, in float, rounded once.
-__device__ __forceinline__ bf16 glu_clamped_pair(float gate, float up, float w, float limit, float alpha) {
+__device__ __forceinline__ bf16 glu_clamped_pair(float gate, float up, float w, float limit, float alpha, float shift) {
     const float g = fminf(gate * w, limit);
     const float u = fminf(fmaxf(up * w, -limit), limit);
-    return __float2bfloat16_rn(g * __fdividef(1.f, 1.f + __expf(-alpha * g)) * (u + 1.f));
+    return __float2bfloat16_rn(g * __fdividef(1.f, 1.f + __expf(-alpha * g)) * (u + shift));
 }
 
 __device__ __forceinline__ bf16 gated_pair(const GemmParams& p, float gate, float up) {
-    if (p.gate_fn == 2) return glu_clamped_pair(gate, up, 1.f, p.glu_limit, p.glu_alpha);
+    if (p.gate_fn == 2) return glu_clamped_pair(gate, up, 1.f, p.glu_limit, p.glu_alpha, p.glu_shift);
     return p.gate_fn ? geglu_pair(gate, up) : swiglu_pair(gate, up);
 }
 
@@ -175,7 +175,7 @@ __device__ __forceinline__ void gt_store16(const GemmParams& p, int row_a, int c
             if (p.act == 2) {
                 const float w = p.row_scale ? p.row_scale[row_a] : 1.f;
 #pragma unroll
-                for (int k = 0; k < 8; ++k) o[k] = glu_clamped_pair(v[2 * k], v[2 * k + 1], w, p.glu_limit, p.glu_alpha);
+                for (int k = 0; k < 8; ++k) o[k] = glu_clamped_pair(v[2 * k], v[2 * k + 1], w, p.glu_limit, p.glu_alpha, p.glu_shift);
             } else {
 #pragma unroll
                 for (int k = 0; k < 8; ++k) o[k] = gated_pair(p, v[2 * k], v[2 * k + 1]);

@@ -902,7 +902,7 @@ ACV_API int acv_gemm_tc_bias(const void* x, int ldx, const void* w, int ldw, voi
     GemmParams p = {};
     p.qkv = 0;
     p.bias = bias;
-    p.glu_limit = limit; p.glu_alpha = alpha;
+    p.glu_limit = limit; p.glu_alpha = alpha; p.glu_shift = 1.f;
     return gemm_tc_run(p, x, ldx, w, ldw, C, ldc, M, N, K, out_f32, act, swap, bn, splits, workspace, workspace_floats,
                        counters, n_counters, status, sm_count, stages, flags, stream);
 }
@@ -913,7 +913,7 @@ ACV_API int acv_gemm_tc_glu(const void* x, int ldx, const void* w, int ldw, void
                             float alpha, int bn, int* status, int sm_count, int stages, int flags, cudaStream_t stream) {
     GemmParams p = {};
     p.qkv = 0;
-    p.glu_limit = limit; p.glu_alpha = alpha;
+    p.glu_limit = limit; p.glu_alpha = alpha; p.glu_shift = 1.f;
     return gemm_tc_run(p, x, ldx, w, ldw, C, ldc, M, N, K, 0, 2, 0, bn, 1, nullptr, 0, nullptr, 0, status, sm_count, stages,
                        flags & ~1, stream);
 }
@@ -921,15 +921,15 @@ ACV_API int acv_gemm_tc_glu(const void* x, int ldx, const void* w, int ldw, void
 // Grouped product, tokens on rows: x [M, K] holds rows grouped by expert in tiles of 128 (tile_expert[i]: the expert of
 // rows [128 i, 128 i + 128); *tiles_used: how many tiles hold rows, both on the device); w stacks `experts` matrices of N
 // rows; C [M, N] (act 0: bfloat16 or float) or [M, N / 2] (act 2: (gate, up) pairs of rows through the clamped gated
-// unit, the accumulators times row_scale[row] first).  Tiles beyond *tiles_used are not computed.
+// unit g * sigmoid(alpha g) * (u + shift), the accumulators times row_scale[row] first).  Tiles beyond *tiles_used are not computed.
 ACV_API int acv_gemm_tc_grouped(const void* x, int ldx, const void* w, int ldw, void* C, int ldc, int M, int N, int K,
                                 int experts, const int* tile_expert, const int* tiles_used, int out_f32, int act,
-                                const float* row_scale, float limit, float alpha, int bn, int* status, int sm_count,
+                                const float* row_scale, float limit, float alpha, float shift, int bn, int* status, int sm_count,
                                 int stages, cudaStream_t stream) {
     GemmParams p = {};
     p.qkv = 0;
     p.tile_expert = tile_expert; p.tiles_used = tiles_used; p.experts = experts;
-    p.row_scale = row_scale; p.glu_limit = limit; p.glu_alpha = alpha;
+    p.row_scale = row_scale; p.glu_limit = limit; p.glu_alpha = alpha; p.glu_shift = shift;
     if (!tile_expert || !tiles_used || (M % GT_BM)) return ACV_ERR_SIZE;
     return gemm_tc_run(p, x, ldx, w, ldw, C, ldc, M, N, K, out_f32, act, 0, bn, 1, nullptr, 0, nullptr, 0, status, sm_count,
                        stages, 0, stream);

@@ -8,7 +8,7 @@
 // sigmoid, g the output gate in front of its sigmoid, x the decay's inner values in front of their tanh.  All float.
 //
 //   acv_delta_blocks    everything that does not need the state, for eight tokens of a request at a time
-//   acv_delta           the recurrence over those blocks, o float
+//   acv_delta           the recurrence over those blocks, o float (also over the blocks of csrc/gated_delta.cu, see there)
 //   acv_delta_step      steps in which every request brings one token: all of the above, the head's norm, weight and gate
 //                       in one launch
 //
@@ -335,14 +335,17 @@ __device__ __forceinline__ constexpr int lane_of(int e) {
 template <int G>
 __device__ __forceinline__ constexpr int place_of(int e) { return G >= 8 ? 0 : e & (8 / G - 1); }
 
-template <int R, int G, int C, int NW, int STAGES>
+// KD: a record as above, state [D, D].  Without it the record is that of a gated delta rule, [kt' 8][rt 8][k' 8] rows, M, N and
+// the block's decay (one number, padded to four), and the state is [D, DV]:  u = kt' S + M v,  o = rt S + N v,
+// S_8 = decay S + sum_j k'_j u_j^T.
+template <int R, int G, int C, int NW, int STAGES, bool KD>
 __global__ void __launch_bounds__(NW * 32)
-delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int ld, float* __restrict__ state,
+delta_kernel(const float* __restrict__ rec, const float* __restrict__ values, int ld, float* __restrict__ state,
              const int* __restrict__ slots, const int* __restrict__ cu_q, const int* __restrict__ first_block,
-             float* __restrict__ o, int H, int D, int vec) {
+             float* __restrict__ o, int H, int D, int DV, int vec) {
     constexpr int DP = R * G, DVT = NW * (32 / G) * C, R2 = R / 2, LEFT = G >= 8 ? 1 : 8 / G;
     constexpr int PF = R < 4 ? 1 : 2;       // pairs in a piece that one load brings
-    constexpr int REC = 33 * DP + 128, SET = REC + 8 * DVT, NT = NW * 32;
+    constexpr int REC = KD ? 33 * DP + 128 : 24 * DP + 132, MATS = (KD ? 33 : 24) * DP, SET = REC + 8 * DVT, NT = NW * 32;
     extern __shared__ __align__(16) float sm[];
     pdl_wait();
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * DVT;
@@ -350,11 +353,11 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
     if (t1 <= t0) return;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int g = lane % G, cl = (warp * (32 / G) + lane / G) * C, c = c0 + cl;
-    const int I = H * D, nb = (t1 - t0 + 7) >> 3;
+    const int I = H * DV, nb = (t1 - t0 + 7) >> 3;
     const int e0 = first_of<G>(lane);
-    float* st = state + ((size_t)slots[seq] * H + h) * D * D;
+    float* st = state + ((size_t)slots[seq] * H + h) * D * DV;
     const float* recs = rec + ((size_t)first_block[seq] * H + h) * REC;
-    const float* vals = proj + (size_t)t0 * ld + 2 * (size_t)I + (size_t)h * D + c0;
+    const float* vals = values + (size_t)t0 * ld + (size_t)h * DV + c0;
 
     auto stage = [&](int b) {
         float* s = sm + (b % STAGES) * SET;
@@ -364,13 +367,13 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
         if (vec) {
             for (int i = tid * 4; i < 8 * DVT; i += NT * 4) {
                 const int tt = i / DVT, e = i % DVT, t = b * 8 + tt;
-                const bool in = t < t1 - t0 && c0 + e < D;
-                cp_async16(smem_u32(vs + i), in ? (const void*)(vals + (size_t)t * ld + e) : (const void*)proj, in);
+                const bool in = t < t1 - t0 && c0 + e < DV;
+                cp_async16(smem_u32(vs + i), in ? (const void*)(vals + (size_t)t * ld + e) : (const void*)values, in);
             }
         } else {
             for (int i = tid; i < 8 * DVT; i += NT) {
                 const int tt = i / DVT, e = i % DVT, t = b * 8 + tt;
-                vs[i] = t < t1 - t0 && c0 + e < D ? vals[(size_t)t * ld + e] : 0.f;
+                vs[i] = t < t1 - t0 && c0 + e < DV ? vals[(size_t)t * ld + e] : 0.f;
             }
         }
     };
@@ -381,8 +384,8 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
 #pragma unroll
         for (int i = 0; i < R2; ++i) {
             const int d = ((i / PF) * G + g) * PF * 2 + (i % PF) * 2;
-            const bool in = c + j < D;
-            S[j][i] = f2_pack(in && d < D ? st[(size_t)d * D + c + j] : 0.f, in && d + 1 < D ? st[(size_t)(d + 1) * D + c + j] : 0.f);
+            const bool in = c + j < DV;
+            S[j][i] = f2_pack(in && d < D ? st[(size_t)d * DV + c + j] : 0.f, in && d + 1 < D ? st[(size_t)(d + 1) * DV + c + j] : 0.f);
         }
 #pragma unroll
     for (int b = 0; b < STAGES - 1; ++b) {
@@ -414,7 +417,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
         if (b + STAGES - 1 < nb) stage(b + STAGES - 1);
         cp_async_commit();
         const float* s = sm + (b % STAGES) * SET;
-        const float* mn = s + 33 * DP;
+        const float* mn = s + MATS;
         const float* vs = s + REC + cl;
         float y[C][8], z[C][8], v[C][8];
         f2 x[R2];
@@ -436,7 +439,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
         for (int i = 0; i < 8; ++i)
 #pragma unroll
             for (int j = 0; j < C; ++j) v[j][i] = vs[i * DVT + j];
-        // this lane's tokens: p (its sum over the values of the tokens before it), later o
+        // this lane's tokens: p (its sum over the values of the tokens before it; the new values u without KD), later o
 #pragma unroll
         for (int l = 0; l < LEFT; ++l) {
             const float4 m0 = *reinterpret_cast<const float4*>(mn + (e0 + l) * 8), m1 = *reinterpret_cast<const float4*>(mn + (e0 + l) * 8 + 4);
@@ -445,27 +448,36 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
                 float a = fmaf(m0.x, v[j][0], y[j][l]), d = m0.y * v[j][1];
                 a = fmaf(m0.z, v[j][2], a); d = fmaf(m0.w, v[j][3], d);
                 a = fmaf(m1.x, v[j][4], a); d = fmaf(m1.y, v[j][5], d);
+                if constexpr (!KD) d = fmaf(m1.w, v[j][7], d);     // (with KD a token's p holds no value of its own)
                 y[j][l] = fmaf(m1.z, v[j][6], a) + d;
             }
         }
-        rows(s + 32 * DP, x);
+        if constexpr (KD) {
+            rows(s + 32 * DP, x);
+        } else {
+            const float decay = mn[128];
+#pragma unroll
+            for (int i = 0; i < R2; ++i) x[i] = f2_pack(decay, decay);
+        }
 #pragma unroll
         for (int j = 0; j < C; ++j)
 #pragma unroll
             for (int i = 0; i < R2; ++i) S[j][i] = f2_mul(x[i], S[j][i]);
+        if constexpr (KD) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            rows(s + (16 + i) * DP, x);
+            for (int i = 0; i < 8; ++i) {
+                rows(s + (16 + i) * DP, x);
 #pragma unroll
-            for (int j = 0; j < C; ++j) {
-                const f2 vv = f2_pack(v[j][i], v[j][i]);
+                for (int j = 0; j < C; ++j) {
+                    const f2 vv = f2_pack(v[j][i], v[j][i]);
 #pragma unroll
-                for (int q = 0; q < R2; ++q) S[j][q] = f2_fma(x[q], vv, S[j][q]);
+                    for (int q = 0; q < R2; ++q) S[j][q] = f2_fma(x[q], vv, S[j][q]);
+                }
             }
         }
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            rows(s + (24 + i) * DP, x);
+            rows(s + ((KD ? 24 : 16) + i) * DP, x);
 #pragma unroll
             for (int j = 0; j < C; ++j) {
                 const float p = G > 1 ? __shfl_sync(0xffffffffu, y[j][place_of<G>(i)], lane_of<G>(i), G) : y[j][i];
@@ -487,7 +499,7 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
                     a = fmaf(m0.z, v[j][2], a); d = fmaf(m0.w, v[j][3], d);
                     a = fmaf(m1.x, v[j][4], a); d = fmaf(m1.y, v[j][5], d);
                     a = fmaf(m1.z, v[j][6], a); d = fmaf(m1.w, v[j][7], d);
-                    if (t < t1 && c + j < D) o[(size_t)t * I + (size_t)h * D + c + j] = a + d;
+                    if (t < t1 && c + j < DV) o[(size_t)t * I + (size_t)h * DV + c + j] = a + d;
                 }
             }
         }
@@ -500,42 +512,38 @@ delta_kernel(const float* __restrict__ rec, const float* __restrict__ proj, int 
             const int d = ((i / PF) * G + g) * PF * 2 + (i % PF) * 2;
             float a, b;
             f2_split(S[j][i], a, b);
-            if (c + j < D && d < D) st[(size_t)d * D + c + j] = a;
-            if (c + j < D && d + 1 < D) st[(size_t)(d + 1) * D + c + j] = b;
+            if (c + j < DV && d < D) st[(size_t)d * DV + c + j] = a;
+            if (c + j < DV && d + 1 < D) st[(size_t)(d + 1) * DV + c + j] = b;
         }
 }
 
-template <int R, int G, int C, int NW, int STAGES>
-static int launch_delta(const float* rec, const float* proj, int ld, float* state, const int* slots, const int* cu_q,
-                        const int* first_block, float* o, int n_seqs, int H, int D, cudaStream_t stream) {
+template <int R, int G, int C, int NW, int STAGES, bool KD>
+static int launch_delta(const float* rec, const float* values, int ld, float* state, const int* slots, const int* cu_q,
+                        const int* first_block, float* o, int n_seqs, int H, int D, int DV, cudaStream_t stream) {
     constexpr int DVT = NW * (32 / G) * C;
-    constexpr size_t smem = (size_t)STAGES * (33 * R * G + 128 + 8 * DVT) * sizeof(float);
+    constexpr size_t smem = (size_t)STAGES * ((KD ? 33 * R * G + 128 : 24 * R * G + 132) + 8 * DVT) * sizeof(float);
     static_assert(smem <= 227 * 1024 && DVT % 4 == 0, "a block's stages fit, values come in 16-byte pieces");
     static AcvSmemConfig cfg;
     if (smem > 48 * 1024)
-        if (int e = acv_ensure_smem(cfg, delta_kernel<R, G, C, NW, STAGES>, (int)smem)) return e;
-    const int vec = D % 4 == 0 && ld % 4 == 0 && !((uintptr_t)proj & 15);
-    const dim3 grid(n_seqs, H, (D + DVT - 1) / DVT);
+        if (int e = acv_ensure_smem(cfg, delta_kernel<R, G, C, NW, STAGES, KD>, (int)smem)) return e;
+    const int vec = DV % 4 == 0 && ld % 4 == 0 && !((uintptr_t)values & 15);
+    const dim3 grid(n_seqs, H, (DV + DVT - 1) / DVT);
     if (grid.y > 65535 || grid.z > 65535) return ACV_ERR_SIZE;
-    acv_launch(PDL_ATTN, delta_kernel<R, G, C, NW, STAGES>, grid, NW * 32, smem, stream, rec, proj, ld, state, slots, cu_q,
-               first_block, o, H, D, vec);
+    acv_launch(PDL_ATTN, delta_kernel<R, G, C, NW, STAGES, KD>, grid, NW * 32, smem, stream, rec, values, ld, state, slots, cu_q,
+               first_block, o, H, D, DV, vec);
     return acv_launch_status();
 }
 
-// After acv_delta_blocks.  first_block: the number of each request's first block among the step's items; o: float [T][H*D];
-// state: float [slots][H][D][D]; heads of up to 512 channels.  form: 0, or a choice among the shapes of a block (timing).
-ACV_API int acv_delta(const float* rec, const float* proj, int ld, float* state, const int* slots, const int* cu_q,
-                      const int* first_block, float* o, int n_seqs, int H, int D, int form, cudaStream_t stream) {
-    if (n_seqs <= 0) return 0;
-    if (H <= 0 || D <= 0 || D > 512) return ACV_ERR_SIZE;
-    if ((uintptr_t)rec & 15) return ACV_ERR_ALIGN;
+template <bool KD>
+static int delta_by_size(const float* rec, const float* values, int ld, float* state, const int* slots, const int* cu_q,
+                         const int* first_block, float* o, int n_seqs, int H, int D, int DV, int form, cudaStream_t stream) {
 #define DL_CASE(RR, GG, CC, WW, SS) \
-    return launch_delta<RR, GG, CC, WW, SS>(rec, proj, ld, state, slots, cu_q, first_block, o, n_seqs, H, D, stream);
+    return launch_delta<RR, GG, CC, WW, SS, KD>(rec, values, ld, state, slots, cu_q, first_block, o, n_seqs, H, D, DV, stream);
     if (D <= 8) DL_CASE(8, 1, 1, 1, 3)
     if (D <= 16) DL_CASE(8, 2, 1, 1, 3)
     if (D <= 32) DL_CASE(8, 4, 1, 4, 3)
     // few columns for the device: four warps to sixteen columns; more: two warps, then one (fewer instructions a column)
-    const long long tiles = (long long)n_seqs * H * ((D + 15) / 16);
+    const long long tiles = (long long)n_seqs * H * ((DV + 15) / 16);
     if (D <= 64) {
         if (!form) form = tiles <= 180 ? 1 : tiles <= 600 ? 2 : 3;
         if (form == 1) DL_CASE(4, 16, 2, 4, 3)
@@ -550,6 +558,20 @@ ACV_API int acv_delta(const float* rec, const float* proj, int ld, float* state,
     if (D <= 256) DL_CASE(8, 32, 1, 4, 3)
     DL_CASE(16, 32, 1, 4, 2)
 #undef DL_CASE
+}
+
+// After acv_delta_blocks, or with `gated` after acv_gated_delta_blocks.  values: rows of `ld` floats whose first H*DV columns are
+// the values (DV = D unless gated); first_block: the number of each request's first block among the step's items; o: float
+// [T][H*DV]; state: float [slots][H][D][DV]; key heads of up to 512 channels.  form: 0, or a choice among the shapes of a
+// block (timing).
+ACV_API int acv_delta(const float* rec, const float* values, int ld, float* state, const int* slots, const int* cu_q,
+                      const int* first_block, float* o, int n_seqs, int H, int D, int DV, int gated, int form,
+                      cudaStream_t stream) {
+    if (n_seqs <= 0) return 0;
+    if (H <= 0 || D <= 0 || D > 512 || DV <= 0 || (!gated && DV != D)) return ACV_ERR_SIZE;
+    if ((uintptr_t)rec & 15) return ACV_ERR_ALIGN;
+    return gated ? delta_by_size<false>(rec, values, ld, state, slots, cu_q, first_block, o, n_seqs, H, D, DV, form, stream)
+                 : delta_by_size<true>(rec, values, ld, state, slots, cu_q, first_block, o, n_seqs, H, D, DV, form, stream);
 }
 
 // ----------------------------------------------------------------------------- one token a request, everything

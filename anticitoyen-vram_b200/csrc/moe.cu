@@ -20,7 +20,8 @@
 #define MOE_TILE 64          // rows of a tile of the grouped products (ops.MOE_TILE)
 
 // gated activation of an expert (ops.GLU_*)
-#define GLU_SWISH_CLAMPED 0  // g = min(a, limit), u = clamp(b, -limit, limit): g * sigmoid(alpha g) * (u + 1)
+#define GLU_SWISH_CLAMPED 0  // g = min(a, limit), u = clamp(b, -limit, limit): g * sigmoid(alpha g) * (u + shift), shift 1
+// (silu(a) * b is the same unit without limits, alpha 1 and shift 0)
 // acv_glu also takes 1, 2, 3: act(a) * b with act the plain activation of that number (gelu_tanh, silu, gelu)
 
 template <typename T> __device__ __forceinline__ float sigmoid_f32(float x);
@@ -28,10 +29,10 @@ template <> __device__ __forceinline__ float sigmoid_f32<float>(float x) { retur
 template <> __device__ __forceinline__ float sigmoid_f32<bf16>(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 template <typename T>
-__device__ __forceinline__ float glu_act(float a, float b, float limit, float alpha) {
+__device__ __forceinline__ float glu_act(float a, float b, float limit, float alpha, float shift = 1.f) {
     const float g = fminf(a, limit);
     const float u = fminf(fmaxf(b, -limit), limit);
-    return g * sigmoid_f32<T>(alpha * g) * (u + 1.f);
+    return g * sigmoid_f32<T>(alpha * g) * (u + shift);
 }
 
 // activation of an expert that has no gate: y = act(W_up x), out = W_down y  (ops.ACTIVATIONS)
@@ -47,12 +48,13 @@ __device__ __forceinline__ float plain_act(float z, int kind) {
 // scores in shared memory, E floats per warp.  ids/weights: [T, top].  gate_w (optional, [H]): the shared
 // expert's gate, sigmoid(<gate_w, h>), one number per token.
 // With z (float [T, ldz]) the logits come from a matrix product made before: columns 0..E-1 the router's, column E
-// the shared expert's gate (when gate is asked for); h and the weights are then not read.
+// the shared expert's gate (when gate is asked for); h and the weights are then not read.  r_bias (optional, [E]): joins the
+// logits that this kernel makes itself.
 template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ w_router,
                                  const float* __restrict__ gate_w, const float* __restrict__ z, int ldz, int T_tokens, int H,
                                  int E, int top, int softmax, int renorm, int* __restrict__ ids, float* __restrict__ weights,
-                                 float* __restrict__ gate, int n_groups, int keep_groups, float renorm_eps) {
+                                 float* __restrict__ gate, const float* __restrict__ r_bias, int n_groups, int keep_groups, float renorm_eps) {
     extern __shared__ float sm_all[];
     pdl_launch_dependents();
     pdl_wait();
@@ -70,7 +72,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int h_stride, const fl
             float d = 0.f;
             for (int k = lane; k < H; k += 32) d = fmaf(to_f32(row[k]), wr[k], d);
             d = warp_sum(d);
-            if (lane == 0) sc[e] = d;
+            if (lane == 0) sc[e] = r_bias ? d + r_bias[e] : d;
         }
         if (gate_w) {
             float d = 0.f;
@@ -159,7 +161,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, int h_stride, const fl
 
 ACV_API int acv_moe_route(const void* h, int h_stride, const float* w_router, const float* gate_w, const float* z, int ldz,
                           int T_tokens, int H, int E, int top, int softmax, int renorm, int* ids, float* weights, float* gate,
-                          int dtype, int n_groups, int keep_groups, float renorm_eps, cudaStream_t stream) {
+                          const float* r_bias, int dtype, int n_groups, int keep_groups, float renorm_eps, cudaStream_t stream) {
     if (T_tokens <= 0) return 0;
     if (E <= 0 || top <= 0 || top > E || E > 4096) return ACV_ERR_SIZE;
     if (n_groups < 1) n_groups = 1;
@@ -168,10 +170,10 @@ ACV_API int acv_moe_route(const void* h, int h_stride, const float* w_router, co
     const int grid = (T_tokens + MR_WARPS - 1) / MR_WARPS;
     if (dtype == ACV_F32)
         acv_launch(PDL_MISC, moe_route_kernel<float>, grid, MR_WARPS * 32, smem, stream, (const float*)h, h_stride, w_router,
-                   gate_w, z, ldz, T_tokens, H, E, top, softmax, renorm, ids, weights, gate, n_groups, keep_groups, renorm_eps);
+                   gate_w, z, ldz, T_tokens, H, E, top, softmax, renorm, ids, weights, gate, r_bias, n_groups, keep_groups, renorm_eps);
     else if (dtype == ACV_BF16)
         acv_launch(PDL_MISC, moe_route_kernel<bf16>, grid, MR_WARPS * 32, smem, stream, (const bf16*)h, h_stride, w_router,
-                   gate_w, z, ldz, T_tokens, H, E, top, softmax, renorm, ids, weights, gate, n_groups, keep_groups, renorm_eps);
+                   gate_w, z, ldz, T_tokens, H, E, top, softmax, renorm, ids, weights, gate, r_bias, n_groups, keep_groups, renorm_eps);
     else
         return ACV_ERR_DTYPE;
     return acv_launch_status();
@@ -296,7 +298,7 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_simt_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, long long w_expert_stride, int ldw,
                      void* __restrict__ C, int ldc, const int* __restrict__ grouped, const int* __restrict__ tile_expert,
-                     const float* __restrict__ row_weight, int top, int N, int K, float limit, float alpha, int pairs) {
+                     const float* __restrict__ row_weight, int top, int N, int K, float limit, float alpha, float shift, int pairs) {
     constexpr bool GLU = MODE == 1, GATHER = MODE != 0;
     __shared__ float As[16][MOE_TILE + 4];
     __shared__ float Ws[16][64 + 4];
@@ -366,7 +368,7 @@ moe_gemm_simt_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, 
             const int gn = n0 + tx * 4 + j;
             if (gn >= N) continue;
             if constexpr (GLU)
-                ((T*)C)[crow + gn] = from_f32<T>(glu_act<T>(acc[i][j] * w, acu[i][j] * w, limit, alpha));
+                ((T*)C)[crow + gn] = from_f32<T>(glu_act<T>(acc[i][j] * w, acu[i][j] * w, limit, alpha, shift));
             else if constexpr (MODE == 2)
                 ((T*)C)[crow + gn] = from_f32<T>(plain_act(acc[i][j] * w, pairs));
             else
@@ -379,13 +381,13 @@ moe_gemm_simt_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, 
 // (C of A's type; the activation's kind travels in `pairs`)
 ACV_API int acv_moe_gemm_simt(const void* A, int lda, const void* W, long long w_expert_stride, int ldw, void* C, int ldc,
                               const int* grouped, const int* tile_expert, const float* row_weight, int top, int max_tiles,
-                              int N, int K, int which, float limit, float alpha, int pairs, int dtype, cudaStream_t stream) {
+                              int N, int K, int which, float limit, float alpha, float shift, int pairs, int dtype, cudaStream_t stream) {
     if (max_tiles <= 0 || N <= 0) return 0;
     if (K <= 0 || top <= 0 || max_tiles > 65535) return ACV_ERR_SIZE;
     dim3 grid((N + 63) / 64, max_tiles);
 #define MG_LAUNCH(TT, G)                                                                                              \
     acv_launch(PDL_GEMM, moe_gemm_simt_kernel<TT, G>, grid, 256, 0, stream, (const TT*)A, lda, (const TT*)W,          \
-               w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, pairs)
+               w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, shift, pairs)
     if (dtype == ACV_F32) {
         if (which == 0) MG_LAUNCH(float, 1); else if (which == 2) MG_LAUNCH(float, 2); else MG_LAUNCH(float, 0);
     } else if (dtype == ACV_BF16) {
@@ -413,7 +415,7 @@ template <int MODE>
 __global__ void __launch_bounds__(MM_THREADS)
 moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const bf16* __restrict__ W, long long w_expert_stride, int ldw,
                     void* __restrict__ C, int ldc, const int* __restrict__ grouped, const int* __restrict__ tile_expert,
-                    const float* __restrict__ row_weight, int top, int N, int K, float limit, float alpha, int pairs) {
+                    const float* __restrict__ row_weight, int top, int N, int K, float limit, float alpha, float shift, int pairs) {
     extern __shared__ __align__(128) unsigned char mm_smem[];
     constexpr bool GLU = MODE == 1, GATHER = MODE != 0;
     constexpr int A_BYTES = MOE_TILE * MM_BK * 2;
@@ -519,7 +521,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const bf16* __restrict_
                 if (col >= N) continue;
                 const float v = acc[nt][half * 2 + e] * w;
                 if constexpr (GLU)
-                    ((bf16*)C)[crow + col] = __float2bfloat16_rn(glu_act<bf16>(v, acu[nt][half * 2 + e] * w, limit, alpha));
+                    ((bf16*)C)[crow + col] = __float2bfloat16_rn(glu_act<bf16>(v, acu[nt][half * 2 + e] * w, limit, alpha, shift));
                 else if constexpr (MODE == 2)
                     ((bf16*)C)[crow + col] = __float2bfloat16_rn(plain_act(v, pairs));
                 else
@@ -533,7 +535,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ A, int lda, const bf16* __restrict_
 // (C bfloat16; the activation's kind travels in `pairs`)
 ACV_API int acv_moe_gemm_mma(const void* A, int lda, const void* W, long long w_expert_stride, int ldw, void* C, int ldc,
                              const int* grouped, const int* tile_expert, const float* row_weight, int top, int max_tiles,
-                             int N, int K, int which, float limit, float alpha, int pairs, cudaStream_t stream) {
+                             int N, int K, int which, float limit, float alpha, float shift, int pairs, cudaStream_t stream) {
     if (max_tiles <= 0 || N <= 0) return 0;
     if (K <= 0 || top <= 0 || max_tiles > 65535) return ACV_ERR_SIZE;
     if ((K % 8) || (lda % 8) || (ldw % 8) || (w_expert_stride % 8) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return ACV_ERR_ALIGN;
@@ -543,7 +545,7 @@ ACV_API int acv_moe_gemm_mma(const void* A, int lda, const void* W, long long w_
         static AcvSmemConfig cfg;
         if (int rc = acv_ensure_smem(cfg, moe_gemm_mma_kernel<1>, smem)) return rc;
         acv_launch(PDL_GEMM, moe_gemm_mma_kernel<1>, grid, MM_THREADS, smem, stream, (const bf16*)A, lda, (const bf16*)W,
-                   w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, pairs);
+                   w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, shift, pairs);
     } else {
         const int smem = MM_STAGES * (MOE_TILE * MM_BK * 2 + MM_BN * MM_BK * 2);
         static AcvSmemConfig cfg;
@@ -551,12 +553,12 @@ ACV_API int acv_moe_gemm_mma(const void* A, int lda, const void* W, long long w_
             static AcvSmemConfig cfg2;
             if (int rc = acv_ensure_smem(cfg2, moe_gemm_mma_kernel<2>, smem)) return rc;
             acv_launch(PDL_GEMM, moe_gemm_mma_kernel<2>, grid, MM_THREADS, smem, stream, (const bf16*)A, lda, (const bf16*)W,
-                       w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, pairs);
+                       w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, shift, pairs);
             return acv_launch_status();
         }
         if (int rc = acv_ensure_smem(cfg, moe_gemm_mma_kernel<0>, smem)) return rc;
         acv_launch(PDL_GEMM, moe_gemm_mma_kernel<0>, grid, MM_THREADS, smem, stream, (const bf16*)A, lda, (const bf16*)W,
-                   w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, pairs);
+                   w_expert_stride, ldw, C, ldc, grouped, tile_expert, row_weight, top, N, K, limit, alpha, shift, pairs);
     }
     return acv_launch_status();
 }

@@ -70,8 +70,8 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_add_rmsnorm": [P, P, P, P, P, I, I, F, I, P],
         "acv_swiglu": [P, P, I, I, I, P],
         "acv_add_bias": [P, I, P, I, I, I, P],
-        "acv_qk_norm_rope_append": [P, I, I, I, I, I, P, P, F, P, I, I, P, P, P, I, P, P, P, I, I, I, I, F, P],
-        "acv_attention_generic": [P, I, P, I, P, P, P, P, P, I, P, I, I, I, I, I, I, F, I, I, I, I, P, P, P],
+        "acv_qk_norm_rope_append": [P, I, I, I, I, I, P, P, F, P, I, I, P, P, P, I, P, P, P, I, I, I, I, F, I, P],
+        "acv_attention_generic": [P, I, P, I, P, P, P, P, P, I, P, I, I, I, I, I, I, F, I, I, I, I, P, P, P, I, P],
         "acv_add_group_rmsnorm": [P, P, F, P, P, P, I, I, I, F, I, I, P],
         "acv_input_conv": [P, P, P, P, P, P, P, I, I, I, I, P, P],
         "acv_add_group_rmsnorm_conv": [P, P, F, P, P, P, P, P, I, I, I, F, I, I, I, P],
@@ -92,9 +92,13 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_retention_gate": [P, I, P, I, P, I, I, I, I, F, F, I, P, I, I, I, P],
         "acv_delta_blocks": [P, I, P, P, P, P, P, P, I, I, I, I, P],
         "acv_delta_record_floats": [I],
-        "acv_delta": [P, P, I, P, P, P, P, P, I, I, I, I, P],
+        "acv_delta": [P, P, I, P, P, P, P, P, I, I, I, I, I, I, P],
         "acv_delta_step_takes": [I, I],
         "acv_delta_step": [P, I, P, P, P, F, P, P, P, P, I, I, I, I, I, I, P],
+        "acv_gated_delta_record_floats": [I],
+        "acv_gated_delta_blocks": [P, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+        "acv_gated_delta_step_takes": [I, I],
+        "acv_gated_delta_step": [P, I, P, P, P, P, F, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
         "acv_gemm_simt": [P, I, P, I, P, I, I, I, I, I, I, P],
         "acv_gemm_simt_batched": [P, I, LL, P, I, LL, P, I, LL, I, I, I, I, I, I, P, I, LL, P],
         "acv_gemm_mma_batched_takes": [P, I, LL, P, I, LL, P, I, LL, I, I],
@@ -117,8 +121,8 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_gemm_tc_qkv": [P, I, P, I, P, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, I, I, I, P, P, F, P, I, P, P, P, I, P, P, P, I, I, P],
         "acv_gemm_tc": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P],
         "acv_gemm_tc_bias": [P, I, P, I, P, I, I, I, I, I, I, I, I, I, P, LL, P, LL, P, I, I, I, P, F, F, P],
-        "acv_attention_decode": [P, I, P, I, P, P, P, P, I, P, P, I, P, I, I, I, I, I, F, I, I, I, P, P, P, LL, LL, LL, I, I, I, I, P, P, P],
-        "acv_attention_tc": [P, I, I, P, I, P, P, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, I, P, I, P, P, P],
+        "acv_attention_decode": [P, I, P, I, P, P, P, P, I, P, P, I, P, I, I, I, I, I, F, I, I, I, P, P, P, LL, LL, LL, I, I, I, I, P, P, P, I, P],
+        "acv_attention_tc": [P, I, I, P, I, P, P, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, I, P, I, P, P, P, I, P],
         "acv_attention_chunk": [P, I, P, I, P, P, P, P, I, P, P, P, I, P, I, I, I, I, I, F, I, I, I, I, P],
         "acv_table_update": [P, I, I, P, I, P],
         "acv_embed_scaled": [P, P, P, I, I, I, F, I, P],
@@ -127,12 +131,12 @@ def _declare(lib: ctypes.CDLL) -> None:
         "acv_heads_norm_append": [P, P, I, P, P, I, I, I, I, I, I, I, P, P, F, P, P, P, I, P, P, P, I, I, I, P],
         "acv_diff_combine": [P, I, I, P, I, I, I, I, F, F, F, I, P],
         "acv_diff_attention_generic": [P, I, P, I, P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, I, F, F, F, I, P],
-        "acv_moe_route": [P, I, P, P, P, I, I, I, I, I, I, I, P, P, P, I, I, I, F, P],
+        "acv_moe_route": [P, I, P, P, P, I, I, I, I, I, I, I, P, P, P, P, I, I, I, F, P],
         "acv_moe_group": [P, I, I, I, I, P, P, P, P, P],
         "acv_moe_gather": [P, I, P, P, I, I, P, P, P, I, I, P],
-        "acv_gemm_tc_grouped": [P, I, P, I, P, I, I, I, I, I, P, P, I, I, P, F, F, I, P, I, I, P],
-        "acv_moe_gemm_simt": [P, I, P, LL, I, P, I, P, P, P, I, I, I, I, I, F, F, I, I, P],
-        "acv_moe_gemm_mma": [P, I, P, LL, I, P, I, P, P, P, I, I, I, I, I, F, F, I, P],
+        "acv_gemm_tc_grouped": [P, I, P, I, P, I, I, I, I, I, P, P, I, I, P, F, F, F, I, P, I, I, P],
+        "acv_moe_gemm_simt": [P, I, P, LL, I, P, I, P, P, P, I, I, I, I, I, F, F, F, I, I, P],
+        "acv_moe_gemm_mma": [P, I, P, LL, I, P, I, P, P, P, I, I, I, I, I, F, F, F, I, P],
         "acv_moe_combine": [P, I, I, P, I, P, I, P, P, I, I, I, I, P],
         "acv_glu": [P, I, P, I, I, I, I, F, F, I, I, P],
         "acv_gemm_tc_glu": [P, I, P, I, P, I, I, I, I, F, F, I, P, I, I, I, P],
@@ -301,13 +305,14 @@ def qk_norm_rope_append(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, he
                         cos_sin: torch.Tensor | None, positions: torch.Tensor, seq_of_token: torch.Tensor,
                         block_table: torch.Tensor | None, k_pages: torch.Tensor | None,
                         v_pages: torch.Tensor | None, table_rows: torch.Tensor | None = None, value_dim: int = 0,
-                        v_scale: float = 1.0) -> None:
+                        v_scale: float = 1.0, tied: bool = False) -> None:
     """Per-head norm, rotation and cache append over the stacked projection qkv [T, (NH+2NKV)*D], in place.
 
     cos_sin float32 [positions, R] (cos of R/2 angles, then sin); pages [NP, NKV, page, D].  ``table_rows``
     (int32 [requests], optional): the row of ``block_table`` of each request of the batch (default: its index).
     ``value_dim`` > 0: value rows of that size (the row is [NH*D | NKV*D | NKV*value_dim], value pages
-    [NP, NKV, page, value_dim]); ``v_scale``: a constant on the values as they enter their pages."""
+    [NP, NKV, page, value_dim]); ``v_scale``: a constant on the values as they enter their pages.  ``tied``: the row is
+    [NH*D | NKV*D]; a head's value is its key as projected, before norm and rotation."""
     _need_cuda(qkv)
     T = qkv.shape[0]
     rot = cos_sin.shape[1] if cos_sin is not None else 0
@@ -318,7 +323,7 @@ def qk_norm_rope_append(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, he
     _check(library().acv_qk_norm_rope_append(
         _p(qkv), qkv.stride(0), T, num_heads, num_kv_heads, head_dim, _p(q_weight), _p(k_weight), eps, _p(cos_sin),
         rot, rows, _p(positions), _p(seq_of_token), _p(block_table), bts, _p(table_rows), _p(k_pages), _p(v_pages), page, n_pages,
-        dtype_code(qkv.dtype), int(value_dim), float(v_scale), _stream()), "qk_norm_rope_append")
+        dtype_code(qkv.dtype), int(value_dim), float(v_scale), 1 if tied else 0, _stream()), "qk_norm_rope_append")
 
 
 def _head_vectors(num_heads: int, *vectors) -> None:
@@ -327,24 +332,33 @@ def _head_vectors(num_heads: int, *vectors) -> None:
             raise KernelError("attention: sinks and slopes are contiguous float32 vectors with one number per query head")
 
 
+def _gate_args(gate: torch.Tensor | None, out: torch.Tensor):
+    if gate is None:
+        return None, 0
+    if gate.shape != out.shape or gate.stride(1) != 1 or gate.dtype != out.dtype or not gate.is_cuda:
+        raise KernelError("attention: the output gate is a view of the result's shape and type with dense rows")
+    return _p(gate), gate.stride(0)
+
+
 def attention_generic(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                       positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor,
                       num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: int = 0,
                       table_rows: torch.Tensor | None = None, value_dim: int = 0, keep_first: int = 0,
-                      sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> torch.Tensor:
+                      sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
+                      gate: torch.Tensor | None = None) -> torch.Tensor:
     """Paged causal attention for every token of the step.  q: rows of num_heads*head_dim (row stride free).
     ``value_dim`` > 0: value rows (and the result's heads) of that size; ``keep_first``: the first keys of a request
     that stay visible behind the window.  ``sinks`` (float32 [num_heads]): exp(sink_h) joins the softmax's denominator
     (a score with no key and no value); ``slopes`` (float32 [num_heads]): slope_h * (i - j) is taken off the score of
-    query i and key j."""
+    query i and key j.  ``gate`` (a view like ``out``): the result is multiplied by sigmoid(gate) in float."""
     _need_cuda(q, out, k_pages)
     _head_vectors(num_heads, sinks, slopes)
     T = q.shape[0]
     _check(library().acv_attention_generic(
         _p(q), q.stride(0), _p(out), out.stride(0), _p(k_pages), _p(v_pages), _p(positions), _p(seq_of_token),
         _p(block_table), block_table.stride(0), _p(table_rows), T, num_heads, num_kv_heads, head_dim, k_pages.shape[2],
-        k_pages.shape[0], scale, window, dtype_code(q.dtype), int(value_dim), int(keep_first), _p(sinks), _p(slopes), _stream()),
-           "attention_generic")
+        k_pages.shape[0], scale, window, dtype_code(q.dtype), int(value_dim), int(keep_first), _p(sinks), _p(slopes), *_gate_args(gate, out),
+        _stream()), "attention_generic")
     return out
 
 
@@ -766,9 +780,10 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, 
                      block_table: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                      window: int, n_splits: int, max_kv: int = 0, cluster_merge: bool = True,
                      table_rows: torch.Tensor | None = None, chunk: int = 0, keep_first: int = 0,
-                     sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> torch.Tensor:
+                     sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
+                     gate: torch.Tensor | None = None) -> torch.Tensor:
     """Attention of requests that bring one token each, over their pages, split over the context.
-    ``sinks``, ``slopes`` (float32 [heads]): as in ``attention_generic``; the sink joins once, where the splits merge.
+    ``sinks``, ``slopes`` (float32 [heads]), ``gate``: as in ``attention_generic``; the sink joins once, where the splits merge.
 
     Up to 8 splits are merged inside a thread-block cluster (through its shared memory); more, or
     ``cluster_merge=False``, go through partial results in scratch memory and a last-arriver merge."""
@@ -782,7 +797,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, 
         _p(kv_len), _p(block_table), block_table.stride(0), _p(table_rows), num_heads, num_kv_heads, head_dim,
         k_pages.shape[2], k_pages.shape[0], scale, window, chunk, n_splits, _p(acc), _p(ml), _p(cnt), acc.numel(), ml.numel(), cnt.numel(),
         max_kv or block_table.shape[1] * k_pages.shape[2], 1 if use_cluster else 0,
-        1 if out.dtype == torch.float32 else 0, int(keep_first), _p(sinks), _p(slopes), _stream()), "attention_decode")
+        1 if out.dtype == torch.float32 else 0, int(keep_first), _p(sinks), _p(slopes), *_gate_args(gate, out), _stream()),
+           "attention_decode")
     return out
 
 
@@ -804,16 +820,17 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pa
                  tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, cu_q: torch.Tensor, kv_len: torch.Tensor,
                  block_table: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                  window: int, table_rows: torch.Tensor | None = None, chunk: int = 0, keep_first: int = 0,
-                 sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> torch.Tensor:
+                 sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
+                 gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of portions of prompts on tcgen05 (tiles of QUERY_TILE query tokens, pages by TMA).
-    ``sinks``, ``slopes`` (float32 [heads]): as in ``attention_generic``."""
+    ``sinks``, ``slopes`` (float32 [heads]), ``gate``: as in ``attention_generic``."""
     _head_vectors(num_heads, sinks, slopes)
     _, _, status = _gemm_buffers(q.device, 0, 0)
     _check(library().acv_attention_tc(
         _p(q), q.stride(0), q.shape[0], _p(out), out.stride(0), _p(k_pages), _p(v_pages), _p(tile_seq), _p(tile_q0),
         n_tiles, _p(cu_q), _p(kv_len), _p(block_table), block_table.stride(0), _p(table_rows), num_heads, num_kv_heads,
         head_dim, k_pages.shape[2], k_pages.shape[0], scale, window, chunk, 1 if out.dtype == torch.float32 else 0, _p(status),
-        int(keep_first), _p(sinks), _p(slopes), _stream()), "attention_tc")
+        int(keep_first), _p(sinks), _p(slopes), *_gate_args(gate, out), _stream()), "attention_tc")
     return out
 
 
@@ -871,13 +888,15 @@ def attention_work_decode(padded: int, max_kv: int) -> tuple[dict, dict]:
 def attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, ctx,
               block_table: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
               window: int = 0, work: dict | None = None, chunk: int = 0, value_dim: int = 0,
-              keep_first: int = 0, sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None) -> torch.Tensor:
+              keep_first: int = 0, sinks: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
+              gate: torch.Tensor | None = None) -> torch.Tensor:
     """Attention of every token of the step over its request's pages.  A query sees the keys at or before its
     position; with ``window`` > 0 the last ``window`` of them, and with ``keep_first`` > 0 also the first
     ``keep_first`` keys of the request; with ``chunk`` > 0 those of its own chunk of ``chunk``
     positions counted from the request's position 0.  ``value_dim``: the size of a value row where it is not ``head_dim``.
     ``sinks`` (float32 [heads]): exp(sink_h) joins the softmax's denominator; ``slopes`` (float32 [heads]): the score of
-    query i and key j loses slope_h (i - j).
+    query i and key j loses slope_h (i - j).  ``gate`` (a view like ``out``): the result times sigmoid(gate), in float, as
+    it leaves the kernel.
 
     ``qkv`` is the stacked projection after norm and rotation (queries are its first
     num_heads*head_dim columns); ``ctx`` is the step's StepContext; ``work`` the step's work lists
@@ -897,7 +916,10 @@ def attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pag
     if not generic and keep_first > 0 and (chunk > 0 or (w["n_tiles"] and not attention_tc_takes(qkv, out, k_pages, head_dim))):
         generic = True
     # sinks and slopes: the generic, the split-KV and the tcgen05 portion kernel know them, the mma.sync portion kernel does not
-    if not generic and (sinks is not None or slopes is not None) and (chunk > 0 or (
+    # (likewise an output gate, which the portion kernel reads in 16-byte pieces)
+    if not generic and gate is not None and (gate.stride(0) % 8 or gate.data_ptr() % 16):
+        generic = True
+    if not generic and (sinks is not None or slopes is not None or gate is not None) and (chunk > 0 or (
             w["n_tiles"] and not attention_tc_takes(qkv, out, k_pages, head_dim))):
         generic = True
     if generic:
@@ -905,7 +927,7 @@ def attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pag
             raise KernelError("attention: the chunked mask is built for the tensor-core kernels' sizes only")
         return attention_generic(qkv, out, k_pages, v_pages, ctx.positions, ctx.seq_of_token, block_table, num_heads,
                                  num_kv_heads, head_dim, scale, window, table_rows=rows, value_dim=value_dim,
-                                 keep_first=keep_first, sinks=sinks, slopes=slopes)
+                                 keep_first=keep_first, sinks=sinks, slopes=slopes, gate=gate)
     if w["n_dec"]:
         kv = min(w["max_dec_kv"], window + keep_first) if window > 0 else w["max_dec_kv"]
         kv = min(kv, chunk) if chunk > 0 else kv
@@ -914,11 +936,11 @@ def attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pag
         attention_decode(qkv, out, k_pages, v_pages, w["dec_tokens"], w["dec_seqs"], w["n_dec"], ctx.kv_len,
                          block_table, num_heads, num_kv_heads, head_dim, scale, window, n_splits, w["max_dec_kv"],
                          cluster_merge=in_clusters, table_rows=rows, chunk=chunk, keep_first=keep_first, sinks=sinks,
-                         slopes=slopes)
+                         slopes=slopes, gate=gate)
     if w["n_tiles"] and attention_tc_takes(qkv, out, k_pages, head_dim):
         attention_tc(qkv, out, k_pages, v_pages, w["tile_seq"], w["tile_q0"], w["n_tiles"], ctx.cu_q, ctx.kv_len,
                      block_table, num_heads, num_kv_heads, head_dim, scale, window, table_rows=rows, chunk=chunk,
-                     keep_first=keep_first, sinks=sinks, slopes=slopes)
+                     keep_first=keep_first, sinks=sinks, slopes=slopes, gate=gate)
     elif w["n_tiles"]:
         attention_chunk(qkv, out, k_pages, v_pages, w["tile_seq"], w["tile_q0"], w["n_tiles"], ctx.cu_q, ctx.kv_len,
                         block_table, num_heads, num_kv_heads, head_dim, scale, window, table_rows=rows,
@@ -1134,6 +1156,7 @@ def diff_combine(maps: torch.Tensor, out: torch.Tensor, num_heads: int, value_di
 # ----------------------------------------------------------------------------- mixture of experts
 MOE_TILE = 64               # rows of a tile of the grouped products (MOE_TILE of csrc/moe.cu)
 GLU_SWISH_CLAMPED = 0       # g = min(a, limit), u = clamp(b, +-limit): g * sigmoid(alpha g) * (u + 1)
+SWIGLU_UNIT = (float("inf"), 1.0, 0.0)      # (limit, alpha, shift) with which g * sigmoid(alpha g) * (u + shift) is silu(a) * b
 
 
 MOE_TC_TILE = 128           # rows of a tile of the grouped tcgen05 product (GT_BM of csrc/gemm_epilogue.cuh)
@@ -1149,12 +1172,14 @@ def moe_max_tiles(rows: int, experts: int, tile: int = MOE_TILE) -> int:
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor | None, gate_w: torch.Tensor | None, top: int, softmax: bool, renorm: bool,
               ids: torch.Tensor, weights: torch.Tensor, gate: torch.Tensor | None, logits: torch.Tensor | None = None,
-              experts: int | None = None, groups: tuple[int, int] | None = None, renorm_eps: float = 0.0) -> None:
+              experts: int | None = None, groups: tuple[int, int] | None = None, renorm_eps: float = 0.0,
+              router_bias: torch.Tensor | None = None) -> None:
     """Router of a mixture of experts, in 32-bit: ids, weights [T, top] (int32, float32); gate [T] = sigmoid(h . gate_w).
     With ``logits`` (float32 [T, >= experts (+ 1)]: the router's columns, then the gate's) the products were made before
     and only the scores and the choice are made here.  ``groups`` = (count, keep): the experts stand in ``count`` equal
     groups of neighbours, a group is worth its best score, and only experts of the ``keep`` best groups can be chosen.
-    ``renorm_eps`` joins the sum that the chosen scores are divided by."""
+    ``renorm_eps`` joins the sum that the chosen scores are divided by.  ``router_bias`` (float32 [experts]): joins the logits
+    that are made here (logits made before hold it already)."""
     _need_cuda(h, ids, weights)
     T, H = h.shape
     n_groups, keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
@@ -1162,13 +1187,13 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor | None, gate_w: torch.Tens
         if logits.dtype != torch.float32 or logits.stride(1) != 1 or experts is None:
             raise KernelError("moe_route: float32 logits and the number of experts are wanted")
         _check(library().acv_moe_route(None, 0, None, None, _p(logits), logits.stride(0), T, H, experts, top, int(softmax),
-                                       int(renorm), _p(ids), _p(weights), _p(gate), dtype_code(h.dtype), n_groups, keep, float(renorm_eps),
+                                       int(renorm), _p(ids), _p(weights), _p(gate), None, dtype_code(h.dtype), n_groups, keep, float(renorm_eps),
                                        _stream()), "moe_route")
         return
     if w_router.dtype != torch.float32 or not w_router.is_contiguous() or h.stride(1) != 1:
         raise KernelError("moe_route: a contiguous float32 router matrix is wanted")
     _check(library().acv_moe_route(_p(h), h.stride(0), _p(w_router), _p(gate_w), None, 0, T, H, w_router.shape[0], top,
-                                   int(softmax), int(renorm), _p(ids), _p(weights), _p(gate), dtype_code(h.dtype), n_groups, keep,
+                                   int(softmax), int(renorm), _p(ids), _p(weights), _p(gate), _p(router_bias), dtype_code(h.dtype), n_groups, keep,
                                    float(renorm_eps), _stream()), "moe_route")
 
 
@@ -1198,10 +1223,10 @@ def moe_gather(h: torch.Tensor, grouped: torch.Tensor, weights: torch.Tensor | N
 
 def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_expert: torch.Tensor, tiles_used: torch.Tensor,
                     glu: bool = False, row_scale: torch.Tensor | None = None, limit: float = 0.0, alpha: float = 0.0,
-                    unary: str | None = None) -> torch.Tensor:
+                    unary: str | None = None, shift: float = 1.0) -> torch.Tensor:
     """The experts' products on tcgen05: x [tiles * 128, K] holds the rows in grouped order, w [E, N, K] the experts'
     matrices; out [rows, N] (bfloat16 or float32), or with ``glu`` [rows, N / 2] bfloat16: w's rows come in (gate, up) pairs
-    and go through the clamped gated unit, the accumulators times ``row_scale[row]`` first.  Without ``glu``:
+    and go through the gated unit g * sigmoid(alpha g) * (u + shift) with its clamps, the accumulators times ``row_scale[row]`` first.  Without ``glu``:
     ``row_scale`` multiplies a row's accumulators, and ``unary`` (a name of ``ACTIVATIONS`` other than the first) is then
     applied to every output, in float."""
     _need_cuda(x, w, out, tile_expert, tiles_used)
@@ -1217,7 +1242,7 @@ def gemm_tc_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_ex
     _check(library().acv_gemm_tc_grouped(_p(x), x.stride(0), _p(w), K, _p(out), out.stride(0), M, N, K, E, _p(tile_expert),
                                          _p(tiles_used), 1 if out.dtype == torch.float32 else 0,
                                          2 if glu else ((ACTIVATIONS[unary] << 4) if unary else 0),
-                                         _p(row_scale), limit, alpha, bn, _p(status), sm_count(x.device), 8, _stream()),
+                                         _p(row_scale), limit, alpha, shift, bn, _p(status), sm_count(x.device), 8, _stream()),
            "gemm_tc_grouped")
     return out
 
@@ -1233,7 +1258,7 @@ def _moe_which(glu: bool, plain_act: str | None, pairs) -> tuple[int, int]:
 
 def moe_gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, grouped: torch.Tensor, tile_expert: torch.Tensor,
                   row_weight: torch.Tensor | None, top: int, glu: bool, limit: float = 0.0, alpha: float = 0.0,
-                  pairs: bool = False, plain_act: str | None = None) -> torch.Tensor:
+                  pairs: bool = False, plain_act: str | None = None, shift: float = 1.0) -> torch.Tensor:
     """The experts' products over the grouped rows on the CUDA cores, 32-bit accumulation.  ``pairs``: with ``glu``, the
     rows of w are (gate, up) pairs instead of all gate rows followed by all up rows.  ``plain_act`` (a name of
     ``ACTIVATIONS``; not with ``glu``): experts without a gate: w [E, N, K], a [T, K] the tokens, out
@@ -1251,7 +1276,7 @@ def moe_gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, grouped: 
         raise KernelError(f"moe_gemm_simt: shapes {tuple(a.shape)} x {tuple(w.shape)} -> {tuple(out.shape)} do not fit")
     _check(library().acv_moe_gemm_simt(_p(a), a.stride(0), _p(w), w.stride(0), w.stride(1), _p(out), out.stride(0),
                                        _p(grouped), _p(tile_expert), _p(row_weight), top, tile_expert.numel(), N, K,
-                                       which, limit, alpha, int(pairs), dtype_code(a.dtype), _stream()), "moe_gemm_simt")
+                                       which, limit, alpha, shift, int(pairs), dtype_code(a.dtype), _stream()), "moe_gemm_simt")
     return out
 
 
@@ -1264,7 +1289,7 @@ def moe_gemm_mma_takes(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 def moe_gemm_mma(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, grouped: torch.Tensor, tile_expert: torch.Tensor,
                  row_weight: torch.Tensor | None, top: int, glu: bool, limit: float = 0.0, alpha: float = 0.0,
-                 pairs: bool = False, plain_act: str | None = None) -> torch.Tensor:
+                 pairs: bool = False, plain_act: str | None = None, shift: float = 1.0) -> torch.Tensor:
     """``moe_gemm_simt`` on the tensor cores (bfloat16 operands, float accumulators; the same arguments)."""
     _need_cuda(a, w, out, grouped, tile_expert)
     E, NW, K = w.shape
@@ -1274,19 +1299,19 @@ def moe_gemm_mma(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, grouped: t
         raise KernelError(f"moe_gemm_mma: shapes {tuple(a.shape)} x {tuple(w.shape)} -> {tuple(out.shape)} do not fit")
     _check(library().acv_moe_gemm_mma(_p(a), a.stride(0), _p(w), w.stride(0), w.stride(1), _p(out), out.stride(0),
                                       _p(grouped), _p(tile_expert), _p(row_weight), top, tile_expert.numel(), N, K,
-                                      which, limit, alpha, int(pairs), _stream()), "moe_gemm_mma")
+                                      which, limit, alpha, shift, int(pairs), _stream()), "moe_gemm_mma")
     return out
 
 
 def moe_experts_up(h: torch.Tensor, gate_up: torch.Tensor, act: torch.Tensor, grouped: torch.Tensor, tile_expert: torch.Tensor,
                    row_weight: torch.Tensor | None, top: int, limit: float, alpha: float, pairs: bool = False,
-                   plain_act: str | None = None) -> torch.Tensor:
+                   plain_act: str | None = None, shift: float = 1.0) -> torch.Tensor:
     """act[grouped row] = gated activation of the row's expert's gate and up products of its token (with ``plain_act``:
     that activation of the expert's one up product); dispatch by shape."""
     glu = plain_act is None
     if moe_gemm_mma_takes(h, gate_up):
-        return moe_gemm_mma(h, gate_up, act, grouped, tile_expert, row_weight, top, glu, limit, alpha, pairs, plain_act)
-    return moe_gemm_simt(h, gate_up, act, grouped, tile_expert, row_weight, top, glu, limit, alpha, pairs, plain_act)
+        return moe_gemm_mma(h, gate_up, act, grouped, tile_expert, row_weight, top, glu, limit, alpha, pairs, plain_act, shift)
+    return moe_gemm_simt(h, gate_up, act, grouped, tile_expert, row_weight, top, glu, limit, alpha, pairs, plain_act, shift)
 
 
 def moe_experts_down(act: torch.Tensor, down: torch.Tensor, out: torch.Tensor, grouped: torch.Tensor, tile_expert: torch.Tensor,
@@ -2029,17 +2054,20 @@ def delta_blocks(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, cu_q:
     return rec
 
 
-def delta(rec: torch.Tensor, proj: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor, num_seqs: int,
-          out: torch.Tensor, num_heads: int, dim: int, work: dict, form: int = 0) -> torch.Tensor:
+def delta(rec: torch.Tensor, values: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor, num_seqs: int,
+          out: torch.Tensor, num_heads: int, dim: int, work: dict, value_dim: int = 0, gated: bool = False, form: int = 0) -> torch.Tensor:
     """S = diag(w) S - (a u) (u^T S) + k v^T, o = S^T r along each request's tokens, per head, over the records of
-    ``delta_blocks`` (and the values in ``proj``); state float32 [slots, heads, dim, dim], out float32 [T, heads * dim].
-    Heads of up to 512 channels.  ``form``: a choice among the kernel's block shapes (0: by the sizes)."""
-    _need_cuda(rec, proj, state, out)
+    ``delta_blocks`` and the ``values`` (a view [T, heads * dim] with dense rows); state float32 [slots, heads, dim, dim], out
+    float32 [T, heads * dim].  ``gated``: over the records of ``gated_delta_blocks`` and its values of ``value_dim`` elements.
+    Key heads of up to 512 channels.  ``form``: a choice among the kernel's block shapes (0: by the sizes)."""
+    _need_cuda(rec, values, state, out)
+    dv = value_dim or dim
     if state.dtype != torch.float32 or not state.is_contiguous() or out.dtype != torch.float32 or not out.is_contiguous() \
-            or state.shape[1:] != (num_heads, dim, dim) or out.shape != (proj.shape[0], num_heads * dim) or not rec.is_contiguous():
-        raise KernelError("delta: a float32 state [slots, heads, dim, dim] and output [T, heads * dim] are wanted")
-    _check(library().acv_delta(_p(rec), _p(proj), proj.stride(0), _p(state), _p(slots), _p(cu_q), _p(work["first_block"]), _p(out),
-                               num_seqs, num_heads, dim, form, _stream()), "delta")
+            or state.shape[1:] != (num_heads, dim, dv) or out.shape != (values.shape[0], num_heads * dv) or not rec.is_contiguous() \
+            or values.dtype != torch.float32 or values.stride(1) != 1 or values.shape[1] != num_heads * dv:
+        raise KernelError("delta: float32 values and output [T, heads * value_dim] and a float32 state [slots, heads, dim, value_dim] are wanted")
+    _check(library().acv_delta(_p(rec), _p(values), values.stride(0), _p(state), _p(slots), _p(cu_q), _p(work["first_block"]), _p(out),
+                               num_seqs, num_heads, dim, dv, 1 if gated else 0, form, _stream()), "delta")
     return out
 
 
@@ -2065,5 +2093,61 @@ def general_delta(proj: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor, weig
         return out
     rec = delta_blocks(proj, w2_t, w0, cu_q, num_heads, dim, work)
     o = torch.empty((T, I), device=proj.device, dtype=torch.float32)
-    delta(rec, proj, state, slots, cu_q, num_seqs, o, num_heads, dim, work)
+    delta(rec, proj[:, 2 * I:3 * I], state, slots, cu_q, num_seqs, o, num_heads, dim, work)
     return retention_gate(o, proj[:, 4 * I:5 * I], out, num_heads, dim, eps, weight=weight, gate_fn="sigmoid")
+
+
+# ----------------------------------------------------------------------------- a gated delta rule behind a short convolution
+def gated_delta_blocks(proj: torch.Tensor, taps_t: torch.Tensor, rate: torch.Tensor, shift: torch.Tensor, ring: torch.Tensor,
+                       slots: torch.Tensor, positions: torch.Tensor, cu_q: torch.Tensor, num_seqs: int, num_heads: int,
+                       num_kv_heads: int, dim: int, value_dim: int, work: dict) -> tuple[torch.Tensor, torch.Tensor]:
+    """Everything in the gated delta recurrence that does not need the state, for every block of ``delta_work``: from a token's
+    row of the input product [q | k | v | z | b | a] (float32) the block's record (csrc/gated_delta.cu), float32 [blocks, heads,
+    record], and the values behind convolution and silu, float32 [T, heads * value_dim].  ``taps_t``: float32 [K, channels of
+    q, k and v]; ``ring``: float32 [slots, K, channels], the convolution's kept inputs, position p in row p mod K."""
+    _need_cuda(proj, taps_t, rate, shift, ring)
+    I = num_heads * value_dim
+    C = 2 * num_kv_heads * dim + I
+    K = taps_t.shape[0]
+    if any(t.dtype != torch.float32 for t in (proj, taps_t, rate, shift, ring)) or proj.stride(1) != 1 or taps_t.shape != (K, C) \
+            or not taps_t.is_contiguous() or not ring.is_contiguous() or ring.shape[1:] != (K, C) or proj.shape[1] < C + I + 2 * num_heads:
+        raise KernelError("gated_delta_blocks: float32 rows [q | k | v | z | b | a], taps [K, channels] and a ring [slots, K, channels] are wanted")
+    lib = library()
+    rec = torch.empty((work["n_items"], num_heads, lib.acv_gated_delta_record_floats(dim)), device=proj.device, dtype=torch.float32)
+    values = torch.empty((proj.shape[0], I), device=proj.device, dtype=torch.float32)
+    _check(lib.acv_gated_delta_blocks(_p(proj), proj.stride(0), _p(taps_t), _p(rate), _p(shift), _p(ring), _p(slots), _p(positions),
+                                      _p(work["seg_seq"]), _p(work["seg_idx"]), _p(cu_q), _p(values), _p(rec), work["n_items"],
+                                      num_seqs, num_kv_heads, num_heads, dim, value_dim, K, _stream()), "gated_delta_blocks")
+    return rec, values
+
+
+def gated_delta(proj: torch.Tensor, taps_t: torch.Tensor, rate: torch.Tensor, shift: torch.Tensor, weight: torch.Tensor, eps: float,
+                ring: torch.Tensor, ring_slots: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor,
+                cu_q: torch.Tensor, num_seqs: int, max_q_len: int, out: torch.Tensor, num_heads: int, num_kv_heads: int, dim: int,
+                value_dim: int, work: dict | None) -> torch.Tensor:
+    """From the input product (``gated_delta_blocks``) to the gated heads: every head's o of the recurrence to unit RMS
+    (``eps``), times ``weight`` (float32 [heads * value_dim]), times silu(z), into ``out`` (a view [T, heads * value_dim] with
+    dense rows); ``state`` float32 [slots, heads, dim, value_dim].  Steps in which every request brings one token are one
+    launch; others blocks, recurrence and gate (``work``: the step's ``delta_work``)."""
+    _need_cuda(proj, taps_t, weight, state, ring, out)
+    T, I = out.shape
+    C = 2 * num_kv_heads * dim + I
+    if weight.dtype != torch.float32 or weight.numel() != I or not weight.is_contiguous() or out.stride(1) != 1:
+        raise KernelError("gated_delta: a float32 weight over all heads and an output with dense rows are wanted")
+    lib = library()
+    if max_q_len == 1 and T == num_seqs and lib.acv_gated_delta_step_takes(dim, value_dim):
+        K = taps_t.shape[0]
+        if any(t.dtype != torch.float32 for t in (proj, taps_t, rate, shift, ring, state)) or proj.stride(1) != 1 \
+                or taps_t.shape != (K, C) or not taps_t.is_contiguous() or not ring.is_contiguous() or ring.shape[1:] != (K, C) \
+                or not state.is_contiguous() or state.shape[1:] != (num_heads, dim, value_dim):
+            raise KernelError("gated_delta: float32 projections, taps, ring and state are wanted")
+        _check(lib.acv_gated_delta_step(_p(proj), proj.stride(0), _p(taps_t), _p(rate), _p(shift), _p(weight), float(eps), _p(ring),
+                                        _p(ring_slots), _p(state), _p(slots), _p(positions), _p(cu_q), _p(out), out.stride(0),
+                                        num_seqs, num_kv_heads, num_heads, dim, value_dim, K, dtype_code(out.dtype), _stream()),
+               "gated_delta_step")
+        return out
+    rec, values = gated_delta_blocks(proj, taps_t, rate, shift, ring, ring_slots, positions, cu_q, num_seqs, num_heads,
+                                     num_kv_heads, dim, value_dim, work)
+    o = torch.empty((T, I), device=proj.device, dtype=torch.float32)
+    delta(rec, values, state, slots, cu_q, num_seqs, o, num_heads, dim, work, value_dim=value_dim, gated=True)
+    return retention_gate(o, proj[:, C:C + I], out, num_heads, value_dim, eps, weight=weight, gate_fn="silu")

@@ -15,6 +15,7 @@ from . import redudra  # noqa: F401  (registers Redudra)
 from . import nizedra  # noqa: F401  (registers Nizedra)
 from . import vadelix  # noqa: F401  (registers Vadelix)
 from . import lodalix  # noqa: F401  (registers Lodalix)
+from . import zogapel  # noqa: F401  (registers Zogapel)
 from .decoder import DecoderModel
 
 __all__ = ["DecoderModel", "build_from_folder", "build_random", "needs_of_plan", "plan_of_folder"]

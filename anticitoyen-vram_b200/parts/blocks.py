@@ -345,6 +345,11 @@ class SandwichBlock:
         parts = [n for _, n in self._norms()] + [self.mixer, self.feed_forward]
         return sum(p.weight_bytes() for p in parts if p is not None)
 
+    def step_weight_bytes(self, num_tokens: int) -> int:
+        parts = [n for _, n in self._norms()] + [self.mixer, self.feed_forward]
+        return sum(p.step_weight_bytes(num_tokens) if hasattr(p, "step_weight_bytes") else p.weight_bytes()
+                   for p in parts if p is not None)
+
     def flops(self, num_tokens: int) -> float:
         return self.mixer.flops(num_tokens) + (self.feed_forward.flops(num_tokens) if self.feed_forward is not None else 0.0)
 

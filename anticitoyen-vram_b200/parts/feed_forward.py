@@ -133,16 +133,19 @@ class RoutedExperts(FeedForward):
     name of ``ops.ACTIVATIONS`` ("gelu": the exact one, with erf), no clamps; ``groups`` = (count, keep): the experts stand in
     ``count`` equal groups of neighbours, a group is worth its best score, and only experts of the ``keep`` best groups can
     be chosen; ``renorm_eps`` joins the sum that the chosen scores are divided by; ``shared_gate`` False: the shared
-    expert's output is added as it is (no tensor shared.sg).
+    expert's output is added as it is (no tensor shared.sg); ``expert_unit`` "silu": the gated unit is
+    silu(W_gate x) * (W_up x), without clamps, slope or the 1 beside u; ``router_bias``: z = W_r h + b (tensor router.b).
+    (Softmax scores divided by the chosen ones' sum are the softmax over the chosen logits alone.)
 
     The step is the same launches whatever the routing is (rows grouped by expert on the device, tiles that belong
     to no expert return at once), so it runs inside a captured graph.  Tensors behind ``prefix``: router, e<i>.gate,
     e<i>.up, e<i>.down, shared.gate, shared.up, shared.down, shared.sg."""
 
-    def __init__(self, hidden_size: int, experts: int, top: int, expert_ff: int, expert_limit: float, shared_ff: int = 0,
+    def __init__(self, hidden_size: int, experts: int, top: int, expert_ff: int, expert_limit: float = 0.0, shared_ff: int = 0,
                  shared_limit: float = 0.0, alpha: float = 1.702, scoring: str = "sigmoid", renormalize: bool = False,
                  weight_on: str = "input", prefix: str = "mlp.", expert_form: str = "glu", activation: str | None = None,
-                 groups: tuple | None = None, renorm_eps: float = 0.0, shared_gate: bool = True) -> None:
+                 groups: tuple | None = None, renorm_eps: float = 0.0, shared_gate: bool = True,
+                 expert_unit: str = "swish_clamped", router_bias: bool = False) -> None:
         if scoring not in ("sigmoid", "softmax"):
             raise ValueError(f"router scoring '{scoring}' is not built (sigmoid and softmax are)")
         if weight_on not in ("input", "output"):
@@ -151,7 +154,15 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"top {top} must lie in 1..{experts}")
         if expert_form not in ("glu", "plain"):
             raise ValueError(f"expert_form is 'glu' or 'plain', got '{expert_form}'")
+        if expert_unit not in ("swish_clamped", "silu"):
+            raise ValueError(f"expert_unit is 'swish_clamped' or 'silu', got '{expert_unit}'")
         self.plain = expert_form == "plain"
+        self.silu = expert_unit == "silu" and not self.plain
+        if self.silu and weight_on != "output":
+            raise ValueError("silu units are not linear in their input: the weight goes on the output")
+        if expert_unit == "swish_clamped" and not self.plain and not expert_limit > 0.0:
+            raise ValueError("the clamped gated unit wants a positive limit")
+        self.router_biased = bool(router_bias)
         if self.plain and (activation not in ops.ACTIVATIONS or ops.ACTIVATIONS[activation] == 0):
             raise ValueError(f"plain experts: no activation '{activation}'")
         if self.plain and weight_on != "output":
@@ -173,6 +184,8 @@ class RoutedExperts(FeedForward):
     def tensor_needs(self):
         H, F, p = self.hidden_size, self.expert_ff, self.prefix
         needs = {p + "router": TensorNeed((self.experts, H))}
+        if self.router_biased:
+            needs[p + "router.b"] = TensorNeed((self.experts,), "bias")
         for e in range(self.experts):
             if not self.plain:
                 needs[f"{p}e{e}.gate"] = TensorNeed((F, H))
@@ -191,6 +204,7 @@ class RoutedExperts(FeedForward):
         p = self.prefix
         w = lambda n: tensors[p + n].to(device=rt.device, dtype=rt.dtype)
         self.router = tensors[p + "router"].to(device=rt.device, dtype=torch.float32).contiguous()
+        self.router_b = tensors[p + "router.b"].to(device=rt.device, dtype=torch.float32).contiguous() if self.router_biased else None
         self.run_dtype = rt.dtype
         # [E, 2F, H]: an expert's gate and up rows; [E, H, F].  bfloat16 with rows of 16-byte alignment: (gate, up) row by
         # row, the layout that the tcgen05 product's epilogue wants (the other kernels read either); else all gate
@@ -223,7 +237,13 @@ class RoutedExperts(FeedForward):
         stacked = torch.cat(rows + [torch.zeros((-len(torch.cat(rows)) % 8, self.hidden_size), device=rt.device)])
         self.router_linear = None
         if rt.dtype == torch.float32 or bool((stacked.to(torch.bfloat16).float() == stacked).all()):
-            self.router_linear = Linear(stacked.to(rt.dtype))
+            bias = None
+            if self.router_b is not None:
+                bias = torch.zeros(len(stacked), device=rt.device, dtype=torch.float32)
+                bias[:self.experts] = self.router_b
+            self.router_linear = Linear(stacked.to(rt.dtype), bias)
+        # (limit, slope, shift) of the experts' gated unit
+        self.unit = ops.SWIGLU_UNIT if self.silu else (self.expert_limit, self.alpha, 1.0)
 
     # ---- cost of a step
     def weight_bytes(self) -> int:
@@ -271,7 +291,7 @@ class RoutedExperts(FeedForward):
                           experts=E, **route)
         else:
             ops.moe_route(h, self.router, self.shared_gate, top, self.scoring == "softmax", self.renormalize, ids, weights, gate,
-                          **route)
+                          router_bias=self.router_b, **route)
         place = torch.empty(rows, device=dev, dtype=torch.int32)
         w_in = weights if self.weight_on == "input" else None
         w_out = weights if self.weight_on == "output" else None
@@ -291,8 +311,9 @@ class RoutedExperts(FeedForward):
             ops.gemm_tc_grouped(hg, self.gate_up, act, tile_expert, used, unary=self.activation)
             parts = torch.empty((tiles * tile, H), device=dev, dtype=h.dtype)
             ops.gemm_tc_grouped(act, self.down, parts, tile_expert, used, row_scale=scale)
-        elif self.pairs and rows >= ops.MOE_TC_ROWS and rows >= ops.MOE_TC_ROWS_PER_EXPERT * E and w_out is None:
-            # many rows: tiles of 128 rows on the tcgen05 product, the tokens' rows copied into grouped order first
+        elif self.pairs and rows >= ops.MOE_TC_ROWS and rows >= ops.MOE_TC_ROWS_PER_EXPERT * E:
+            # many rows: tiles of 128 rows on the tcgen05 product, the tokens' rows copied into grouped order first; a row's
+            # weight joins where it belongs, on the first product's accumulators (input) or the second's (output)
             tile = ops.MOE_TC_TILE
             tiles = ops.moe_max_tiles(rows, E, tile)
             grouped = torch.empty(tiles * tile, device=dev, dtype=torch.int32)
@@ -301,19 +322,21 @@ class RoutedExperts(FeedForward):
             ops.moe_group(ids, E, grouped, place, tile_expert, tile, used)
             hg = torch.empty((tiles * tile, H), device=dev, dtype=h.dtype)
             scale = torch.empty(tiles * tile, device=dev, dtype=torch.float32)
-            ops.moe_gather(h, grouped, w_in, top, hg, scale, used, tile)
+            ops.moe_gather(h, grouped, weights, top, hg, scale, used, tile)
             act = torch.empty((tiles * tile, F), device=dev, dtype=h.dtype)
-            ops.gemm_tc_grouped(hg, self.gate_up, act, tile_expert, used, True, scale, self.expert_limit, self.alpha)
+            limit, alpha, shift = self.unit
+            ops.gemm_tc_grouped(hg, self.gate_up, act, tile_expert, used, True, scale if w_in is not None else None, limit, alpha, shift=shift)
             # the experts' outputs leave the product as bfloat16 (as every projection's do); their sum is 32-bit
             parts = torch.empty((tiles * tile, H), device=dev, dtype=h.dtype)
-            ops.gemm_tc_grouped(act, self.down, parts, tile_expert, used)
+            ops.gemm_tc_grouped(act, self.down, parts, tile_expert, used, row_scale=scale if w_out is not None else None)
         else:
             grouped = torch.empty(tiles * ops.MOE_TILE, device=dev, dtype=torch.int32)
             tile_expert = torch.empty(tiles, device=dev, dtype=torch.int32)
             ops.moe_group(ids, E, grouped, place, tile_expert)
             act = torch.empty((tiles * ops.MOE_TILE, F), device=dev, dtype=h.dtype)
-            ops.moe_experts_up(h, self.gate_up, act, grouped, tile_expert, w_in, top, self.expert_limit, self.alpha, self.pairs,
-                               plain_act=self.activation if self.plain else None)
+            limit, alpha, shift = self.unit
+            ops.moe_experts_up(h, self.gate_up, act, grouped, tile_expert, w_in, top, limit, alpha, self.pairs,
+                               plain_act=self.activation if self.plain else None, shift=shift)
             parts = torch.empty((tiles * ops.MOE_TILE, H), device=dev, dtype=torch.float32)
             ops.moe_experts_down(act, self.down, parts, grouped, tile_expert, w_out, top)
         shared = None
@@ -321,7 +344,9 @@ class RoutedExperts(FeedForward):
             shared = self.shared_down(self.shared_gate_up(h, unary=self.activation))
         elif self.shared_ff:
             sact = torch.empty((T, self.shared_ff), device=dev, dtype=h.dtype)
-            if self.shared_pairs and ops.linear_bf16_glu_takes(h, self.shared_gate_up.weight):
+            if self.silu:
+                ops.glu(self.shared_gate_up(h), sact, ops.ACTIVATIONS["silu"], 0.0, 0.0, self.shared_pairs)
+            elif self.shared_pairs and ops.linear_bf16_glu_takes(h, self.shared_gate_up.weight):
                 ops.linear_bf16_glu(h, self.shared_gate_up.weight, sact, self.shared_limit, self.alpha)
             else:
                 gu = self.shared_gate_up(h)
@@ -374,6 +399,8 @@ class DenseFF(FeedForward):
         return self.up.flops(num_tokens) + self.down.flops(num_tokens)
 
     def forward(self, h, ctx):
+        if self.activation != "xielu":      # in the product's epilogue where there is one
+            return self.down(self.up(h, unary=self.activation))
         z = self.up(h)
         ops.activation(z, z, self.activation, self.p0, self.p1)
         return self.down(z)

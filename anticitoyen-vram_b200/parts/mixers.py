@@ -49,7 +49,10 @@ class Attention(Mixer):
     (1 - lambda) v + lambda v_source, lambda its own number in ``tensor``.
     ``sink``: the softmax's denominator also holds exp(sink_h), a score with no key and no value: a tensor's name (one
     learned number per query head) or a constant for all heads.  ``slope_rate`` r: slope_h (i - j) is taken off the score
-    of query i and key j, slope_h = 2^(-r (h + 1) / heads)."""
+    of query i and key j, slope_h = 2^(-r (h + 1) / heads).
+    ``tied_values``: there is no value projection; a head's value is its key as projected, before norm and rotation (both are
+    kept, one beside the other).  ``gate``: the name of a matrix W_g over the heads' values: the heads side by side are
+    multiplied by sigmoid(W_g h) in front of W_o, in the attention kernels, in 32-bit, before they are rounded."""
 
     ROLES = ("q", "k", "v", "o")
 
@@ -59,7 +62,7 @@ class Attention(Mixer):
                  names: dict | None = None, out_scale: float = 1.0, qk_norm_weights: bool = True,
                  score: dict | None = None, qk_norm_scope: str = "head", value_norm_eps: float | None = None,
                  q_temp: tuple | None = None, value_share: dict | None = None, sink: str | float | None = None,
-                 slope_rate: float | None = None) -> None:
+                 slope_rate: float | None = None, tied_values: bool = False, gate: str | None = None) -> None:
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads are not a multiple of {num_kv_heads} kv heads")
         if qk_norm_scope not in ("head", "all"):
@@ -81,6 +84,11 @@ class Attention(Mixer):
         if (self.wide or sink is not None or slope_rate is not None) and (score or keep_first or out_scale != 1.0):
             raise ValueError("attention: sinks, slopes and the steps over whole projections are not built beside score steps, "
                              "kept first tokens or an output factor")
+        self.tied_values, self.gate = bool(tied_values), gate
+        if (self.tied_values or gate is not None) and (self.wide or score):
+            raise ValueError("attention: tied values and an output gate are not built beside score steps or steps over whole projections")
+        if self.tied_values and value_dim not in (None, 0, head_dim):
+            raise ValueError(f"attention: values that are the keys have the keys' size {head_dim}, not {value_dim}")
         self.hidden_size = hidden_size
         self.num_heads, self.num_kv_heads, self.head_dim = num_heads, num_kv_heads, head_dim
         self.qk_norm_weights = bool(qk_norm_weights)
@@ -110,8 +118,10 @@ class Attention(Mixer):
         self.q_size = num_heads * head_dim
         self.kv_size = num_kv_heads * head_dim
         self.v_size = num_kv_heads * self.value_dim
-        self.in_size = self.q_size + self.kv_size + self.v_size      # columns of the stacked input projection
         self.inner_size = num_heads * self.value_dim                 # columns in front of the output projection
+        # columns of the stacked input projection: [q | k | v | gate], the last two where the layer has them
+        self.gate_at = self.q_size + self.kv_size + (0 if self.tied_values else self.v_size)
+        self.in_size = self.gate_at + (self.inner_size if gate is not None else 0)
 
     def cache_need(self):
         return PagedNeed(self.num_kv_heads, self.head_dim, self.window,
@@ -132,6 +142,8 @@ class Attention(Mixer):
         needs = {}
         for role, n_out, n_in in (("q", self.q_size, H), ("k", self.kv_size, H), ("v", self.v_size, H),
                                   ("o", H, self.inner_size)):
+            if role == "v" and self.tied_values:
+                continue
             needs[self.prefix + self.names[role]] = TensorNeed((n_out, n_in))
             if self.bias is not False and role + ".bias" in self.names:
                 needs[self.prefix + self.names[role + ".bias"]] = TensorNeed((n_out,), "bias", optional=self.bias is None)
@@ -139,6 +151,8 @@ class Attention(Mixer):
             whole = self.qk_norm_scope == "all"
             needs[self.prefix + self.names.get("q_norm", "q_norm.weight")] = TensorNeed((self.q_size if whole else self.head_dim,), "norm")
             needs[self.prefix + self.names.get("k_norm", "k_norm.weight")] = TensorNeed((self.kv_size if whole else self.head_dim,), "norm")
+        if self.gate is not None:
+            needs[self.prefix + self.gate] = TensorNeed((self.inner_size, H))
         if isinstance(self.sink, str):
             needs[self.prefix + self.sink] = TensorNeed((self.num_heads,), "norm")
         if self.value_share is not None and "tensor" in self.value_share:
@@ -160,7 +174,12 @@ class Attention(Mixer):
             name = self.prefix + self.names.get(role + ".bias", "\0")
             return tensors[name].to(device=rt.device, dtype=torch.float32) if name in tensors else None
 
-        self.qkv = Linear.stacked([w("q"), w("k"), w("v")], [b("q"), b("k"), b("v")])
+        roles = ("q", "k") if self.tied_values else ("q", "k", "v")
+        rows, biases = [w(r) for r in roles], [b(r) for r in roles]
+        if self.gate is not None:
+            rows.append(tensors[self.prefix + self.gate].to(device=rt.device, dtype=rt.dtype))
+            biases.append(None)
+        self.qkv = Linear.stacked(rows, biases)
         self.o = Linear(w("o"), b("o"))
         self.q_norm = self.k_norm = None
         f = lambda n: tensors[n].to(device=rt.device, dtype=torch.float32).contiguous()
@@ -197,7 +216,8 @@ class Attention(Mixer):
         rotary = self.position.rotary_table()
         if self.qkv.bias is not None or self.o.bias is not None or rotary is None or rotary.shape[1] != self.head_dim \
                 or self.value_dim != self.head_dim or self.keep_first or self.out_scale != 1.0 or self.wide \
-                or self.sinks is not None or self.slopes is not None or self.score is not None:
+                or self.sinks is not None or self.slopes is not None or self.score is not None or self.tied_values \
+                or self.gate is not None:
             return None
         return {"num_heads": self.num_heads, "num_kv_heads": self.num_kv_heads, "head_dim": self.head_dim,
                 "window": self.window, "scale": self.scale, "w_qkv": self.qkv.weight, "w_o": self.o.weight,
@@ -219,7 +239,7 @@ class Attention(Mixer):
             return
         ops.attention(qkv, out, cache.k_pages, cache.v_pages, ctx, table, NH, NKV, D, self.scale, self.window,
                       work=ctx.work[self.metadata_key], value_dim=DV, keep_first=self.keep_first, sinks=self.sinks,
-                      slopes=self.slopes)
+                      slopes=self.slopes, gate=qkv[:, self.gate_at:self.in_size] if self.gate is not None else None)
 
     def _prepare(self, qkv, ctx, table, rows, kp, vp) -> None:
         """The steps over a token's whole projection, rotation and append in one launch."""
@@ -279,6 +299,8 @@ class Attention(Mixer):
         eps = self.qk_norm_eps if self.qk_norm_eps is not None else 0.0
         rotary = self.position.rotary_table()
         extra = {"value_dim": DV, "v_scale": self.out_scale} if (DV != D or self.out_scale != 1.0) else {}
+        if self.tied_values:
+            extra["tied"] = True
         if self.wide:
             self._prepare(qkv, ctx, table, rows, kp, vp)
         elif rotary is not None:
@@ -289,6 +311,8 @@ class Attention(Mixer):
             ops.qk_norm_rope_append(qkv, NH, NKV, D, self.q_norm, self.k_norm, eps, None, ctx.positions,
                                     ctx.seq_of_token, table if kp is not None else None, kp, vp, table_rows=rows, **extra)
         else:
+            if self.tied_values:
+                raise ValueError("attention: values that are the keys want rotary positions by table, or none")
             if self.q_norm is not None:
                 ops.qk_norm_rope_append(qkv, NH, NKV, D, self.q_norm, self.k_norm, eps, None, ctx.positions,
                                         ctx.seq_of_token, None, None, None, **extra)
@@ -303,7 +327,7 @@ class Attention(Mixer):
     def forward(self, h, ctx, cache: CacheView):
         NH, NKV, D = self.num_heads, self.num_kv_heads, self.head_dim
         if self.value_dim != D or self.out_scale != 1.0 or self.score is not None or isinstance(self.position, NoPosition) \
-                or self.wide or self.sinks is not None or self.slopes is not None:
+                or self.wide or self.sinks is not None or self.slopes is not None or self.tied_values or self.gate is not None:
             qkv = self.qkv(h)
             out = torch.empty((qkv.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
             self.mix(qkv, ctx, cache, out)

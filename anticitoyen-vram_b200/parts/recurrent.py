@@ -424,3 +424,111 @@ class GeneralDelta(Mixer):
         out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
         self.inner(h, ctx, cache, out)
         return self.o(out)
+
+
+@register("mixer", "gated_delta")
+class GatedDelta(Mixer):
+    """A gated delta rule (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule") behind a short
+    convolution; q and k of ``num_kv_heads`` heads of ``dim``, values, gates and states of ``num_heads`` heads of ``value_dim``,
+    head h reading the q and k of head h / (num_heads / num_kv_heads):
+
+        q, k, v = silu(conv(W h))          a causal convolution of ``conv`` taps per channel, the last tap the current token's
+        q <- q / sqrt(sum(q^2) + 1e-6) dim^(-1/2),    k <- k / sqrt(sum(k^2) + 1e-6)                                  per head
+        beta = sigmoid(W_b h),    g = exp(-exp(A_log) softplus(W_a h + dt_bias))                              one per head
+        S <- g S;    u = beta (v - S^T k);    S <- S + k u^T;    o = S^T q                              S: [dim, value_dim]
+
+    Each head's o is brought to unit RMS (``norm_eps``) and multiplied by one weight that all heads share, then by
+    silu(W_g h); W_o.  A request keeps S and the convolution's last inputs (in a ring of ``conv`` rows), float32.  32-bit in
+    every run precision: all of the above behind the projections, which leave their product as float.
+    Tensors behind ``prefix`` (``names`` renames them): q, k, v, q.conv, k.conv, v.conv, g, b, a, A_log, dt_bias, norm, o."""
+
+    NAMES = {n: n for n in ("q", "k", "v", "q.conv", "k.conv", "v.conv", "g", "b", "a", "A_log", "dt_bias", "norm", "o")}
+    metadata_key = "delta_blocks"       # the recurrence takes a request's tokens in blocks (``ops.delta_work``)
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, value_dim: int, conv: int, norm_eps: float,
+                 prefix: str = "mix.", names: dict | None = None) -> None:
+        if num_heads % num_kv_heads:
+            raise ValueError(f"{num_heads} heads are not a multiple of {num_kv_heads} kv heads")
+        if conv < 1:
+            raise ValueError("the convolution has at least one tap")
+        self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, int(num_heads), int(num_kv_heads)
+        self.dim, self.value_dim, self.taps = int(dim), int(value_dim), int(conv)
+        self.norm_eps = float(norm_eps)
+        self.prefix = prefix
+        self.names = {**self.NAMES, **(names or {})}
+        self.qk_size = self.num_kv_heads * self.dim
+        self.inner_size = self.num_heads * self.value_dim
+        self.channels = 2 * self.qk_size + self.inner_size      # what the convolution spans
+
+    def _n(self, role: str) -> str:
+        return self.prefix + self.names[role]
+
+    def step_metadata(self, q_lens, kv_lens, cu_q) -> StepMetadata:
+        return StepMetadata(*ops.delta_work(q_lens))
+
+    def decode_metadata(self, padded: int, max_kv: int) -> StepMetadata:
+        return StepMetadata(*ops.delta_work_decode(padded))
+
+    def cache_need(self):
+        return {"state": StateNeed((self.num_heads, self.dim, self.value_dim), "float32"),
+                "inputs": StateNeed((self.taps, self.channels), "float32")}
+
+    def tensor_needs(self):
+        W, H, I, K = self.hidden_size, self.num_heads, self.inner_size, self.taps
+        needs = {}
+        for role, n in (("q", self.qk_size), ("k", self.qk_size), ("v", I)):
+            needs[self._n(role)] = TensorNeed((n, W))
+            needs[self._n(role + ".conv")] = TensorNeed((n, K))
+        needs[self._n("g")] = TensorNeed((I, W))
+        for role in ("b", "a"):
+            needs[self._n(role)] = TensorNeed((H, W))
+        for role in ("A_log", "dt_bias"):
+            needs[self._n(role)] = TensorNeed((H,), "bias")
+        needs[self._n("norm")] = TensorNeed((self.value_dim,), "norm")
+        needs[self._n("o")] = TensorNeed((W, I))
+        return needs
+
+    def load(self, tensors, rt: Runtime) -> None:
+        w = lambda role: tensors[self._n(role)].to(device=rt.device, dtype=rt.dtype)
+        f = lambda role: tensors[self._n(role)].to(device=rt.device, dtype=torch.float32).contiguous()
+        # everything that reads the mixer's input is one product, [q | k | v | g | b | a] (and zero rows that make its output's
+        # rows 16-byte pieces); it leaves as float
+        rows = [w(role) for role in ("q", "k", "v", "g", "b", "a")]
+        pad = -sum(t.shape[0] for t in rows) % 8
+        if pad:
+            rows.append(torch.zeros((pad, self.hidden_size), device=rt.device, dtype=rt.dtype))
+        self.qkv = Linear.stacked(rows)
+        self.taps_t = torch.cat([f("q.conv"), f("k.conv"), f("v.conv")]).t().contiguous()
+        # the decay's rate is a constant of the weights: folded once, in float64
+        self.rate = tensors[self._n("A_log")].to(torch.float64).exp().to(device=rt.device, dtype=torch.float32).contiguous()
+        self.shift = f("dt_bias")
+        self.norm_weight = f("norm").repeat(self.num_heads).contiguous()
+        self.o = Linear(w("o"))
+
+    def weight_bytes(self) -> int:
+        return self.qkv.weight_bytes() + self.o.weight_bytes() + \
+            (self.taps_t.numel() + self.rate.numel() + self.shift.numel() + self.value_dim) * 4
+
+    def flops(self, num_tokens: int) -> float:
+        return self.qkv.flops(num_tokens) + self.o.flops(num_tokens)
+
+    def mixing_flops(self, q_lens, kv_lens) -> float:
+        # per token, head and state element: the decay, the products with k and q and the update; per channel the taps
+        per = 7.0 * self.num_heads * self.dim * self.value_dim + 2.0 * self.channels * self.taps
+        return per * sum(q_lens)
+
+    def cache_bytes_read(self, q_lens, kv_lens, itemsize: int) -> int:
+        return len(q_lens) * (self.num_heads * self.dim * self.value_dim + (self.taps - 1) * self.channels) * 4
+
+    def inner(self, h, ctx, cache: CacheView, out) -> None:
+        state, inputs = cache.parts["state"], cache.parts["inputs"]
+        proj = self.qkv(h, out_dtype=torch.float32)
+        ops.gated_delta(proj, self.taps_t, self.rate, self.shift, self.norm_weight, self.norm_eps, inputs.state,
+                        ctx.state_slots[inputs.group], state.state, ctx.state_slots[state.group], ctx.positions, ctx.cu_q,
+                        ctx.num_seqs, ctx.max_q_len, out, self.num_heads, self.num_kv_heads, self.dim, self.value_dim,
+                        ctx.work.get(self.metadata_key))
+
+    def forward(self, h, ctx, cache: CacheView):
+        out = torch.empty((h.shape[0], self.inner_size), device=h.device, dtype=h.dtype)
+        self.inner(h, ctx, cache, out)
+        return self.o(out)

@@ -312,7 +312,7 @@ def delta_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, rank
     us_all = _time(lambda i: ops.general_delta(proj, w2_t, w0, weight, 1e-6, state, slots, cu, batch, q_len, out, H, D, rank, work), reps)
     rec = ops.delta_blocks(proj, w2_t, w0, cu, H, D, work)
     us_prep = _time(lambda i: ops.delta_blocks(proj, w2_t, w0, cu, H, D, work), reps)
-    us = _time(lambda i: ops.delta(rec, proj, state, slots, cu, batch, o, H, D, work), reps)
+    us = _time(lambda i: ops.delta(rec, proj[:, 2 * H * D:3 * H * D], state, slots, cu, batch, o, H, D, work), reps)
     us_gate = _time(lambda i: ops.retention_gate(o, proj[:, 4 * I:5 * I], out, H, D, 1e-6, weight=weight, gate_fn="sigmoid"), reps)
     flops = 10.0 * H * D * D * T        # five multiply-adds a state element and token
     print(f"delta q_len={q_len} batch={batch} heads={H} of {D}x{D}: all {us_all:.1f} us, recurrence {us:.1f} us ({flops / us / 1e6:.2f} "
