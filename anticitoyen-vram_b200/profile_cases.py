@@ -322,6 +322,40 @@ def delta_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, rank
             "tflops_f32": flops / us / 1e6}
 
 
+def gated_delta_case(q_len: int, batch: int, reps: int, H: int = 16, G: int = 8, D: int = 128, DV: int = 128, taps: int = 4,
+                     form: int = 0) -> dict:
+    """The gated delta rule behind its input product: convolution and blocks, recurrence and gate of ``batch`` portions of
+    ``q_len`` tokens, or the one launch of steps of single tokens."""
+    T, I = q_len * batch, H * DV
+    C = 2 * G * D + I
+    dev = "cuda:0"
+    proj = torch.randn(T, C + I + 2 * H, device=dev)
+    taps_t = torch.randn(taps, C, device=dev) * 0.5
+    rate, shift = torch.full((H,), 0.1, device=dev), torch.zeros(H, device=dev)
+    weight = torch.ones(I, device=dev)
+    state, ring = torch.zeros(batch, H, D, DV, device=dev), torch.zeros(batch, taps, C, device=dev)
+    slots = torch.arange(batch, dtype=torch.int32, device=dev)
+    cu = torch.arange(0, T + 1, q_len, dtype=torch.int32, device=dev)
+    positions = torch.arange(T, dtype=torch.int32, device=dev) % q_len
+    out = torch.empty(T, I, device=dev, dtype=torch.bfloat16)
+    o = torch.empty(T, I, device=dev)
+    arrays, values = ops.delta_work([q_len] * batch)
+    work = {**{k: torch.as_tensor(v).to(dev) for k, v in arrays.items()}, **values}
+    us_all = _time(lambda i: ops.gated_delta(proj, taps_t, rate, shift, weight, 1e-6, ring, slots, state, slots, positions, cu, batch,
+                                             q_len, out, H, G, D, DV, work), reps)
+    blocks = lambda i: ops.gated_delta_blocks(proj, taps_t, rate, shift, ring, slots, positions, cu, batch, H, G, D, DV, work)
+    rec, vals = blocks(0)
+    us_prep = _time(blocks, reps)
+    us = _time(lambda i: ops.delta(rec, vals, state, slots, cu, batch, o, H, D, work, value_dim=DV, gated=True, form=form), reps)
+    us_gate = _time(lambda i: ops.retention_gate(o, proj[:, C:C + I], out, H, DV, 1e-6, weight=weight, gate_fn="silu"), reps)
+    flops = 7.0 * H * D * DV * T
+    print(f"gated delta q_len={q_len} batch={batch} heads={H}/{G} of {D}x{DV} form {form}: all {us_all:.1f} us, recurrence {us:.1f} us "
+          f"({flops / us / 1e6:.2f} TFLOP/s float), blocks {us_prep:.1f} us, gate {us_gate:.1f} us; "
+          f"all: state {2 * batch * H * D * DV * 4 / us_all / 1e3:.0f} GB/s")
+    return {"kernel": "gated_delta", "q_len": q_len, "batch": batch, "us": us, "us_all": us_all, "us_blocks": us_prep, "us_gate": us_gate,
+            "tflops_f32": flops / us / 1e6}
+
+
 def wkv_case(q_len: int, batch: int, reps: int, H: int = 32, D: int = 64, C: int = 2048, rank: int = 32) -> dict:
     """Time mixing's own kernels for ``batch`` requests that bring ``q_len`` tokens each: the five mixes of the token
     shift, the decays, and the recurrence of 32 heads of 64 x 64 with decays of the token's own."""
@@ -495,6 +529,12 @@ CASES = {
     "delta_prefill_b8": lambda r: delta_case(512, 8, r),
     "delta_prefill_128": lambda r: delta_case(2048, 1, r, H=16, D=128),
     "delta_decode_b64": lambda r: delta_case(1, 64, r),
+    "delta_decode_b64_128": lambda r: delta_case(1, 64, r, H=16, D=128),
+    "gated_delta_prefill": lambda r: gated_delta_case(2048, 1, r),
+    "gated_delta_prefill_64": lambda r: gated_delta_case(2048, 1, r, H=32, G=16, D=64, DV=64),
+    "gated_delta_prefill_b8": lambda r: gated_delta_case(512, 8, r),
+    "gated_delta_decode_b64": lambda r: gated_delta_case(1, 64, r),
+    "gated_delta_decode_b8": lambda r: gated_delta_case(1, 8, r),
     "wkv_prefill": lambda r: wkv_case(2048, 1, r),
     "wkv_prefill_small": lambda r: wkv_case(512, 1, r),
     "wkv_decode_b64": lambda r: wkv_case(1, 64, r),

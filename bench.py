@@ -431,6 +431,117 @@ def run_lodalix(args) -> int:
     return 0
 
 
+ZOGAPEL_SIZES = {
+    # width; attention: heads, kv heads, head size, rotated part, window; recurrence: value heads, query/key heads, key size,
+    # value size, taps; dense feed-forward size (two matrices); mixture: experts, choices, an expert's size
+    "s": dict(width=2048, heads=16, kv_heads=4, dim=128, rot=64, window=1024, d_heads=16, d_kv=8, d_dim=128, d_vdim=128, taps=4,
+              ff=9216, experts=32, top=4, e_ff=768),
+    "m": dict(width=4096, heads=32, kv_heads=8, dim=128, rot=64, window=2048, d_heads=32, d_kv=16, d_dim=128, d_vdim=128, taps=4,
+              ff=18432, experts=64, top=6, e_ff=1024),
+}
+
+
+def run_zogapel(args) -> int:
+    """``--design zogapel``: prefill and decode throughput of the Zogapel design at layer sizes of real models (random
+    weights; six layers: windowed attention whose values are its keys and the gated delta rule in turn, a dense feed-forward
+    in every third layer and a mixture in the others), beside the closest models of the framework at equal size: a Vadelix
+    model with windowed attention of the same heads, its own recurrence with as much state, and feed-forwards of equal weight
+    count; one layer of Lodalix for the delta rule (as many heads of the same size); one of Nizedra for the dense unit.
+    Whole steps through the step function, and the mixer and feed-forward of each kind of layer alone with their
+    rooflines (L2 flushed before each timed run).  One JSON line."""
+    import torch
+
+    from acvram_b200 import bench as B
+    from acvram_b200.config import LodalixConfig, NizedraConfig, VadelixConfig, ZogapelConfig
+    from acvram_b200.engine.runner import ModelRunner
+    from acvram_b200.models import build_random
+
+    pk, pk_src = peaks()
+    K, W = args.steps, args.warmup
+    page = 64
+    layers, vocab = args.layers or 6, 32768
+    out = {"design": "zogapel", "beside": ["vadelix", "lodalix", "nizedra"], "layers": layers, "vocab": vocab, "dtype": "bf16",
+           "page_size": page, "data": "synthetic token ids, random weights", "peaks": {**pk, "source": pk_src}, "sizes": {}}
+    for name in args.sizes.split(","):
+        z = ZOGAPEL_SIZES[name]
+        heads = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                 "mask": {"size": z["window"]}}
+        rot = {"base": 1e6, "dims": z["rot"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+        gated = {"heads": z["d_heads"], "kv_heads": z["d_kv"], "dim": z["d_dim"], "vdim": z["d_vdim"], "conv": z["taps"]}
+        dense, moe = {"kind": "dense", "ff": z["ff"]}, {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["e_ff"]}}
+        zcfg = ZogapelConfig.from_dict({
+            "architecture": "Zogapel", "vocab": vocab, "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [{"type": "delta", "mixer": gated, "mlp": moe if i % 3 else dense} if i % 2 else
+                       {"type": "attention", "mixer": {**heads, "rot": rot}, "mlp": moe if i % 3 else dense} for i in range(layers)]})
+        # (a gated unit has three matrices, a plain expert two; the relative's mixture always has a shared expert: a small one)
+        v_dense = {"kind": "dense", "ff": z["ff"] * 2 // 3}
+        v_moe = {"kind": "moe", "expert": {"ff": z["e_ff"] * 3 // 2}, "shared": {"ff": 64},
+                 "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 1, "keep": 1}}}
+        v_mixer = {**heads, "v_mix": False, "q_temp": {"coef": 0.1, "every": 512}}
+        state = z["d_heads"] * z["d_dim"] * z["d_vdim"]
+        wkv = {"heads": state // (64 * 64), "dim": 64}
+        vcfg = VadelixConfig.from_dict({
+            "architecture": "Vadelix", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6, "groups": 1}, "residual_mult": 1.0,
+            "canon": {"taps": 1},
+            "layers": [{"type": "wkv", "mixer": wkv, "mlp": v_moe if i % 3 else v_dense} if i % 2 else
+                       {"type": "attention_2", "mixer": v_mixer, "mlp": v_moe if i % 3 else v_dense} for i in range(layers)]})
+        lcfg = LodalixConfig.from_dict({
+            "architecture": "Lodalix", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [{"type": "general_delta", "mixer": {"heads": z["d_heads"], "dim": z["d_dim"]}, "mlp": None}]})
+        light = {"heads": z["d_heads"], "dim": z["d_dim"], "vdim": z["d_vdim"], "decay": [1.0 - 2.0 ** (-4 - i % 8) for i in range(z["d_heads"])]}
+        ncfg = NizedraConfig.from_dict({"architecture": "Nizedra", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6},
+                                        "layers": [{"type": "lightning", "mixer": light, "mlp": dense}]})
+        kinds_of = {"zogapel": (("attention", 0, "dense"), ("gated_delta", 1, "moe")),
+                    "vadelix": (("attention", 0, "gated_unit"), ("wkv", 1, "moe")),
+                    "lodalix": (("general_delta", 0, None),), "nizedra": (("lightning", 0, "dense"),)}
+        res = {"sizes": dict(z)}
+        for arm, cfg in (("zogapel", zcfg), ("vadelix", vcfg), ("lodalix", lcfg), ("nizedra", ncfg)):
+            model = build_random(cfg, seed=0, dtype=torch.bfloat16, device="cuda:0")
+            batch_max = 64
+            tokens = batch_max * (args.context + 2 * (K + W) + 2 * page) + 4096
+            runner = ModelRunner(model, page, tokens // page + 8, batch_max + 2, max_len=8192)
+            if not args.no_cuda_graphs:
+                runner.enable_graphs()
+            r = {"weights_gb": round(model.weight_bytes() / 1e9, 3)}
+            try:
+                if arm in ("zogapel", "vadelix"):
+                    pre = B.time_prefill(runner, 2048, reps=5, warmup=3)
+                    flops = B.prefill_flops(model, 2048)
+                    r["prefill_2048"] = {"tokens_per_s": round(pre["tokens_per_s"], 1), "ms": round(pre["ms"], 3),
+                                         "tflops_frac": round(flops / (pre["ms"] * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)}
+                    for b in (8, 64):
+                        names = [f"d{b}-{i}" for i in range(b)]
+                        B.fill_contexts(runner, names, args.context)
+                        try:
+                            d = B.time_decode(runner, names, K, W)
+                        finally:
+                            for n in names:
+                                runner.release(n)
+                        nbytes = B.decode_step_bytes(model, b, args.context + W + K // 2)
+                        r[f"decode_b{b}"] = {"tokens_per_s": round(d["tokens_per_s"], 1), "ms_per_step": round(d["ms_per_step"], 4),
+                                             "hbm_frac": round(nbytes / (d["ms_per_step"] * 1e-3) / 1e9 / pk["hbm_gbs"], 4)}
+                for kind, layer, unit in kinds_of[arm]:
+                    if layer >= layers:
+                        continue
+                    for label, ql, kl in (("prefill_2048", [2048], [2048]), ("decode_b64", [1] * 64, [args.context] * 64)):
+                        for part, v in B.time_parts(runner, ql, kl, layer=layer).items():
+                            what = kind if part == "mixer" else unit
+                            if what is None:
+                                continue
+                            sec = v["ms"] * 1e-3
+                            r[f"{what}_{label}"] = {"us": round(v["ms"] * 1e3, 1),
+                                                    "tflops_frac": round(v["flops"] / sec / (pk["bf16_tflops"] * 1e12), 4),
+                                                    "hbm_frac": round(v["bytes"] / sec / 1e9 / pk["hbm_gbs"], 4)}
+            except B.Refused as exc:
+                r["refused"] = str(exc)
+            res[arm + "_result"] = r
+            del runner, model
+            _free_device_memory()
+        out["sizes"][name] = res
+    print(json.dumps(out))
+    return 0
+
+
 def run_vadelix(args) -> int:
     """``--design vadelix``: prefill and decode throughput of the Vadelix design at layer sizes of real models (random
     weights; six layers: time mixing, rotated attention with sinks, windowed attention with slopes, twice, gated
@@ -791,7 +902,7 @@ def main() -> int:
     ap.add_argument("--page-size", type=int, default=16, help="tokens in a page of the cache (the engine's own default is 64)")
     ap.add_argument("--skip-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--no-cuda-graphs", action="store_true")
-    ap.add_argument("--design", default="", choices=["", "zotonex", "redudra", "nizedra", "vadelix", "lodalix"],
+    ap.add_argument("--design", default="", choices=["", "zotonex", "redudra", "nizedra", "vadelix", "lodalix", "zogapel"],
                     help="measure another design beside its closest relative instead of the headline (see run_design)")
     ap.add_argument("--sizes", default="s,m", help="with --design: which of its sizes (s: width 2048, m: width 4096)")
     ap.add_argument("--time-limit", type=float, default=240.0,
@@ -812,6 +923,8 @@ def main() -> int:
         return run_vadelix(args)
     if args.design == "lodalix":
         return run_lodalix(args)
+    if args.design == "zogapel":
+        return run_zogapel(args)
     if args.design:
         return run_design(args)
     return run_ours(args)
