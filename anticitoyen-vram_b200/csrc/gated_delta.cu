@@ -29,6 +29,7 @@
 
 #define GD_TOK 8
 #define GD_UNIT_EPS 1e-6f
+#define GD_CHANNELS 256         // query channels of a thread block of the blocks' kernel, where heads are small enough
 
 static int gated_delta_pad(int D) {
     int p = 8;
@@ -82,40 +83,39 @@ __device__ __forceinline__ void keep_inputs(const float* __restrict__ x, int ld,
 }
 
 // ----------------------------------------------------------------------------- the blocks' records
-// grid (blocks of tokens, G); H / G heads belong to a thread block, and so do their channels of the convolution.
+// grid (blocks of tokens, tiles of `ng` q/k heads); the heads that read them belong to a thread block, and so do their channels
+// of the convolution.
 template <int KT>
 __global__ void __launch_bounds__(256)
 gated_delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ wt, const float* __restrict__ rate,
                           const float* __restrict__ shift, float* ring, const int* __restrict__ slots,
                           const int* __restrict__ positions, const int* __restrict__ item_seq, const int* __restrict__ item_idx,
                           const int* __restrict__ cu_q, float* __restrict__ values, float* __restrict__ rec, int G, int H,
-                          int D, int DV, int DP, int K) {
+                          int D, int DV, int DP, int K, int ng) {
     extern __shared__ __align__(16) float sm[];
     const int PD = (D + 3) & ~3, r = H / G;
-    float* rows = sm;                       // [16][PD]: y_q of the eight tokens, y_k
-    float* qk = rows + 16 * PD;             // [8][8]
-    float* kk = qk + 64;                    // [8][8]
-    float* inv = kk + 64;                   // [16]: what brings y_q, y_k to their length
-    float* wa = inv + 16;                   // [8 warps][128]: A, Q of the head that a warp is at
-    float* coef = wa + 8 * 128;             // [r][144]
+    float* rows = sm;                       // [ng][16][PD]: y_q of the eight tokens, y_k
+    float* gram = rows + (size_t)ng * 16 * PD;      // [ng][144]: <q, k> [8][8], <k, k> [8][8], what brings y_q, y_k to their length [16]
+    float* wa = gram + ng * 144;            // [8 warps][128]: A, Q of the head that a warp is at
+    float* coef = wa + 8 * 128;             // [ng r][144]
     pdl_wait();
-    const int item = blockIdx.x, grp = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int item = blockIdx.x, g0 = blockIdx.y * ng, gn = min(ng, G - g0), hn = gn * r, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int seq = item_seq[item], idx = item_idx[item];
     const int first = cu_q[seq], off = idx * GD_TOK, t0 = first + off, len = cu_q[seq + 1] - first;
     const int n = min(GD_TOK, len - off), pos = positions[t0];
     const int C = 2 * G * D + H * DV, I = H * DV;
     float* slot = ring + (size_t)slots[seq] * K * C;
     const float* base = proj + (size_t)t0 * ld;
-    for (int ch = tid; ch < 2 * D; ch += 256) {
-        const bool is_k = ch >= D;
-        const int e = is_k ? ch - D : ch, c = (is_k ? G * D : 0) + grp * D + e;
+    for (int ch = tid; ch < 2 * gn * D; ch += 256) {
+        const bool is_k = ch >= gn * D;
+        const int at = is_k ? ch - gn * D : ch, gl = at / D, e = at - gl * D, c = (is_k ? G * D : 0) + g0 * D + at;
         float y[GD_TOK];
         conv8<KT>(base + c, ld, wt + c, C, K, slot + c, off, pos, n, y);
 #pragma unroll
-        for (int t = 0; t < GD_TOK; ++t) rows[(size_t)((is_k ? 8 : 0) + t) * PD + e] = t < n ? gd_silu(y[t]) : 0.f;
+        for (int t = 0; t < GD_TOK; ++t) rows[(size_t)(gl * 16 + (is_k ? 8 : 0) + t) * PD + e] = t < n ? gd_silu(y[t]) : 0.f;
     }
-    for (int ch = tid; ch < r * DV; ch += 256) {
-        const int at = grp * r * DV + ch, c = 2 * G * D + at;
+    for (int ch = tid; ch < hn * DV; ch += 256) {
+        const int at = g0 * r * DV + ch, c = 2 * G * D + at;
         float y[GD_TOK];
         conv8<KT>(base + c, ld, wt + c, C, K, slot + c, off, pos, n, y);
 #pragma unroll
@@ -125,50 +125,57 @@ gated_delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* _
     __syncthreads();
     if (idx == 0 && K > 1 && K <= GD_TOK + 1) {     // no other block reads these channels' kept inputs (off >= K - 1 there)
         const float* p = proj + (size_t)first * ld;
-        for (int ch = tid; ch < 2 * D + r * DV; ch += 256) {
-            const int c = ch < D ? grp * D + ch : ch < 2 * D ? G * D + grp * D + ch - D : 2 * G * D + grp * r * DV + ch - 2 * D;
+        const int w = gn * D;
+        for (int ch = tid; ch < 2 * w + hn * DV; ch += 256) {
+            const int c = ch < w ? g0 * D + ch : ch < 2 * w ? G * D + g0 * D + ch - w : 2 * G * D + g0 * r * DV + ch - 2 * w;
             keep_inputs(p + c, ld, slot + c, C, K, len, pos);
         }
     }
     // a warp one token's row of both matrices
-    {
-        const float* q = rows + (size_t)warp * PD;
-        const float* k = rows + (size_t)(8 + warp) * PD;
+    for (int u = warp; u < gn * 8; u += 8) {
+        const int gl = u >> 3, i = u & 7;
+        const float* base_q = rows + (size_t)gl * 16 * PD;
+        const float* base_k = base_q + (size_t)8 * PD;
         float a[8], b[8], qq = 0.f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) a[j] = b[j] = 0.f;
         for (int e = lane; e < D; e += 32) {
-            const float qe = q[e], ke = k[e];
+            const float qe = base_q[(size_t)i * PD + e], ke = base_k[(size_t)i * PD + e];
             qq = fmaf(qe, qe, qq);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                const float kj = rows[(size_t)(8 + j) * PD + e];
+                const float kj = base_k[(size_t)j * PD + e];
                 a[j] = fmaf(qe, kj, a[j]);
                 b[j] = fmaf(ke, kj, b[j]);
             }
         }
+        // both rows' sixteen sums over the lanes: every exchange halves the values that a lane still carries
+        const bool up4 = lane & 16, up3 = lane & 8, up2 = lane & 4, up1 = lane & 2;
+        float x[8], y[4], z[2];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = (up4 ? b[j] : a[j]) + __shfl_xor_sync(0xffffffffu, up4 ? a[j] : b[j], 16);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = (up3 ? x[j + 4] : x[j]) + __shfl_xor_sync(0xffffffffu, up3 ? x[j] : x[j + 4], 8);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) z[j] = (up2 ? y[j + 2] : y[j]) + __shfl_xor_sync(0xffffffffu, up2 ? y[j] : y[j + 2], 4);
+        float sum = (up1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, up1 ? z[0] : z[1], 2);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
         qq = warp_sum(qq);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            a[j] = warp_sum(a[j]);
-            b[j] = warp_sum(b[j]);
-        }
-        if (lane == 0) {
-            inv[warp] = 1.f / (sqrtf(qq + GD_UNIT_EPS) * sqrtf((float)D));
-#pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                qk[warp * 8 + j] = a[j];
-                kk[warp * 8 + j] = b[j];
-                if (j == warp) inv[8 + warp] = 1.f / sqrtf(b[j] + GD_UNIT_EPS);
-            }
-        }
+        float* gm = gram + gl * 144;
+        const int j = (up3 ? 4 : 0) + (up2 ? 2 : 0) + (up1 ? 1 : 0);
+        if (!(lane & 1)) gm[(up4 ? 64 : 0) + i * 8 + j] = sum;
+        if (lane == 0) gm[128 + i] = 1.f / (sqrtf(qq + GD_UNIT_EPS) * sqrtf((float)D));
+        if (up4 && j == i && !(lane & 1)) gm[136 + i] = 1.f / sqrtf(sum + GD_UNIT_EPS);
     }
     __syncthreads();
     const size_t rs = 24 * (size_t)DP + 132;
-    float* out = rec + ((size_t)item * H + (size_t)grp * r) * rs;
+    float* out = rec + ((size_t)item * H + (size_t)g0 * r) * rs;
     // a warp a head; lane j (mod 8) owns column j
-    for (int hh = warp; hh < r; hh += 8) {
-        const int h = grp * r + hh, j = lane & 7;
+    for (int hh = warp; hh < hn; hh += 8) {
+        const int h = g0 * r + hh, j = lane & 7;
+        const float* qk = gram + hh / r * 144;
+        const float* kk = qk + 64;
+        const float* inv = qk + 128;
         float beta = 0.f, g = 1.f;
         if (j < n) {
             const float* row = base + (size_t)j * ld + C + I;
@@ -220,8 +227,9 @@ gated_delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* _
         const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
         x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
     };
-    for (int u = tid; u < r * DP; u += 256) {
+    for (int u = tid; u < hn * DP; u += 256) {
         const int hh = u / DP, e = u - hh * DP;
+        const float* mine = rows + (size_t)(hh / r) * 16 * PD + e;
         float* o = out + hh * rs + e;
         if (e >= D) {
 #pragma unroll
@@ -231,12 +239,12 @@ gated_delta_blocks_kernel(const float* __restrict__ proj, int ld, const float* _
         const float* cf = coef + hh * 144;
         float k[8], x[8], gam[8], dec[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) k[i] = rows[(size_t)(8 + i) * PD + e];
+        for (int i = 0; i < 8; ++i) k[i] = mine[(size_t)(8 + i) * PD];
         row8(cf + 128, gam);
         row8(cf + 136, dec);
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            float s = 0.f, t = gam[i] * rows[(size_t)i * PD + e];
+            float s = 0.f, t = gam[i] * mine[(size_t)i * PD];
             row8(cf + i * 8, x);
 #pragma unroll
             for (int l = 0; l <= i; ++l) s = fmaf(x[l], k[l], s);
@@ -275,16 +283,20 @@ ACV_API int acv_gated_delta_blocks(const float* proj, int ld, const float* wt, c
     if (G <= 0 || G > 65535 || H <= 0 || H % G || D <= 0 || D > 512 || DV <= 0 || K < 1 || ld < 2 * G * D + 2 * H * DV + 2 * H)
         return ACV_ERR_SIZE;
     const int PD = (D + 3) & ~3, C = 2 * G * D + H * DV;
-    const size_t smem = ((size_t)16 * PD + 144 + 8 * 128 + (size_t)(H / G) * 144) * sizeof(float);
+    // q/k heads of a thread block: enough for its threads, and for its warps where a warp makes a head's matrices
+    auto bytes = [&](int n) { return (8 * 128 + (size_t)n * (16 * PD + 144 + (size_t)(H / G) * 144)) * sizeof(float); };
+    int ng = 1;
+    while (ng * 2 <= G && ng * 2 * D <= GD_CHANNELS && bytes(ng * 2) <= 64 * 1024) ng *= 2;
+    const size_t smem = bytes(ng);
     if (smem > 200 * 1024) return ACV_ERR_SIZE;
-    const dim3 grid(n_items, G);
+    const dim3 grid(n_items, (G + ng - 1) / ng);
 #define GB_LAUNCH(N)                                                                                                          \
     do {                                                                                                                      \
         static AcvSmemConfig cfg;                                                                                             \
         if (smem > 48 * 1024)                                                                                                 \
             if (int e = acv_ensure_smem(cfg, gated_delta_blocks_kernel<N>, (int)smem)) return e;                              \
         acv_launch(PDL_MISC, gated_delta_blocks_kernel<N>, grid, 256, smem, stream, proj, ld, wt, rate, shift, ring, slots,   \
-                   positions, item_seq, item_idx, cu_q, values, rec, G, H, D, DV, gated_delta_pad(D), K);                     \
+                   positions, item_seq, item_idx, cu_q, values, rec, G, H, D, DV, gated_delta_pad(D), K, ng);                 \
     } while (0)
     if (K <= 4) GB_LAUNCH(4);
     else GB_LAUNCH(0);

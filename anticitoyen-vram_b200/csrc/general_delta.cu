@@ -544,6 +544,19 @@ static int delta_by_size(const float* rec, const float* values, int ld, float* s
     if (D <= 32) DL_CASE(8, 4, 1, 4, 3)
     // few columns for the device: four warps to sixteen columns; more: two warps, then one (fewer instructions a column)
     const long long tiles = (long long)n_seqs * H * ((DV + 15) / 16);
+    if constexpr (!KD) {        // (shorter records: measured to want their own shapes)
+        if (D > 32 && D <= 128 && !form) form = tiles <= 180 ? 1 : tiles <= 600 ? 2 : 3;
+        if (D > 32 && D <= 64) {
+            if (form == 1) DL_CASE(8, 8, 2, 2, 4)
+            if (form == 2) DL_CASE(4, 16, 4, 2, 4)
+            DL_CASE(8, 8, 4, 1, 3)
+        }
+        if (D > 64 && D <= 128) {
+            if (form == 1) DL_CASE(8, 16, 2, 4, 4)
+            if (form == 2) DL_CASE(8, 16, 4, 2, 3)
+            DL_CASE(16, 8, 4, 2, 4)
+        }
+    }
     if (D <= 64) {
         if (!form) form = tiles <= 180 ? 1 : tiles <= 600 ? 2 : 3;
         if (form == 1) DL_CASE(4, 16, 2, 4, 3)
