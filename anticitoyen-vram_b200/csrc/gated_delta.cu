@@ -309,9 +309,11 @@ ACV_API int acv_gated_delta_blocks(const float* proj, int ld, const float* wt, c
 
 // ----------------------------------------------------------------------------- one token a request, everything
 // A block of 256 threads a (request, head).  A thread holds RPT rows of four neighbouring columns: c4 = DV / 4 threads cover a
-// row, NG = 256 / c4 groups of rows stand side by side; sums over rows pass through shared memory.
-template <typename T, int RPT>
-__global__ void __launch_bounds__(256)
+// row, NG = 256 / c4 groups of rows stand side by side; sums over rows pass through shared memory.  What the block needs beside
+// the state is asked for in front of it and all at once (FEW: up to four taps and two channels of the convolution a thread),
+// so that no chain of loads stands between the state's arrival and its way back.
+template <typename T, int RPT, bool FEW>
+__global__ void __launch_bounds__(256, RPT <= 16 ? 2 : 1)
 gated_delta_step_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ wt, const float* __restrict__ rate,
                         const float* __restrict__ shift, const float* __restrict__ weight, float eps, float* ring,
                         const int* __restrict__ ring_slots, float* __restrict__ state, const int* __restrict__ slots,
@@ -333,25 +335,55 @@ gated_delta_step_kernel(const float* __restrict__ proj, int ld, const float* __r
     float* st = state + ((size_t)slots[seq] * H + h) * D * DV;
     const int g = tid / c4n, col = (tid - g * c4n) << 2;
     const bool owner = g < NG;
+    const float* row = proj + (size_t)t * ld;
+    const int pos = positions[t];
+    float* slot = ring + (size_t)ring_slots[seq] * K * C;
+    auto channel = [&](int i) { return i < D ? grp * D + i : i < 2 * D ? G * D + grp * D + i - D : 2 * G * D + h * DV + i - 2 * D; };
+    const float b_in = row[C + H * DV + h], a_in = row[C + H * DV + H + h], rate_h = rate[h], shift_h = shift[h];
+    float x[2], tap[2][4], kept[2][3];
+    if constexpr (FEW) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            const int i = tid + 256 * n, c = channel(i);
+            const bool in = i < 2 * D + DV;
+            x[n] = in ? row[c] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) tap[n][j] = in && j < K ? wt[(size_t)(K - 1 - j) * C + c] : 0.f;
+#pragma unroll
+            for (int j = 1; j < 4; ++j) kept[n][j - 1] = in && j < K && j <= pos ? slot[(size_t)((pos - j) % K) * C + c] : 0.f;
+        }
+    }
     float4 S[RPT];
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
         const int d = g + i * NG;
         S[i] = owner && d < D ? *reinterpret_cast<const float4*>(st + (size_t)d * DV + col) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    const float* row = proj + (size_t)t * ld;
-    const int pos = positions[t];
-    float* slot = ring + (size_t)ring_slots[seq] * K * C;
-    for (int i = tid; i < 2 * D + DV; i += 256) {
-        const int c = i < D ? grp * D + i : i < 2 * D ? G * D + grp * D + i - D : 2 * G * D + h * DV + i - 2 * D;
-        const float x = row[c];
-        float y = wt[(size_t)(K - 1) * C + c] * x;
-        for (int j = 1; j < K && j <= pos; ++j) y = fmaf(wt[(size_t)(K - 1 - j) * C + c], slot[(size_t)((pos - j) % K) * C + c], y);
+    const float z0 = tid < DV ? row[C + h * DV + tid] : 0.f, w0 = tid < DV ? weight[(size_t)h * DV + tid] : 0.f;
+    auto take = [&](int i, int c, float in, float y) {
         // the heads of a group share their q and k channels: one of them keeps the input (in the row that nobody reads now)
-        if (K > 1 && (i >= 2 * D || h == grp * r)) slot[(size_t)(pos % K) * C + c] = x;
+        if (K > 1 && (i >= 2 * D || h == grp * r)) slot[(size_t)(pos % K) * C + c] = in;
         (i < D ? qs[i] : i < 2 * D ? ks[i - D] : vs[i - 2 * D]) = gd_silu(y);
+    };
+    if constexpr (FEW) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            const int i = tid + 256 * n;
+            float y = tap[n][0] * x[n];
+#pragma unroll
+            for (int j = 1; j < 4; ++j) y = fmaf(tap[n][j], kept[n][j - 1], y);
+            if (i < 2 * D + DV) take(i, channel(i), x[n], y);
+        }
+    } else {
+        for (int i = tid; i < 2 * D + DV; i += 256) {
+            const int c = channel(i);
+            const float in = row[c];
+            float y = wt[(size_t)(K - 1) * C + c] * in;
+            for (int j = 1; j < K && j <= pos; ++j) y = fmaf(wt[(size_t)(K - 1 - j) * C + c], slot[(size_t)((pos - j) % K) * C + c], y);
+            take(i, c, in, y);
+        }
     }
-    const float beta = gd_sigmoid(row[C + H * DV + h]), dec = gd_decay(row[C + H * DV + H + h], rate[h], shift[h]);
+    const float beta = gd_sigmoid(b_in), dec = gd_decay(a_in, rate_h, shift_h);
     __syncthreads();
     float qq = 0.f, kk = 0.f;               // (every warp for itself)
     for (int e = lane; e < D; e += 32) {
@@ -406,7 +438,7 @@ gated_delta_step_kernel(const float* __restrict__ proj, int ld, const float* __r
     const float inv_rms = 1.f / sqrtf(block_sum(sq, red) / (float)DV + eps);
     for (int c = tid; c < DV; c += 256)
         out[(size_t)t * ldo + (size_t)h * DV + c] =
-            from_f32<T>(us[c] * inv_rms * weight[(size_t)h * DV + c] * gd_silu(row[C + h * DV + c]));
+            from_f32<T>(us[c] * inv_rms * (c == tid ? w0 : weight[(size_t)h * DV + c]) * gd_silu(c == tid ? z0 : row[C + h * DV + c]));
 }
 
 static size_t gated_delta_step_smem(int D, int DV) {
@@ -434,19 +466,23 @@ ACV_API int acv_gated_delta_step(const float* proj, int ld, const float* wt, con
     const int NG = 256 / (DV / 4), rows = (D + NG - 1) / NG;
     const size_t smem = gated_delta_step_smem(D, DV);
     const dim3 grid(n_seqs, H);
+    const bool few = K <= 4 && 2 * D + DV <= 512;
+#define GS_LAUNCH(TT, N, F)                                                                                                 \
+    acv_launch(PDL_ATTN, gated_delta_step_kernel<TT, N, F>, grid, 256, smem, stream, proj, ld, wt, rate, shift, weight, eps, \
+               ring, ring_slots, state, slots, positions, cu_q, (TT*)out, ldo, G, H, D, DV, K)
 #define GS_CASE(N)                                                                                                          \
     if (rows <= N) {                                                                                                        \
-        if (dtype == ACV_F32)                                                                                               \
-            acv_launch(PDL_ATTN, gated_delta_step_kernel<float, N>, grid, 256, smem, stream, proj, ld, wt, rate, shift, weight, \
-                       eps, ring, ring_slots, state, slots, positions, cu_q, (float*)out, ldo, G, H, D, DV, K);             \
-        else if (dtype == ACV_BF16)                                                                                         \
-            acv_launch(PDL_ATTN, gated_delta_step_kernel<bf16, N>, grid, 256, smem, stream, proj, ld, wt, rate, shift, weight, \
-                       eps, ring, ring_slots, state, slots, positions, cu_q, (bf16*)out, ldo, G, H, D, DV, K);              \
-        else                                                                                                                \
+        if (dtype == ACV_F32) {                                                                                             \
+            if (few) GS_LAUNCH(float, N, true); else GS_LAUNCH(float, N, false);                                            \
+        } else if (dtype == ACV_BF16) {                                                                                     \
+            if (few) GS_LAUNCH(bf16, N, true); else GS_LAUNCH(bf16, N, false);                                              \
+        } else {                                                                                                            \
             return ACV_ERR_DTYPE;                                                                                           \
+        }                                                                                                                   \
         return acv_launch_status();                                                                                         \
     }
     GS_CASE(1) GS_CASE(2) GS_CASE(4) GS_CASE(8) GS_CASE(16) GS_CASE(32)
 #undef GS_CASE
+#undef GS_LAUNCH
     return ACV_ERR_SIZE;
 }
