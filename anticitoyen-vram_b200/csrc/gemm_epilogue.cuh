@@ -75,7 +75,7 @@ __device__ __forceinline__ bf16 swiglu_pair(float gate, float up) {
 
 // The tanh form of gelu in float: 0.5 z (1 + tanh y) = z / (1 + exp(-2 y)), y = sqrt(2/pi) (z + 0.044715 z^3).  The
 // exponential and the quotient are the hardware's approximations, a few units in the last place of a float, in front of a
-// rounding to bfloat16: the four epilogue warps of a tile would otherwise wait for tanhf (2048 x 9216 x 2048: 28 us of it).
+// rounding to bfloat16.
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
     return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }

@@ -212,6 +212,8 @@ GATE_CASES = [
     (8, 8, 64, 64, [6000, 5000], [1, 1], 0),                # and merged by the last arriver
     (2, 1, 128, 8, [131, 9], [1, 1], 64),                   # small pages
     (5, 5, 64, 128, [140, 500], [139, 3], 0),
+    (40, 2, 64, 16, [90, 61, 17], [30, 1, 1], 50),          # more heads to a key head than the tensor-core kernels take
+    (4, 2, 256, 16, [50, 33], [20, 1], 20),
 ]
 
 
